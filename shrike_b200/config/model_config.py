@@ -341,6 +341,39 @@ class GatedLinearRecurrenceSpec(PartSpec):
 
 
 @dataclass(frozen=True)
+class ChannelDeltaSpec(PartSpec):
+    """A delta rule whose state decays per key channel.  q and k have `num_kv_heads` heads of `head_dim`, v has
+    `num_heads` heads of `value_dim`; head h uses q/k head h // (num_heads / num_kv_heads).  q, k and v each pass a
+    causal convolution of `conv` taps over time per channel and a SiLU; q and k are divided per head by
+    sqrt(sum of squares + `unit_eps`), q also multiplied by head_dim^(-1/2).  Per head, from S = 0,
+
+        S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+
+    with beta = sigmoid(Wb x) and g = exp(-exp(A_log) softplus(Wa2 Wa1 x + dt_bias)) per key channel.  Every head's o
+    is divided by its root mean square, scaled by one weight of the head's size that all heads share, multiplied by
+    sigmoid(Wg2 Wg1 x) and projected.  `decay_rank` and `gate_rank`, the rows of Wa1 and Wg1, are what a model's
+    tensors say (None); a number here is used for random weights.  Gates, state and recurrence are 32-bit."""
+
+    width: int
+    num_heads: int
+    num_kv_heads: int
+    head_dim: int
+    value_dim: int
+    conv: int
+    eps: float
+    unit_eps: float = 1e-6
+    decay_rank: int | None = None
+    gate_rank: int | None = None
+    kind: str = field(init=False, default="channel_delta")
+
+    def __post_init__(self):
+        if self.num_heads % self.num_kv_heads:
+            raise ConfigError(f"heads={self.num_heads} is not a multiple of kv_heads={self.num_kv_heads}")
+        if not 1 <= self.conv <= 32:
+            raise ConfigError(f"a short convolution has 1 to 32 taps, got {self.conv}")
+
+
+@dataclass(frozen=True)
 class HyperConnectionSpec(PartSpec):
     """How a sublayer's result y joins a residual of `streams` streams x_1 .. x_S, and how the sublayer reads them:
     u = sum_s in[s] x_s is what the sublayer's norm sees; afterwards, all streams at once from the old ones,
@@ -427,6 +460,16 @@ class GatedMLPSpec(PartSpec):
 
 
 @dataclass(frozen=True)
+class MLPSpec(PartSpec):
+    """Dense feed-forward without a gate: down(act(up(x))).  `activation` "relu2": the square of relu."""
+
+    width: int
+    intermediate: int
+    activation: str = "relu2"
+    kind: str = field(init=False, default="mlp")
+
+
+@dataclass(frozen=True)
 class RoutedExpertsSpec(PartSpec):
     """A mixture of gated feed-forward experts: router logits in 32-bit, softmax over all experts,
     the `top` largest, their scores divided by the sum of those (+ `renorm_eps`); the output is the
@@ -448,6 +491,14 @@ class RoutedExpertsSpec(PartSpec):
     scoring: str = "softmax"
     renormalise: bool = True
     weight_on: str = "output"
+    # the activation "clamped_swish" clamps at `limit` (the shared expert at `shared_limit`), see `GatedMLPSpec`
+    limit: float | None = None
+    shared_limit: float | None = None
+    # `correction`: a learned number per expert is added to the scores for the choice; the weights are without it
+    correction: bool = False
+    # `groups` (count, keep): the experts form `count` equal groups of neighbours, a group counts as much as its best
+    # expert, and only experts of the best `keep` groups can be chosen
+    groups: tuple | None = None
     kind: str = field(init=False, default="routed_experts")
 
     def __post_init__(self):
@@ -457,6 +508,14 @@ class RoutedExpertsSpec(PartSpec):
             raise ConfigError(f"router scoring {self.scoring!r}; known: softmax, sigmoid")
         if self.weight_on not in ("output", "input"):
             raise ConfigError(f"an expert's weight sits on its output or its input, got {self.weight_on!r}")
+        if self.groups is not None:
+            count, keep = self.groups
+            if self.experts % count:
+                raise ConfigError(f"router: {self.experts} experts do not form {count} equal groups")
+            if not 1 <= keep <= count:
+                raise ConfigError(f"router: groups.keep={keep} must lie in 1..groups.count={count}")
+            if self.top > keep * (self.experts // count):
+                raise ConfigError(f"router: top={self.top} of {keep} groups of {self.experts // count} experts")
 
 
 @dataclass(frozen=True)
@@ -477,6 +536,28 @@ class TokenPositionEmbeddingSpec(PartSpec):
     width: int
     max_positions: int
     kind: str = field(init=False, default="token_position_embedding")
+
+
+@dataclass(frozen=True)
+class TokenSideTableSpec(PartSpec):
+    """A second table of token rows beside the embedding: `parts` parts of `dim` numbers a token, from which the
+    model's `TokenSideSpec` parts read theirs."""
+
+    vocab: int
+    parts: int
+    dim: int
+    kind: str = field(init=False, default="token_side_table")
+
+
+@dataclass(frozen=True)
+class TokenSideSpec(PartSpec):
+    """A further input a layer takes for its tokens: with e part `index` of the token's row of the side table,
+    y = proj (gelu_tanh(gate x) * e), x the residual itself; a norm of y is what joins the residual."""
+
+    width: int
+    dim: int
+    index: int
+    kind: str = field(init=False, default="token_side")
 
 
 @dataclass(frozen=True)
@@ -577,6 +658,8 @@ class ModelConfig:
     # a residual that is not one row a token (several streams): made from the embedding's output before the first
     # layer, turned into the final norm's input after the last
     residual: PartSpec | None = None
+    # a table of further inputs per token that layers read parts of (a `TokenSideTableSpec`)
+    side_table: PartSpec | None = None
 
     def __post_init__(self):
         if self.embedding is None:

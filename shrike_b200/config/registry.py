@@ -36,8 +36,10 @@ class TensorNames:
     embedding_prefix: str | None = None
     head_prefix: str | None = None
     pass_entry_prefix: str = "pass_entry."   # before the parameters of `ModelConfig.pass_entry` (role "pass_entry")
+    side_table_prefix: str = "side_table."   # before those of `ModelConfig.side_table` (role "side_table")
     # (role, a part's own parameter name) -> the name's last piece in this architecture's files; None:
-    # the part's own names are the files' names.  Roles: a layer's roles, "final_norm", "embedding", "head", "pass_entry".
+    # the part's own names are the files' names.  Roles: a layer's roles, "final_norm", "embedding", "head", "pass_entry",
+    # "side_table".
     local_name: Callable[[str, str], str] | None = None
 
     def local(self, role: str, local: str) -> str:
@@ -51,6 +53,9 @@ class TensorNames:
 
     def pass_entry_name(self, local: str) -> str:
         return self.pass_entry_prefix + self.local("pass_entry", local)
+
+    def side_table_name(self, local: str) -> str:
+        return self.side_table_prefix + self.local("side_table", local)
 
     def embedding_name(self, local: str) -> str:
         if local == "weight":

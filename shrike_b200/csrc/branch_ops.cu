@@ -3,6 +3,8 @@
 //
 //   norm_rows      resid += norm(branch) and the sum cast to the activation type, or
 //                  out = norm(resid[rows]) for a few gathered rows; RMS or layer norm, bias optional
+//   norm_join      resid += norm(branch) (+ a row), then out = norm(resid): the norm on one sublayer's output and
+//                  the norm before the next one from one pass over the row; also on gathered rows
 //   qk_norm_store  queries and keys of a fused q|k projection: RMS over the whole projection (all
 //                  heads at once), a position-dependent query temperature, keys into the key pages
 //                  and the keys as projected into the value pages
@@ -205,6 +207,138 @@ norm_rows_kernel(float* __restrict__ resid, const TD* __restrict__ branch, int p
       }
     }
   }
+}
+
+// ------------------------------------------------------------ a norm on both sides of a sublayer
+// One block per row; both RMS statistics from registers.  rows == nullptr: x = resid[row] + norm(sum of the branch's
+// partials) * branch_weight (+ row_add); resid[row] = x; out[row] = x / sqrt(mean(x^2) + eps) * weight.  rows !=
+// nullptr: the same for row rows[r] into out[r], the residual stays.  PT: groups of VEC elements a thread may hold; PT
+// = 1 (few rows: latency counts) reads the weights before the wait, no kernel writes them.
+template <typename TO, int VEC, int PT>
+__global__ void __launch_bounds__(PT == 4 ? 256 : 1024, PT == 4 ? 4 : 1)
+norm_join_kernel(float* __restrict__ resid, const float* __restrict__ branch, int partials, long long partial_stride,
+                 const int* __restrict__ rows, const float* __restrict__ branch_weight, float branch_eps,
+                 const float* __restrict__ row_add, const float* __restrict__ weight, float eps, TO* __restrict__ out, int width) {
+  __shared__ float scratch[33];
+  constexpr bool EARLY = PT == 1;
+  let_dependents_start();
+  const int groups = width / VEC;
+  float early_b[VEC] = {}, early_w[VEC] = {}, early_r[VEC] = {};
+  if (EARLY && threadIdx.x < groups) {
+    const int at = threadIdx.x * VEC;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+      early_b[e] = branch_weight[at + e];
+      early_w[e] = weight[at + e];
+      early_r[e] = row_add != nullptr ? row_add[at + e] : 0.f;
+    }
+  }
+  wait_for_previous();
+  const int out_row = blockIdx.x;
+  const int row = rows != nullptr ? rows[out_row] : out_row;
+  float* x = resid + static_cast<size_t>(row) * width;
+  const float* d = branch + static_cast<size_t>(row) * width;
+  TO* y = out + static_cast<size_t>(out_row) * width;
+  float held[PT][VEC], base[PT][VEC];
+  float squares = 0.f;
+#pragma unroll
+  for (int it = 0; it < PT; ++it) {
+    const int g = threadIdx.x + it * blockDim.x;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) held[it][e] = base[it][e] = 0.f;
+    if (g < groups) {
+      if constexpr (VEC == 4) {
+        load4<float>(x + g * 4, base[it]);
+        if (EARLY) sum_partials4(d + g * 4, partial_stride, partials, held[it]);
+        else load_sum4_in_turn<float>(d + g * 4, partial_stride, partials, held[it]);
+      } else {
+        base[it][0] = x[g];
+        held[it][0] = sum_partials(d + g, partial_stride, partials);
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) squares = fmaf(held[it][e], held[it][e], squares);
+    }
+  }
+  const float gain = 1.0f / sqrtf(block_sum(squares, scratch) / static_cast<float>(width) + branch_eps);
+  squares = 0.f;
+#pragma unroll
+  for (int it = 0; it < PT; ++it) {
+    const int g = threadIdx.x + it * blockDim.x;
+    if (g < groups) {
+      float w[VEC], add[VEC] = {};
+      if (EARLY) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) { w[e] = early_b[e]; add[e] = early_r[e]; }
+      } else if constexpr (VEC == 4) {
+        load4<float>(branch_weight + g * 4, w);
+        if (row_add != nullptr) load4<float>(row_add + g * 4, add);
+      } else {
+        w[0] = branch_weight[g];
+        if (row_add != nullptr) add[0] = row_add[g];
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        float v = __fadd_rn(base[it][e], __fmul_rn(__fmul_rn(held[it][e], gain), w[e]));
+        if (row_add != nullptr) v = __fadd_rn(v, add[e]);
+        held[it][e] = v;
+        squares = fmaf(v, v, squares);
+      }
+      if (rows == nullptr) {
+        if constexpr (VEC == 4) store4<float>(x + g * 4, held[it]);
+        else x[g] = held[it][0];
+      }
+    }
+  }
+  const float scale = 1.0f / sqrtf(block_sum(squares, scratch) / static_cast<float>(width) + eps);
+#pragma unroll
+  for (int it = 0; it < PT; ++it) {
+    const int g = threadIdx.x + it * blockDim.x;
+    if (g < groups) {
+      float w[VEC], r[VEC];
+      if (EARLY) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) w[e] = early_w[e];
+      } else if constexpr (VEC == 4) {
+        load4<float>(weight + g * 4, w);
+      } else {
+        w[0] = weight[g];
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) r[e] = __fmul_rn(__fmul_rn(held[it][e], scale), w[e]);
+      if constexpr (VEC == 4) store4<TO>(y + g * 4, r);
+      else y[g] = from_float<TO>(r[0]);
+    }
+  }
+}
+
+template <typename TO>
+static int launch_norm_join(float* resid, const float* branch, int partials, long long partial_stride, const int* rows,
+                            const float* branch_weight, float branch_eps, const float* row_add, const float* weight, float eps,
+                            void* out, int n, int width, cudaStream_t stream) {
+  const uintptr_t addresses = reinterpret_cast<uintptr_t>(resid) | reinterpret_cast<uintptr_t>(branch) |
+                              reinterpret_cast<uintptr_t>(branch_weight) | reinterpret_cast<uintptr_t>(row_add) |
+                              reinterpret_cast<uintptr_t>(weight) | reinterpret_cast<uintptr_t>(out);
+  const bool vec = width % 4 == 0 && addresses % 16 == 0 && (partials == 1 || partial_stride % 4 == 0);
+  const int groups = vec ? width / 4 : width;
+  const bool few = n <= 256 && groups <= 1024;
+  int threads = ((few ? groups : (groups + 3) / 4) + 31) / 32 * 32;
+  threads = threads < 64 ? 64 : (threads > 1024 ? 1024 : threads);
+  if (static_cast<long long>(threads) * MAX_PER_THREAD < groups) return SHRIKE_BAD_ARGUMENT;
+  const bool four = !few && threads <= 256;
+#define SHRIKE_NORM_JOIN_LAUNCH(V, P)                                                                                       \
+  launch_dependent(norm_join_kernel<TO, V, P>, n, threads, 0, stream, resid, branch, partials, partial_stride, rows,         \
+                   branch_weight, branch_eps, row_add, weight, eps, static_cast<TO*>(out), width)
+#define SHRIKE_NORM_JOIN_CASE(V)                     \
+  do {                                               \
+    if (few) SHRIKE_NORM_JOIN_LAUNCH(V, 1);          \
+    else if (four) SHRIKE_NORM_JOIN_LAUNCH(V, 4);    \
+    else SHRIKE_NORM_JOIN_LAUNCH(V, MAX_PER_THREAD); \
+  } while (0)
+  if (vec) SHRIKE_NORM_JOIN_CASE(4);
+  else SHRIKE_NORM_JOIN_CASE(1);
+#undef SHRIKE_NORM_JOIN_CASE
+#undef SHRIKE_NORM_JOIN_LAUNCH
+  return SHRIKE_OK;
 }
 
 // ------------------------------------------------------------ queries and keys of a q|k projection
@@ -432,6 +566,27 @@ SHRIKE_API int shrike_norm_rows(float* resid, const void* branch, int branch_dty
     else SHRIKE_NORM_ROWS(float, float);
   }
 #undef SHRIKE_NORM_ROWS
+  if (status != SHRIKE_OK) return status;
+  return shrike_launch_status();
+}
+
+// rows == null: resid += norm(branch) * branch_weight (+ row_add), out = norm(resid) * weight, n rows; else out[r] for row
+// rows[r], n = number of rows, the residual stays.  branch float32 [*, width] or a stack of `partials`.
+SHRIKE_API int shrike_norm_join(float* resid, const float* branch, int partials, long long partial_stride, const int* rows,
+                                const float* branch_weight, float branch_eps, const float* row_add, const float* weight,
+                                float eps, void* out, int out_dtype, int n, int width, cudaStream_t stream) {
+  using namespace branch;
+  if (n <= 0) return SHRIKE_OK;
+  if (width <= 0 || partials < 1 || branch == nullptr || branch_weight == nullptr || weight == nullptr || out == nullptr)
+    return SHRIKE_BAD_ARGUMENT;
+  int status;
+  if (out_dtype == SHRIKE_BF16)
+    status = launch_norm_join<__nv_bfloat16>(resid, branch, partials, partial_stride, rows, branch_weight, branch_eps, row_add,
+                                             weight, eps, out, n, width, stream);
+  else if (out_dtype == SHRIKE_F32)
+    status = launch_norm_join<float>(resid, branch, partials, partial_stride, rows, branch_weight, branch_eps, row_add, weight,
+                                     eps, out, n, width, stream);
+  else return SHRIKE_BAD_ARGUMENT;
   if (status != SHRIKE_OK) return status;
   return shrike_launch_status();
 }

@@ -171,6 +171,14 @@ template <typename T> __device__ __forceinline__ float act_times(int act, float 
   return act == SHRIKE_ACT_GELU_TANH ? gelu_tanh_times<T>(g, u) : silu_times<T>(g, u);
 }
 
+// Activations of an ungated feed-forward: relu2 is max(z, 0)^2, formed in float32 and rounded once.
+enum : int { SHRIKE_PLAIN_NONE = 0, SHRIKE_PLAIN_RELU2 = 1 };
+template <typename T> __device__ __forceinline__ T plain_act(int act, T z) {
+  if (act != SHRIKE_PLAIN_RELU2) return z;
+  const float v = fmaxf(to_float(z), 0.f);
+  return from_float<T>(__fmul_rn(v, v));
+}
+
 // The first key a query at position `last` sees.  span > 0: the `span` latest keys (a sliding window);
 // span < 0: positions are cut into runs of -span counted from position 0, and a query sees its own run only;
 // span == 0: every key.  Never decreases as `last` grows, so a tile's first row gives the tile's first key.

@@ -377,6 +377,91 @@ SHRIKE_API int shrike_silu_mul(const void* gate_up, void* out, int dtype, int n,
   return shrike_act_mul(gate_up, out, dtype, n, inter, block, SHRIKE_ACT_SILU, stream);
 }
 
+// ------------------------------------------------ activation of an ungated feed-forward, in place
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) plain_act_kernel(T* __restrict__ x, long long groups, int act) {
+  let_dependents_start();
+  wait_for_previous();
+  struct alignas(sizeof(T) * VEC) Pack { T v[VEC]; };
+  const long long stride = static_cast<long long>(gridDim.x) * blockDim.x;
+  for (long long g = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; g < groups; g += 2 * stride) {
+    Pack p = *reinterpret_cast<const Pack*>(x + g * VEC), q;   // two groups in flight
+    const bool more = g + stride < groups;
+    if (more) q = *reinterpret_cast<const Pack*>(x + (g + stride) * VEC);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) p.v[j] = plain_act<T>(act, p.v[j]);
+    *reinterpret_cast<Pack*>(x + g * VEC) = p;
+    if (more) {
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) q.v[j] = plain_act<T>(act, q.v[j]);
+      *reinterpret_cast<Pack*>(x + (g + stride) * VEC) = q;
+    }
+  }
+}
+
+template <typename T>
+static void launch_plain_act(void* x, long long count, int act, cudaStream_t stream) {
+  constexpr int WIDE = 16 / sizeof(T);
+  const bool vec = count % WIDE == 0 && reinterpret_cast<uintptr_t>(x) % 16 == 0;
+  const long long groups = vec ? count / WIDE : count;
+  const unsigned blocks = static_cast<unsigned>(max(1LL, min((groups + 511) / 512, 16384LL)));
+  if (vec) launch_dependent(plain_act_kernel<T, WIDE>, blocks, 256, 0, stream, static_cast<T*>(x), groups, act);
+  else launch_dependent(plain_act_kernel<T, 1>, blocks, 256, 0, stream, static_cast<T*>(x), groups, act);
+}
+
+// x (`count` elements) <- act(x), `act` one of SHRIKE_PLAIN_*.
+SHRIKE_API int shrike_plain_act(void* x, int dtype, long long count, int act, cudaStream_t stream) {
+  if (count <= 0) return SHRIKE_OK;
+  if (act != SHRIKE_PLAIN_RELU2) return SHRIKE_BAD_ARGUMENT;
+  if (dtype == SHRIKE_F32) launch_plain_act<float>(x, count, act, stream);
+  else if (dtype == SHRIKE_BF16) launch_plain_act<__nv_bfloat16>(x, count, act, stream);
+  else return SHRIKE_BAD_ARGUMENT;
+  return shrike_launch_status();
+}
+
+// ------------------------------------------------ a side input's gate times the token's own row
+// gate [partials][n][padded] float32; out[token][c] = gelu_tanh(gate) * table[id][first + c] for c < dim, zero up to
+// `padded`.  A token id of -1 - r stands for previous[r], as in the embedding.
+template <typename T>
+__global__ void __launch_bounds__(256) side_gate_kernel(const float* __restrict__ gate, int partials, long long stride,
+                                                        const T* __restrict__ table, int table_width, int vocab,
+                                                        const int* __restrict__ ids, const int* __restrict__ previous,
+                                                        int num_previous, int first, int dim, int padded, T* __restrict__ out,
+                                                        int n) {
+  let_dependents_start();
+  wait_for_previous();
+  const long long total = static_cast<long long>(n) * padded;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const int token = static_cast<int>(i / padded), c = static_cast<int>(i - static_cast<long long>(token) * padded);
+    float v = 0.f;
+    if (c < dim) {
+      int id = ids[token];
+      if (id < 0 && previous != nullptr) id = previous[min(-1 - id, num_previous - 1)];
+      id = min(max(id, 0), vocab - 1);   // never read outside the table
+      v = gelu_tanh_times<T>(sum_partials(gate + i, stride, partials), to_float(table[static_cast<size_t>(id) * table_width + first + c]));
+    }
+    out[i] = from_float<T>(v);
+  }
+}
+
+SHRIKE_API int shrike_side_gate(const float* gate, int partials, long long stride, const void* table, int dtype, int table_width,
+                                int vocab, const int* ids, const int* previous, int num_previous, int first, int dim,
+                                int padded, void* out, int n, cudaStream_t stream) {
+  if (n <= 0) return SHRIKE_OK;
+  if (dim < 1 || padded < dim || first < 0 || first + dim > table_width || vocab < 1 || partials < 1) return SHRIKE_BAD_ARGUMENT;
+  if (num_previous < 1) previous = nullptr;
+  const long long total = static_cast<long long>(n) * padded;
+  const unsigned blocks = static_cast<unsigned>(min((total + 255) / 256, 65536LL));
+  if (dtype == SHRIKE_F32)
+    launch_dependent(side_gate_kernel<float>, blocks, 256, 0, stream, gate, partials, stride, static_cast<const float*>(table), table_width,
+                     vocab, ids, previous, num_previous, first, dim, padded, static_cast<float*>(out), n);
+  else if (dtype == SHRIKE_BF16)
+    launch_dependent(side_gate_kernel<__nv_bfloat16>, blocks, 256, 0, stream, gate, partials, stride, static_cast<const __nv_bfloat16*>(table),
+                     table_width, vocab, ids, previous, num_previous, first, dim, padded, static_cast<__nv_bfloat16*>(out), n);
+  else return SHRIKE_BAD_ARGUMENT;
+  return shrike_launch_status();
+}
+
 // --------------------------------------- bias + rotary + key/value store
 // One thread per rotation pair; blockIdx.x is the token, blockIdx.y a slice of the
 // (head, pair) space over the q, k and v heads (many slices for few tokens, one for many).  qkv is the float32 result of the fused projection,

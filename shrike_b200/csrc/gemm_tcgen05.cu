@@ -71,6 +71,7 @@ struct Args {
   int gated;            // nonzero (1 + activation code): the weight rows come in runs of 16 gate rows and the 16 up
                         // rows of the same features; out is [T][N / 2] bfloat16 = act(gate) * up
   float act_limit;      // the clamp of the activation SHRIKE_ACT_CLAMPED_SWISH
+  int plain_act;        // SHRIKE_PLAIN_*: applied to the result, rounded to bfloat16 first, of an ungated product
 };
 
 __global__ void __launch_bounds__(THREADS, 3)
@@ -224,7 +225,7 @@ gemm_swap_ab_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
             const size_t at = static_cast<size_t>(t) * args.n + row;
             if (partial) static_cast<float*>(args.out)[static_cast<size_t>(split) * args.tokens * args.n + at] = value;
             else if (args.out_dtype == SHRIKE_F32) static_cast<float*>(args.out)[at] = value;
-            else static_cast<__nv_bfloat16*>(args.out)[at] = __float2bfloat16_rn(value);
+            else static_cast<__nv_bfloat16*>(args.out)[at] = plain_act(args.plain_act, __float2bfloat16_rn(value));
           }
         }
       }
@@ -266,7 +267,8 @@ SHRIKE_API int shrike_gemm_tc_splits(int tokens, int n, int k) {
 // strides) and both 16-byte aligned.  splits == 1: out is [tokens, n] of out_dtype.
 // splits > 1 (as shrike_gemm_tc_splits says): out is [splits, tokens, n] float32.
 static int launch_gemm_tc(const void* x, const void* w, const float* bias, void* out, int out_dtype, int tokens,
-                          int n, int k, int splits, int gated, int* status, cudaStream_t stream, float act_limit = 0.f) {
+                          int n, int k, int splits, int gated, int* status, cudaStream_t stream, float act_limit = 0.f,
+                          int plain_act = SHRIKE_PLAIN_NONE) {
   using namespace tc;
   if (tokens <= 0 || n <= 0) return SHRIKE_OK;
   if (k <= 0 || k % 8 || splits < 1 || (out_dtype != SHRIKE_F32 && out_dtype != SHRIKE_BF16)) return SHRIKE_BAD_ARGUMENT;
@@ -314,6 +316,7 @@ static int launch_gemm_tc(const void* x, const void* w, const float* bias, void*
   args.stages = stages;
   args.gated = gated;
   args.act_limit = act_limit;
+  args.plain_act = plain_act;
   args.out_dtype = out_dtype;
   cudaLaunchConfig_t config = {};
   config.gridDim = dim3((n + BM - 1) / BM, splits, token_tiles);
@@ -333,6 +336,14 @@ static int launch_gemm_tc(const void* x, const void* w, const float* bias, void*
 SHRIKE_API int shrike_gemm_tc(const void* x, const void* w, const float* bias, void* out, int out_dtype, int tokens,
                               int n, int k, int splits, int* status, cudaStream_t stream) {
   return launch_gemm_tc(x, w, bias, out, out_dtype, tokens, n, k, splits, 0, status, stream);
+}
+
+// An ungated feed-forward's first product with its activation: out [tokens, n] bfloat16 = act(x w^T), the product
+// rounded to bfloat16 before the activation; `act` one of SHRIKE_PLAIN_*.
+SHRIKE_API int shrike_gemm_tc_act(const void* x, const void* w, void* out, int tokens, int n, int k, int act, int* status,
+                                  cudaStream_t stream) {
+  if (act != SHRIKE_PLAIN_RELU2) return SHRIKE_BAD_ARGUMENT;
+  return launch_gemm_tc(x, w, nullptr, out, SHRIKE_BF16, tokens, n, k, 1, 0, status, stream, 0.f, act);
 }
 
 // The gated feed-forward's first product with its activation: w [n, k] holds, in runs of 32 rows,

@@ -911,7 +911,7 @@ template <typename T>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 route_top_kernel(const T* __restrict__ x, const float* __restrict__ router, const float* __restrict__ shared_gate,
                  float* __restrict__ weights, int n, int width, int experts, int top, int columns, float renorm_eps,
-                 int sigmoid_scores, int renormalise) {
+                 int sigmoid_scores, int renormalise, const float* __restrict__ correction, int group_count, int group_keep) {
   extern __shared__ float route_shared[];   // [ROUTE_WARPS][rows] sums of the warps, then [rows] scores in the first row
   let_dependents_start();
   wait_for_previous();
@@ -988,6 +988,57 @@ route_top_kernel(const T* __restrict__ x, const float* __restrict__ router, cons
   }
   __syncwarp();
   float chosen_sum = 0.f;
+  if (correction != nullptr || group_count > 0) {
+    // the choice goes by score + correction among the experts of the best groups; the weights are the scores.  Rows one
+    // and two of the warps' sums are used up: they hold the choice scores and the groups' best.
+    float* choice = route_shared + rows;
+    float* group_best = choice + rows;
+    for (int e = lane; e < experts; e += 32) {
+      if (sigmoid_scores) score[e] = 1.0f / (1.0f + expf(-score[e]));
+      choice[e] = score[e] + (correction != nullptr ? correction[e] : 0.f);
+    }
+    __syncwarp();
+    if (group_count > 0) {
+      const int each = experts / group_count;
+      for (int g = lane; g < group_count; g += 32) {
+        float top_of = -INFINITY;
+        for (int e = g * each; e < (g + 1) * each; ++e) top_of = fmaxf(top_of, choice[e]);
+        group_best[g] = top_of;
+      }
+      __syncwarp();
+      for (int e = lane; e < experts; e += 32) {
+        const int g = e / each;
+        const float own = group_best[g];
+        int before = 0;   // groups that rank before this one; the lower index wins a tie
+        for (int other = 0; other < group_count; ++other)
+          before += group_best[other] > own || (group_best[other] == own && other < g);
+        if (before >= group_keep) choice[e] = -INFINITY;
+      }
+      __syncwarp();
+    }
+    for (int round = 0; round < top; ++round) {
+      float mine = -INFINITY;
+      int where = experts;
+      for (int e = lane; e < experts; e += 32)
+        if (choice[e] > mine) { mine = choice[e]; where = e; }
+#pragma unroll
+      for (int offset = 16; offset > 0; offset >>= 1) {
+        const float other = __shfl_xor_sync(0xffffffffu, mine, offset);
+        const int other_where = __shfl_xor_sync(0xffffffffu, where, offset);
+        if (other > mine || (other == mine && other_where < where)) { mine = other; where = other_where; }
+      }
+      if (where < experts) {
+        const float weight = score[where];
+        chosen_sum += weight;
+        if (lane == 0) {
+          out[where] = weight;
+          choice[where] = -INFINITY;
+        }
+      }
+      __syncwarp();
+    }
+    top = 0;   // the choice is made
+  }
   // `top` rounds of a warp-wide argmax; the lowest index wins a tie.  A pick is marked by a value below every score.
   const float below = sigmoid_scores ? -INFINITY : -1.f;
   for (int round = 0; round < top; ++round) {
@@ -1022,7 +1073,7 @@ route_top_kernel(const T* __restrict__ x, const float* __restrict__ router, cons
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
 act_mul_blocks_kernel(const T* __restrict__ gate_up, const float* __restrict__ weights, T* __restrict__ out, int n, int inter,
-                      int experts, int each, int columns, int act, float limit, int weight_input) {
+                      int experts, int each, int columns, int act, float limit, int weight_input, float shared_limit) {
   let_dependents_start();
   wait_for_previous();
   // VEC consecutive columns a thread (one 16-byte access each way when VEC > 1; the launcher sees to it that a
@@ -1037,6 +1088,7 @@ act_mul_blocks_kernel(const T* __restrict__ gate_up, const float* __restrict__ w
       const int c = group * VEC;
       const int block = c < experts * each ? c / each : experts;
       const float share = w[block];
+      const float clamp = block < experts ? limit : shared_limit;
       Pack r;
       if (share == 0.f) {
         // an expert the token did not choose contributes exactly nothing, whatever its gate and up columns hold
@@ -1048,8 +1100,8 @@ act_mul_blocks_kernel(const T* __restrict__ gate_up, const float* __restrict__ w
         for (int j = 0; j < VEC; ++j) {
           // the weight on the expert's INPUT reaches gate and up alike (both are linear in it): act(w g) (w u)
           const float gate = to_float(g.v[j]), up = to_float(u.v[j]);
-          r.v[j] = from_float<T>(weight_input ? act_times<T>(act, __fmul_rn(share, gate), __fmul_rn(share, up), limit)
-                                              : __fmul_rn(act_times<T>(act, gate, up, limit), share));
+          r.v[j] = from_float<T>(weight_input ? act_times<T>(act, __fmul_rn(share, gate), __fmul_rn(share, up), clamp)
+                                              : __fmul_rn(act_times<T>(act, gate, up, clamp), share));
         }
       }
       *reinterpret_cast<Pack*>(o + c) = r;
@@ -1246,21 +1298,35 @@ SHRIKE_API int shrike_matrix_memory_out(const float* numerator, const float* den
 // when shared_gate is null).
 // `sigmoid_scores`: an expert's score is the sigmoid of its logit instead of its softmax share; `renormalise` 0: the
 // chosen experts keep their scores as they are.
-SHRIKE_API int shrike_route_top_scores(const void* x, int dtype, const float* router, const float* shared_gate, float* weights, int n,
+// `correction` (float32 [experts], null: none) is added to the scores for the choice alone; `group_count` > 0: equal groups
+// of neighbouring experts, of which only those of the `group_keep` groups with the largest choice score can be chosen.
+SHRIKE_API int shrike_route_top_groups(const void* x, int dtype, const float* router, const float* shared_gate, float* weights, int n,
                                        int width, int experts, int top, int columns, float renorm_eps, int sigmoid_scores,
-                                       int renormalise, cudaStream_t stream) {
+                                       int renormalise, const float* correction, int group_count, int group_keep,
+                                       cudaStream_t stream) {
   if (n <= 0) return SHRIKE_OK;
   if (experts < 1 || top < 1 || top > experts || experts > 1024 || (columns != experts && columns != experts + 1)) return SHRIKE_BAD_ARGUMENT;
+  if (group_count > 0 && (experts % group_count || group_keep < 1 || group_keep > group_count || top > group_keep * (experts / group_count)))
+    return SHRIKE_BAD_ARGUMENT;
   const unsigned blocks = static_cast<unsigned>(n);
   const size_t smem = static_cast<size_t>(ROUTE_WARPS) * (experts + 1) * sizeof(float);
   if (dtype == SHRIKE_F32)
     launch_dependent(route_top_kernel<float>, blocks, ROUTE_WARPS * 32, smem, stream, static_cast<const float*>(x), router,
-                     shared_gate, weights, n, width, experts, top, columns, renorm_eps, sigmoid_scores, renormalise);
+                     shared_gate, weights, n, width, experts, top, columns, renorm_eps, sigmoid_scores, renormalise, correction,
+                     group_count, group_keep);
   else if (dtype == SHRIKE_BF16)
     launch_dependent(route_top_kernel<__nv_bfloat16>, blocks, ROUTE_WARPS * 32, smem, stream, static_cast<const __nv_bfloat16*>(x),
-                     router, shared_gate, weights, n, width, experts, top, columns, renorm_eps, sigmoid_scores, renormalise);
+                     router, shared_gate, weights, n, width, experts, top, columns, renorm_eps, sigmoid_scores, renormalise, correction,
+                     group_count, group_keep);
   else return SHRIKE_BAD_ARGUMENT;
   return shrike_launch_status();
+}
+
+SHRIKE_API int shrike_route_top_scores(const void* x, int dtype, const float* router, const float* shared_gate, float* weights, int n,
+                                       int width, int experts, int top, int columns, float renorm_eps, int sigmoid_scores,
+                                       int renormalise, cudaStream_t stream) {
+  return shrike_route_top_groups(x, dtype, router, shared_gate, weights, n, width, experts, top, columns, renorm_eps, sigmoid_scores,
+                                 renormalise, nullptr, 0, 0, stream);
 }
 
 SHRIKE_API int shrike_route_top(const void* x, int dtype, const float* router, const float* shared_gate, float* weights, int n,
@@ -1269,8 +1335,10 @@ SHRIKE_API int shrike_route_top(const void* x, int dtype, const float* router, c
 }
 
 // `weight_input` 1: an expert's weight multiplies its input, out = act(w gate) * (w up), instead of its output.
-SHRIKE_API int shrike_act_mul_blocks_at(const void* gate_up, const float* weights, void* out, int dtype, int n, int inter, int experts,
-                                        int each, int columns, int act, float limit, int weight_input, cudaStream_t stream) {
+// `shared_limit`: the clamp of the shared expert's columns.
+SHRIKE_API int shrike_act_mul_blocks_limits(const void* gate_up, const float* weights, void* out, int dtype, int n, int inter, int experts,
+                                            int each, int columns, int act, float limit, int weight_input, float shared_limit,
+                                            cudaStream_t stream) {
   if (n <= 0) return SHRIKE_OK;
   if (inter < 1 || experts < 1 || each < 1 || experts * each > inter || !known_activation(act)) return SHRIKE_BAD_ARGUMENT;
   if (experts * each < inter && columns != experts + 1) return SHRIKE_BAD_ARGUMENT;
@@ -1282,22 +1350,27 @@ SHRIKE_API int shrike_act_mul_blocks_at(const void* gate_up, const float* weight
     const dim3 grid(max(1, min(64, (groups + 255) / 256)), max(1, min(n, 65535)));
     if (vec)
       launch_dependent(act_mul_blocks_kernel<float, 4>, grid, 256, 0, stream, static_cast<const float*>(gate_up), weights,
-                       static_cast<float*>(out), n, inter, experts, each, columns, act, limit, weight_input);
+                       static_cast<float*>(out), n, inter, experts, each, columns, act, limit, weight_input, shared_limit);
     else
       launch_dependent(act_mul_blocks_kernel<float, 1>, grid, 256, 0, stream, static_cast<const float*>(gate_up), weights,
-                       static_cast<float*>(out), n, inter, experts, each, columns, act, limit, weight_input);
+                       static_cast<float*>(out), n, inter, experts, each, columns, act, limit, weight_input, shared_limit);
   } else if (dtype == SHRIKE_BF16) {
     const bool vec = aligned && inter % wide_bf16 == 0 && each % wide_bf16 == 0;
     const int groups = vec ? inter / wide_bf16 : inter;
     const dim3 grid(max(1, min(64, (groups + 255) / 256)), max(1, min(n, 65535)));
     if (vec)
       launch_dependent(act_mul_blocks_kernel<__nv_bfloat16, 8>, grid, 256, 0, stream, static_cast<const __nv_bfloat16*>(gate_up),
-                       weights, static_cast<__nv_bfloat16*>(out), n, inter, experts, each, columns, act, limit, weight_input);
+                       weights, static_cast<__nv_bfloat16*>(out), n, inter, experts, each, columns, act, limit, weight_input, shared_limit);
     else
       launch_dependent(act_mul_blocks_kernel<__nv_bfloat16, 1>, grid, 256, 0, stream, static_cast<const __nv_bfloat16*>(gate_up),
-                       weights, static_cast<__nv_bfloat16*>(out), n, inter, experts, each, columns, act, limit, weight_input);
+                       weights, static_cast<__nv_bfloat16*>(out), n, inter, experts, each, columns, act, limit, weight_input, shared_limit);
   } else return SHRIKE_BAD_ARGUMENT;
   return shrike_launch_status();
+}
+
+SHRIKE_API int shrike_act_mul_blocks_at(const void* gate_up, const float* weights, void* out, int dtype, int n, int inter, int experts,
+                                        int each, int columns, int act, float limit, int weight_input, cudaStream_t stream) {
+  return shrike_act_mul_blocks_limits(gate_up, weights, out, dtype, n, inter, experts, each, columns, act, limit, weight_input, limit, stream);
 }
 
 SHRIKE_API int shrike_act_mul_blocks(const void* gate_up, const float* weights, void* out, int dtype, int n, int inter, int experts,

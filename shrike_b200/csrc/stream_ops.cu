@@ -16,7 +16,8 @@
 //                    f = lower + (1 - lower) sigmoid(. + bias), token by token with the state slice in registers; for long
 //                    portions in three launches over runs of tokens (every run from a zero state and its decay, the
 //                    runs' states carried in order, every run again from the state it starts from).
-//   head_rms         every head of a row over its root mean square, times one weight of the head's size.
+//   head_rms         every head of a row over its root mean square, times one weight of the head's size, times the
+//                    sigmoid of columns of a fused projection (optional).
 //
 // Sums, norms, gates, decays and states are float32; a result is rounded once, when it is stored in the activation type.
 #include <cooperative_groups.h>
@@ -497,19 +498,47 @@ __global__ void __launch_bounds__(256) gated_scan_carry_kernel(const ScanArgs a)
 }
 
 // ------------------------------------------------------------------------------------------------ head_rms
-template <typename TO>
+// A warp a head; VEC = 4: 16-byte accesses.  `gates` (may be null): the result is multiplied by the sigmoid of column
+// gate_at + (head, element) of a fused projection ([partials][N][gate_width]).
+template <typename TO, int VEC>
 __global__ void __launch_bounds__(128) head_rms_kernel(const float* __restrict__ x, const float* __restrict__ weight,
-                                                       TO* __restrict__ out, int n, int heads, int size, float eps) {
+                                                       TO* __restrict__ out, int n, int heads, int size, float eps,
+                                                       const float* __restrict__ gates, int partials, long long stride,
+                                                       int gate_width, int gate_at) {
   let_dependents_start();
   wait_for_previous();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long unit = static_cast<long long>(blockIdx.x) * 4 + warp;
   if (unit >= static_cast<long long>(n) * heads) return;
   const float* row = x + unit * size;
+  const int groups = size / VEC;
+  const float* gate_row = gates != nullptr ? gates + (unit / heads) * gate_width + gate_at + (unit % heads) * size : nullptr;
   float squares = 0.f;
-  for (int d = lane; d < size; d += 32) squares = __fmaf_rn(row[d], row[d], squares);
+  for (int g = lane; g < groups; g += 32) {
+    float v[VEC];
+    if constexpr (VEC == 4) load4<float>(row + g * 4, v);
+    else v[0] = row[g];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) squares = __fmaf_rn(v[e], v[e], squares);
+  }
   const float r = rsqrtf(warp_sum(squares) / static_cast<float>(size) + eps);
-  for (int d = lane; d < size; d += 32) out[unit * size + d] = from_float<TO>(row[d] * r * (weight != nullptr ? weight[d] : 1.f));
+  for (int g = lane; g < groups; g += 32) {
+    float v[VEC], z[VEC] = {};
+    if constexpr (VEC == 4) {
+      load4<float>(row + g * 4, v);
+      if (gate_row != nullptr) sum_partials4(gate_row + g * 4, stride, partials, z);
+    } else {
+      v[0] = row[g];
+      if (gate_row != nullptr) z[0] = sum_partials(gate_row + g, stride, partials);
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+      v[e] = v[e] * r * (weight != nullptr ? weight[g * VEC + e] : 1.f);
+      if (gate_row != nullptr) v[e] = v[e] / (1.0f + expf(-z[e]));
+    }
+    if constexpr (VEC == 4) store4<TO>(out + unit * size + g * 4, v);
+    else out[unit * size + g] = from_float<TO>(v[0]);
+  }
 }
 
 }  // namespace streams
@@ -657,18 +686,37 @@ SHRIKE_API int shrike_gated_scan(const float* fused, int partials, long long str
   return shrike_launch_status();
 }
 
+// Only the state's update of the convolution: a thread a sequence and channel (for a caller whose own kernel convolves).
+SHRIKE_API int shrike_short_conv_keep(const float* fused, int partials, long long stride, int total, float* state,
+                                      const int* q_start, const int* state_slot, int channels, int taps_count, int num_seqs,
+                                      int num_slots, cudaStream_t stream) {
+  if (num_seqs <= 0 || taps_count <= 1) return SHRIKE_OK;
+  if (channels < 1 || channels > total || taps_count > MAX_TAPS || partials < 1 || num_seqs > 65535) return SHRIKE_BAD_ARGUMENT;
+  ConvArgs a = {fused, stride, partials, total, nullptr, nullptr, state, q_start, state_slot, nullptr, nullptr,
+                0, channels, taps_count, num_seqs, num_slots};
+  const dim3 keep(static_cast<unsigned>((channels + 255) / 256), static_cast<unsigned>(num_seqs));
+  launch_dependent(short_conv_keep_kernel, keep, 256, 0, stream, a);
+  return shrike_launch_status();
+}
+
+// `gates` (null: none): [partials][N][gate_width] float32, `stride` elements between partials; see the kernel.
 SHRIKE_API int shrike_head_rms(const float* x, const float* weight, void* out, int dtype, int n, int heads, int size,
-                               float eps, cudaStream_t stream) {
+                               float eps, const float* gates, int partials, long long stride, int gate_width, int gate_at,
+                               cudaStream_t stream) {
   if (n <= 0) return SHRIKE_OK;
-  if (heads < 1 || size < 1) return SHRIKE_BAD_ARGUMENT;
+  if (heads < 1 || size < 1 || partials < 1) return SHRIKE_BAD_ARGUMENT;
+  if (gates != nullptr && (gate_at < 0 || gate_at + heads * size > gate_width)) return SHRIKE_BAD_ARGUMENT;
   const long long units = static_cast<long long>(n) * heads;
   const long long blocks = (units + 3) / 4;
   if (blocks > 0x7fffffffLL) return SHRIKE_BAD_ARGUMENT;
-  if (dtype == SHRIKE_F32)
-    launch_dependent(head_rms_kernel<float>, static_cast<unsigned>(blocks), 128, 0, stream, x, weight, static_cast<float*>(out), n, heads, size, eps);
-  else if (dtype == SHRIKE_BF16)
-    launch_dependent(head_rms_kernel<__nv_bfloat16>, static_cast<unsigned>(blocks), 128, 0, stream, x, weight,
-                     static_cast<__nv_bfloat16*>(out), n, heads, size, eps);
+  const bool vec = size % 4 == 0 && (reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out)) % 16 == 0 &&
+                   (gates == nullptr || (reinterpret_cast<uintptr_t>(gates) % 16 == 0 && gate_at % 4 == 0 && gate_width % 4 == 0 && stride % 4 == 0));
+#define SHRIKE_HEAD_RMS(T, V)                                                                                               \
+  launch_dependent(head_rms_kernel<T, V>, static_cast<unsigned>(blocks), 128, 0, stream, x, weight, static_cast<T*>(out), n, heads, \
+                   size, eps, gates, partials, stride, gate_width, gate_at)
+  if (dtype == SHRIKE_F32) { if (vec) SHRIKE_HEAD_RMS(float, 4); else SHRIKE_HEAD_RMS(float, 1); }
+  else if (dtype == SHRIKE_BF16) { if (vec) SHRIKE_HEAD_RMS(__nv_bfloat16, 4); else SHRIKE_HEAD_RMS(__nv_bfloat16, 1); }
   else return SHRIKE_BAD_ARGUMENT;
+#undef SHRIKE_HEAD_RMS
   return shrike_launch_status();
 }

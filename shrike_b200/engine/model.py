@@ -86,6 +86,13 @@ class DecoderModel:
             self.pass_entry = cls(spec, {local: tensors[names.pass_entry_name(local)] for local in cls.parameters(spec)},
                                   ops, runtime)
             parts.append(self.pass_entry)
+        self.side_table = None
+        if config.side_table is not None:
+            spec = config.side_table
+            cls = part_class("side_table", spec.kind)
+            self.side_table = cls(spec, {local: tensors[names.side_table_name(local)] for local in cls.parameters(spec)},
+                                  ops, runtime)
+            parts.append(self.side_table)
         self.residual = None
         if config.residual is not None:
             spec = config.residual
@@ -154,6 +161,8 @@ class DecoderModel:
             self.pass_entry.before_embedding(ctx)   # it may ask the embedding for a second copy of its output
         resid = self.embedding.forward(ctx)
         delta = None
+        if self.side_table is not None:
+            self.side_table.begin(ctx)
         if self.pass_entry is not None:
             self.pass_entry.begin(resid, ctx)   # it keeps what it needs of the embedding's output
         if self.residual is not None:

@@ -6,7 +6,7 @@ under the system's temporary folder).  Its file name carries a hash of the sourc
 headers, flags and macro definitions, so an edited source is rebuilt and an
 unchanged one is loaded as is.  Only what is asked for is compiled: a float32
 replay never builds the tensor-core kernels, and attention is built for the head
-size of the model at hand.  While nvcc runs, a line is printed every few seconds.
+size of the model at hand.  The sources of a library are compiled side by side.  While nvcc runs, a line is printed every few seconds.
 """
 
 from __future__ import annotations
@@ -21,6 +21,7 @@ import sys
 import tempfile
 import threading
 import time
+from concurrent.futures import ThreadPoolExecutor
 from pathlib import Path
 
 CSRC = Path(__file__).resolve().parents[1] / "csrc"
@@ -75,6 +76,37 @@ def library_path(name: str, sources, defines=None, extra_flags=()) -> Path:
     return build_dir() / f"{name}-{_digest(sources, defines or {}, list(extra_flags))}.so"
 
 
+def _run(command, name) -> None:
+    process = subprocess.run(command, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)
+    if process.returncode != 0:
+        raise BuildError(f"nvcc failed for {name}:\n{' '.join(command)}\n{process.stdout}")
+
+
+def _compile_objects(nvcc, name, sources, defines, extra_flags, flags, folder) -> list[Path]:
+    """An object file per source, compiled side by side; one whose source, headers and flags have not changed is kept."""
+    objects, pending = [], []
+    for source in sources:
+        stem = f"{name}-{Path(source).stem}"
+        target = folder / f"{stem}-{_digest([source], defines, list(extra_flags))}.o"
+        objects.append(target)
+        if not target.is_file():
+            pending.append((source, stem, target))
+
+    def compile_one(job):
+        source, stem, target = job
+        scratch = target.with_suffix(f".tmp{os.getpid()}.o")
+        _run([nvcc, *BASE_FLAGS, *ARCH_FLAGS, *flags, "-c", "-o", str(scratch), str(CSRC / source)], name)
+        os.replace(scratch, target)
+        for stale in folder.glob(f"{stem}-*.o"):
+            if stale != target and ".tmp" not in stale.name:
+                stale.unlink(missing_ok=True)
+
+    if pending:
+        with ThreadPoolExecutor(max_workers=max(1, min(len(pending), os.cpu_count() or 1))) as pool:
+            list(pool.map(compile_one, pending))
+    return objects
+
+
 def compile_library(name: str, sources, defines=None, extra_flags=(), verbose=True) -> Path:
     """Builds (if needed) and returns the path of the library."""
     defines = defines or {}
@@ -89,13 +121,9 @@ def compile_library(name: str, sources, defines=None, extra_flags=(), verbose=Tr
                 return target
             nvcc = find_nvcc()
             scratch = target.with_suffix(f".tmp{os.getpid()}.so")
-            command = [nvcc, *BASE_FLAGS, *ARCH_FLAGS, *extra_flags]
-            command += [f"-D{key}={value}" for key, value in sorted(defines.items())]
-            command += ["-o", str(scratch)] + [str(CSRC / s) for s in sources]
             started = time.time()
             if verbose:
                 print(f"[shrike_b200] compiling {name} for sm_100a ...", file=sys.stderr, flush=True)
-            process = subprocess.Popen(command, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)
             done = threading.Event()
 
             def heartbeat():
@@ -103,14 +131,17 @@ def compile_library(name: str, sources, defines=None, extra_flags=(), verbose=Tr
                     print(f"[shrike_b200] still compiling {name} ({time.time() - started:.0f}s)",
                           file=sys.stderr, flush=True)
 
-            beat = threading.Thread(target=heartbeat, daemon=True)
             if verbose:
-                beat.start()
-            output, _ = process.communicate()
-            done.set()
-            if process.returncode != 0:
+                threading.Thread(target=heartbeat, daemon=True).start()
+            flags = [*extra_flags, *(f"-D{key}={value}" for key, value in sorted(defines.items()))]
+            try:
+                objects = _compile_objects(nvcc, name, sources, defines, extra_flags, flags, target.parent)
+                _run([nvcc, *BASE_FLAGS, *ARCH_FLAGS, *flags, "-o", str(scratch), *map(str, objects)], name)
+            except BuildError:
                 scratch.unlink(missing_ok=True)
-                raise BuildError(f"nvcc failed for {name}:\n{' '.join(command)}\n{output}")
+                raise
+            finally:
+                done.set()
             os.replace(scratch, target)
             for stale in target.parent.glob(f"{name}-*.so"):   # older builds of the same library
                 if stale != target and ".tmp" not in stale.name:
@@ -132,7 +163,7 @@ def load_library(name: str, sources, defines=None, extra_flags=()) -> ctypes.CDL
 
 
 # The libraries of this package.
-CORE_SOURCES = ["elementwise.cu", "branch_ops.cu", "parallel_ops.cu", "decay_ops.cu", "stream_ops.cu", "gemm_fp32.cu", "sampling.cu"]
+CORE_SOURCES = ["elementwise.cu", "branch_ops.cu", "parallel_ops.cu", "decay_ops.cu", "stream_ops.cu", "delta_ops.cu", "gemm_fp32.cu", "sampling.cu"]
 ATTENTION_SOURCES = ["attention_generic.cu", "attention_bf16.cu", "attention_tcgen05.cu"]
 
 

@@ -60,7 +60,11 @@ _LIMITS = {
     "stream_norm": "1 to 8 streams, at most four pending sums, a row that fits an SM's shared memory",
     "short_conv": "1 to 32 taps, at most 65535 sequences, the convolved channels the projection's first columns",
     "gated_scan": "heads of at most 1024 rows, at most 65535 sequences, heads and runs of tokens, the row at least as wide as q, f and v, the state's heads at least dim * vdim floats",
-    "route_top": "at most 1024 experts, 1 <= top <= experts, the weights [N, experts] or [N, experts + 1]",
+    "route_top": "at most 1024 experts, 1 <= top <= experts, the weights [N, experts] or [N, experts + 1], groups of equal size that hold enough experts",
+    "norm_join": "the row width must be at most 32768 (8192 when it is no multiple of 4)",
+    "side_gate": "the gate at least as wide as the token's part, which lies inside the table's rows",
+    "delta_prep": "1 to 32 taps, heads a multiple of kv heads, beta and the low-rank columns behind q, k and v inside the row",
+    "delta_scan": "heads of at most 1024 rows, at most 65535 sequences and heads, the state's heads on 16-byte borders and at least dim * vdim floats",
     "act_mul_blocks": "experts * each columns at most, the rest the shared expert's, which needs the weights' last column",
     "paged_attention_bf16": "at most 65535 sequences and heads, heads a multiple of kv heads, at most 32 splits",
 }
@@ -113,6 +117,8 @@ class CudaOps:
             self.gemm_tc.shrike_gemm_tc_gated_act.restype = _I
             self.gemm_tc.shrike_gemm_tc_gated_act_limit.argtypes = [_P, _P, _P, _I, _I, _I, _I, _F, _P, _P]
             self.gemm_tc.shrike_gemm_tc_gated_act_limit.restype = _I
+            self.gemm_tc.shrike_gemm_tc_act.argtypes = [_P, _P, _P, _I, _I, _I, _I, _P, _P]
+            self.gemm_tc.shrike_gemm_tc_act.restype = _I
             self.gemm_tc.shrike_gemm_tc_splits.argtypes = [_I, _I, _I]
             self.gemm_tc.shrike_gemm_tc_splits.restype = _I
         self._scratch = None     # partial results of split single-token attention
@@ -172,13 +178,23 @@ class CudaOps:
         lib.shrike_gated_scan.argtypes = [_P, _I, _LL, _I, _P, _P, _P, _P, _P, _P] + [_I] * 7 + [_P, _P, _P, _I, _I, _P]
         lib.shrike_gated_scan_runs.argtypes = [_I, _I, _I]
         lib.shrike_gated_scan_runs.restype = _LL
-        lib.shrike_head_rms.argtypes = [_P, _P, _P, _I, _I, _I, _I, _F, _P]
+        lib.shrike_head_rms.argtypes = [_P, _P, _P, _I, _I, _I, _I, _F, _P, _I, _LL, _I, _I, _P]
         lib.shrike_head_prep_norms.argtypes = [_P, _I, _LL, _I, _P, _P, _P, _I, _P, _P, _F, _P, _P, _P, _P, _P] + [_I] * 10 + [_P]
         lib.shrike_route_top_scores.argtypes = [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P]
         lib.shrike_act_mul_blocks_at.argtypes = [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P]
+        lib.shrike_route_top_groups.argtypes = [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P, _I, _I, _P]
+        lib.shrike_act_mul_blocks_limits.argtypes = [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _F, _P]
+        lib.shrike_norm_join.argtypes = [_P, _P, _I, _LL, _P, _P, _F, _P, _P, _F, _P, _I, _I, _I, _P]
+        lib.shrike_plain_act.argtypes = [_P, _I, _LL, _I, _P]
+        lib.shrike_side_gate.argtypes = [_P, _I, _LL, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _P, _I, _P]
+        lib.shrike_short_conv_keep.argtypes = [_P, _I, _LL, _I, _P, _P, _P, _I, _I, _I, _I, _P]
+        lib.shrike_delta_prep.argtypes = [_P, _I, _LL, _I, _P, _P, _P, _P, _P, _P, _P, _P] + [_I] * 11 + [_F, _F, _I, _P]
+        lib.shrike_delta_scan.argtypes = [_P, _P, _P, _I, _LL, _I, _P, _P, _P, _P, _P, _P] + [_I] * 7 + [_P]
         for name in ("shrike_decay_scan", "shrike_norm_gate", "shrike_latent_rope_store", "shrike_concat_cast",
                      "shrike_stream_norm", "shrike_short_conv", "shrike_gated_scan", "shrike_head_rms",
-                     "shrike_head_prep_norms", "shrike_route_top_scores", "shrike_act_mul_blocks_at"):
+                     "shrike_head_prep_norms", "shrike_route_top_scores", "shrike_act_mul_blocks_at",
+                     "shrike_route_top_groups", "shrike_act_mul_blocks_limits", "shrike_norm_join", "shrike_plain_act",
+                     "shrike_side_gate", "shrike_short_conv_keep", "shrike_delta_prep", "shrike_delta_scan"):
             getattr(lib, name).restype = _I
         for name in ("shrike_embed_scaled", "shrike_act_mul_limit", "shrike_tanh_norm", "shrike_head_prep",
                      "shrike_matrix_memory_scan", "shrike_matrix_memory_out", "shrike_route_top", "shrike_act_mul_blocks"):
@@ -350,6 +366,29 @@ class CudaOps:
         _check(self.core.shrike_norm_rows(
             _ptr(resid), _ptr(branch), code, partials, stride, None, _ptr(weight), _ptr(bias), eps, int(layer_norm),
             _ptr(out), -1 if out is None else _DTYPE_CODE[out.dtype], n, width, self._stream()), "norm_add")
+
+    def norm_join(self, resid, branch, branch_weight, branch_eps, row_add, weight, eps, out, rows=None):
+        """resid += branch / rms(branch) * branch_weight (+ `row_add` [W], every row), then out = resid / rms(resid) *
+        weight, `branch` float32 [N, W] or a [P, N, W] stack of partial sums.  With `rows` (int32 [R]) only out[r] for
+        row rows[r] is written, the residual stays."""
+        _dense(resid, torch.float32, "residual")
+        _dense(branch, torch.float32, "branch output")
+        _dense(weight, torch.float32, "norm weight")
+        _dense(branch_weight, torch.float32, "norm weight")
+        n, width = resid.shape
+        if tuple(branch.shape[-2:]) != (n, width):
+            raise KernelError(f"branch output {tuple(branch.shape)} does not fit the residual {tuple(resid.shape)}")
+        count = n
+        if rows is not None:
+            _dense(rows, torch.int32, "rows")
+            count = rows.shape[0]
+        if tuple(out.shape) != (count, width) or not out.is_contiguous():
+            raise KernelError(f"norm output {tuple(out.shape)} does not fit {count} rows of {width}")
+        partials, stride = self._stack(branch)
+        self.launches += 1
+        _check(self.core.shrike_norm_join(_ptr(resid), _ptr(branch), partials, stride, _ptr(rows), _ptr(branch_weight), branch_eps,
+                                          _ptr(row_add), _ptr(weight), eps, _ptr(out), _DTYPE_CODE[out.dtype], count, width,
+                                          self._stream()), "norm_join")
 
     def gather_norm(self, resid, rows, weight, bias, eps, out, layer_norm=True):
         """out[r] = norm(resid[rows[r]]): the final norm on the wanted rows only."""
@@ -729,6 +768,46 @@ class CudaOps:
                "gemm_tcgen05")
         return True
 
+    PLAIN_ACTIVATIONS = {"relu2": 1}   # activations of an ungated feed-forward: the codes the kernels take
+
+    def linear_act(self, x, w, out, activation="relu2"):
+        """act(x w^T) into `out` [N, O] in the engine's type; for few tokens in bfloat16 the activation is applied inside
+        the product (same bits), otherwise by a kernel in place."""
+        act = self.PLAIN_ACTIVATIONS[activation]
+        n, k = x.shape
+        _dense(out, self.dtype, "activation")
+        if self.gemm_tc is not None and n <= self.tensor_core_gemm_max_tokens and k % 8 == 0:
+            _dense(x, torch.bfloat16, "linear input")
+            _dense(w, torch.bfloat16, "linear weight")
+            if w.shape[1] != k or tuple(out.shape) != (n, w.shape[0]):
+                raise KernelError(f"linear: shapes x{tuple(x.shape)} w{tuple(w.shape)} out{tuple(out.shape)}")
+            self.launches += 1
+            _check(self.gemm_tc.shrike_gemm_tc_act(_ptr(x), _ptr(w), _ptr(out), n, w.shape[0], k, act, _ptr(self.status),
+                                                   self._stream()), "gemm_tcgen05")
+            return
+        self.linear(x, w, out)
+        self.launches += 1
+        _check(self.core.shrike_plain_act(_ptr(out), self.code, out.numel(), act, self._stream()), "plain_act")
+
+    def side_gate(self, gate, table, ids, previous, first, dim, out):
+        """out[n, c] = gelu_tanh(gate[n, c]) * table[ids[n], first + c] for c < dim, zero behind (`gate` float32 [N, padded]
+        or a K-split stack, `out` [N, padded], `table` [vocab, at least first + dim] in the engine's type).  An id of -1 - r
+        is replaced on the device by `previous[r]`, as in `embed`."""
+        _dense(gate, torch.float32, "side gate")
+        _dense(table, self.dtype, "side table")
+        _dense(ids, torch.int32, "token ids")
+        _dense(out, self.dtype, "side input")
+        n, padded = out.shape
+        if gate.shape[-1] != padded or gate.shape[-2] != n or ids.numel() < n:
+            raise KernelError(f"side_gate: gate{tuple(gate.shape)} out{tuple(out.shape)}")
+        if previous is not None:
+            _dense(previous, torch.int32, "previous tokens")
+        partials, stride = self._stack(gate)
+        self.launches += 1
+        _check(self.core.shrike_side_gate(_ptr(gate), partials, stride, _ptr(table), self.code, table.shape[1], table.shape[0],
+                                          _ptr(ids), _ptr(previous), 0 if previous is None else previous.numel(), first, dim,
+                                          padded, _ptr(out), n, self._stream()), "side_gate")
+
     def tanh_norm(self, resid, terms=(), row_add=None, rows=None, norms=()):
         """resid += sum over `terms` of scale * pending (each `(tensor, scale)`, the tensor float32 [N, W] or
         a K-split stack [P, N, W]) + `row_add` (float32 [W], added to every row); then, for each of up to two
@@ -924,47 +1003,59 @@ class CudaOps:
                                             n, width, self._stream()), "concat_cast")
 
     def head_linear(self, x, w, out, heads):
-        """out[n, h, :] = w[h] x[n, h, :]: x [N, heads * P] in the engine's type, w [heads, V, P], out float32
-        [N, heads * V].  One batched library product over the heads, reading and writing in place through strides."""
+        """out[n, h, :] = w[h] x[n, h, :]: x [N, heads * P] in the engine's type, w [heads, V, P], out float32 or in the
+        engine's type [N, heads * V].  One batched library product over the heads, reading and writing in place through strides."""
         n = x.shape[0]
         _dense(x, self.dtype, "head inputs")
-        _dense(out, torch.float32, "head outputs")
+        _dense(out, out.dtype, "head outputs")
         if w.dim() != 3 or w.shape[0] != heads or x.shape[1] != heads * w.shape[2] or out.shape[1] != heads * w.shape[1]:
             raise KernelError(f"head_linear: x{tuple(x.shape)} w{tuple(w.shape)} out{tuple(out.shape)}")
         self.library_calls += 1
         a = x.view(n, heads, w.shape[2]).transpose(0, 1)          # [heads, N, P]
         target = out.view(n, heads, w.shape[1]).transpose(0, 1)   # [heads, N, V]
-        if self.dtype == torch.float32:
+        if out.dtype == self.dtype:
             torch.bmm(a, w.transpose(1, 2), out=target)
         else:
             torch.bmm(a, w.transpose(1, 2), out_dtype=torch.float32, out=target)
 
-    def route_top(self, x, router, shared_gate, weights, top, renorm_eps, scoring="softmax", renormalise=True):
+    def route_top(self, x, router, shared_gate, weights, top, renorm_eps, scoring="softmax", renormalise=True, correction=None,
+                  groups=None):
         """weights [N, E (+ 1)] float32: softmax(router x) over all E experts in 32-bit, the `top` largest
         divided by their sum (+ renorm_eps), 0 elsewhere; a last column, when there is one, holds
         sigmoid(shared_gate . x) (1 when `shared_gate` is None).  `scoring` "sigmoid": an expert's score is the
-        sigmoid of its own logit; `renormalise` False: the chosen keep their scores as they are."""
+        sigmoid of its own logit; `renormalise` False: the chosen keep their scores as they are.  `correction` (float32
+        [E]) is added to the scores for the choice alone; `groups` (count, keep): only experts of the `keep` best of `count`
+        equal groups of neighbours, by each group's largest choice score, can be chosen."""
+        if correction is not None:
+            _dense(correction, torch.float32, "choice correction")
+            if correction.numel() != router.shape[0]:
+                raise KernelError("one choice correction per expert")
+        count, keep = groups if groups is not None else (0, 0)
         _dense(x, self.dtype, "router input")
         _dense(router, torch.float32, "router weight")
         _dense(weights, torch.float32, "expert weights")
         self.launches += 1
-        _check(self.core.shrike_route_top_scores(_ptr(x), self.code, _ptr(router), _ptr(shared_gate), _ptr(weights), x.shape[0],
+        _check(self.core.shrike_route_top_groups(_ptr(x), self.code, _ptr(router), _ptr(shared_gate), _ptr(weights), x.shape[0],
                                                  x.shape[1], router.shape[0], top, weights.shape[1], renorm_eps,
-                                                 int(scoring == "sigmoid"), int(bool(renormalise)), self._stream()), "route_top")
+                                                 int(scoring == "sigmoid"), int(bool(renormalise)), _ptr(correction), count, keep,
+                                                 self._stream()), "route_top")
 
-    def act_mul_blocks(self, gate_up, weights, out, experts, each, activation="silu", limit=None, weight_on="output"):
+    def act_mul_blocks(self, gate_up, weights, out, experts, each, activation="silu", limit=None, weight_on="output",
+                       shared_limit=None):
         """out[n, c] = act(gate[n, c]) * up[n, c] * weights[n, e(c)] for gate_up [N, 2 I] (gate columns, then up
         columns): column c belongs to expert c // each while c < experts * each, else to the shared expert
         (the last column of `weights`).  `weight_on` "input": the weight w multiplies the expert's input, which
-        reaches gate and up alike, out = act(w gate) * (w up)."""
+        reaches gate and up alike, out = act(w gate) * (w up).  `shared_limit`: the clamp of the shared expert's columns,
+        where it differs from `limit`."""
         _dense(gate_up, self.dtype, "gate_up")
         _dense(out, self.dtype, "activation")
         _dense(weights, torch.float32, "expert weights")
         n, inter = out.shape
         self.launches += 1
-        _check(self.core.shrike_act_mul_blocks_at(_ptr(gate_up), _ptr(weights), _ptr(out), self.code, n, inter, experts, each,
-                                                  weights.shape[1], self.ACTIVATIONS[activation], self._limit(activation, limit),
-                                                  int(weight_on == "input"), self._stream()), "act_mul_blocks")
+        _check(self.core.shrike_act_mul_blocks_limits(
+            _ptr(gate_up), _ptr(weights), _ptr(out), self.code, n, inter, experts, each, weights.shape[1],
+            self.ACTIVATIONS[activation], self._limit(activation, limit), int(weight_on == "input"),
+            self._limit(activation, limit if shared_limit is None else shared_limit), self._stream()), "act_mul_blocks")
 
     # ---- several residual streams, a short convolution, a gated recurrence -----------------------------
     def stream_norm(self, streams, pending, join, in_weights, norm_weight, eps, out, rows=None, sum_out=None):
@@ -1052,13 +1143,72 @@ class CudaOps:
             _ptr(out), num_seqs, num_heads, dim, vdim, state.shape[-1], state.shape[0], run, _ptr(run_state), _ptr(run_decay),
             _ptr(run_first), runs, int(self.dtype == torch.bfloat16), self._stream()), "gated_scan")
 
-    def head_rms(self, x, weight, eps, out, heads):
-        """out[n, h, :] = x[n, h, :] / sqrt(mean(x[n, h, :]^2) + eps) * weight for x float32 [N, heads * size]."""
+    def head_rms(self, x, weight, eps, out, heads, gate_source=None, gate_at=0):
+        """out[n, h, :] = x[n, h, :] / sqrt(mean(x[n, h, :]^2) + eps) * weight for x float32 [N, heads * size]; with
+        `gate_source` (float32 [N, total] or a K-split stack) times the sigmoid of its columns from `gate_at` on."""
         _dense(x, torch.float32, "head outputs")
         n, width = x.shape
+        partials, stride, gate_width = 1, 0, 0
+        if gate_source is not None:
+            _dense(gate_source, torch.float32, "gate source")
+            partials, stride = self._stack(gate_source)
+            gate_width = gate_source.shape[-1]
         self.launches += 1
         _check(self.core.shrike_head_rms(_ptr(x), _ptr(weight), _ptr(out), _DTYPE_CODE[out.dtype], n, heads, width // heads, eps,
-                                         self._stream()), "head_rms")
+                                         _ptr(gate_source), partials, stride, gate_width, gate_at, self._stream()), "head_rms")
+
+    # ---- a delta rule with a decay per key channel -------------------------------------------------------
+    def delta_prep(self, fused, taps, conv_state, q_start, state_slot, seq_of_token, mixed, beta, low, num_seqs, num_heads,
+                   num_kv_heads, dim, vdim, beta_at, low_at, unit_eps, longest=0):
+        """A fused projection ([N, total] float32 or a K-split stack) whose first columns are q (G dim) | k (G dim) | v (H
+        vdim): a causal convolution over time per channel (`taps` [channels, T]; the T - 1 values before a portion's first
+        token from `conv_state` [slots, T - 1, channels], which is left holding the portion's last ones), a SiLU, q and k
+        per head over sqrt(sum of squares + unit_eps), q times dim^(-1/2), into `mixed` [N, channels]; the sigmoid of the H
+        columns from `beta_at` into `beta`; the columns from `low_at` cast into `low`.  `longest`: the most new tokens a
+        sequence of the batch brings (the batch's shape; 0: not known)."""
+        _dense(fused, torch.float32, "fused projection")
+        _dense(taps, torch.float32, "convolution taps")
+        _dense(conv_state, torch.float32, "convolution state")
+        _dense(mixed, torch.float32, "q, k and v")
+        _dense(beta, torch.float32, "beta")
+        _dense(low, self.dtype, "low-rank rows")
+        partials, stride = self._stack(fused)
+        n, total = fused.shape[-2], fused.shape[-1]
+        channels, count = taps.shape
+        if channels != 2 * num_kv_heads * dim + num_heads * vdim or tuple(mixed.shape) != (n, channels):
+            raise KernelError(f"delta_prep: taps {tuple(taps.shape)}, q, k and v {tuple(mixed.shape)}")
+        if count > 1 and tuple(conv_state.shape[1:]) != (count - 1, channels):
+            raise KernelError("delta_prep: conv_state [slots, T - 1, channels]")
+        self.launches += 1
+        _check(self.core.shrike_delta_prep(
+            _ptr(fused), partials, stride, total, _ptr(taps), _ptr(conv_state), _ptr(q_start), _ptr(state_slot),
+            _ptr(seq_of_token), _ptr(mixed), _ptr(beta), _ptr(low), self.code, n, num_heads, num_kv_heads, dim, vdim, count,
+            beta_at, low_at, low.shape[1], conv_state.shape[0], unit_eps, float(dim) ** -0.5, int(longest), self._stream()),
+            "delta_prep")
+        if count > 1 and longest != 1:   # only after every token has read the old state
+            self.launches += 1
+            _check(self.core.shrike_short_conv_keep(_ptr(fused), partials, stride, total, _ptr(conv_state), _ptr(q_start),
+                                                    _ptr(state_slot), channels, count, num_seqs, conv_state.shape[0],
+                                                    self._stream()), "short_conv")
+
+    def delta_scan(self, mixed, beta, gates, rate, bias, state, q_start, state_slot, out, num_seqs, num_heads, num_kv_heads,
+                   dim, vdim, q_lens=None):
+        """The delta rule over the batch's new tokens, per value head h with q/k head h // (H / G) of `mixed` (as
+        `delta_prep` leaves it): S <- diag(g) S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q, with g =
+        exp(-rate[h] softplus(z + bias)), z column h dim + d of `gates` ([N, at least H dim] float32 or a K-split stack).
+        `state` float32 [slots, H, at least dim * vdim, a multiple of four] is read and left updated for the slots
+        `state_slot` names (-1: zeros out, nothing kept); `out` float32 [N, H * vdim]."""
+        for name, tensor in (("q, k and v", mixed), ("beta", beta), ("gates", gates), ("rate", rate), ("bias", bias),
+                             ("state", state), ("scan output", out)):
+            _dense(tensor, torch.float32, name)
+        partials, stride = self._stack(gates)
+        if state.dim() != 3 or state.shape[1] != num_heads or state.shape[2] < dim * vdim or bias.numel() != num_heads * dim:
+            raise KernelError(f"state {tuple(state.shape)} does not fit {num_heads} heads of {dim} x {vdim}")
+        self.launches += 1
+        _check(self.core.shrike_delta_scan(
+            _ptr(mixed), _ptr(beta), _ptr(gates), partials, stride, gates.shape[-1], _ptr(rate), _ptr(bias), _ptr(state),
+            _ptr(q_start), _ptr(state_slot), _ptr(out), num_seqs, num_heads, num_kv_heads, dim, vdim, state.shape[2],
+            state.shape[0], self._stream()), "delta_scan")
 
     def sample(self, logits, temperature, top_p, seeds, out):
         _dense(logits, torch.float32, "logits")

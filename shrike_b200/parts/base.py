@@ -45,6 +45,10 @@ be checked and the cache sized before anything is put on the device):
   join (a block that lists one per sublayer, roles "mixer_join" and "feed_forward_join")
       read_norm(streams_f32[N,S*W], pending | None, norm) -> normed[N,W]
           the pending sublayer result joins the streams, then the next sublayer's input is formed and normed
+  side input (a layer lists one as a further role; reads the model's side table through ctx.carried["side_table"])
+      forward(x[N,W], ctx) -> delta[N,W]       x: the residual in the activation type
+  side table (`ModelConfig.side_table`)
+      begin(ctx)                               once a forward pass: leaves itself for the layers' side inputs
   residual (a model whose residual is several streams a token; `ModelConfig.residual`)
       begin(resid_f32[N,W], ctx) -> streams_f32[N,S*W]       right after the embedding
       finish(streams, pending, rows_i32[R], norm) -> normed[R,W]   the final norm's input on the wanted rows
@@ -70,11 +74,21 @@ class ParamSpec:
 
     init: "matrix" | "table" (N(0, 0.02)), "bias" (N(0, 0.02)), "norm" (1 + N(0, 0.1)),
     "around_zero" (N(0, 0.1)), "sink" (N(0, 1)), "mix" ([W, 2 W]: identity | 0, plus N(0, 0.02)),
-    "conv" (N(0, 0.4)), "unit_interval" (sigmoid of N(0, 1)), "stream_mix" ([S, S]: identity plus N(0, 0.15)).
+    "conv" (N(0, 0.4)), "unit_interval" (sigmoid of N(0, 1)), "stream_mix" ([S, S]: identity plus N(0, 0.15)),
+    "decay_rate" (N(0, 0.5)), "decay_bias" (N(-3, 1): softplus of it spans slow and quick decays), "choice" (N(0, 0.01)),
+    "side_table" (N(0, 1)).
+
+    `free`: axes whose extent the model's tensor gives (the rank of a low-rank product, which no configuration key
+    names); `shape` holds there what random weights use.
     """
 
     shape: tuple[int, ...]
     init: str
+    free: tuple[int, ...] = ()
+
+    def fits(self, shape) -> bool:
+        return len(shape) == len(self.shape) and all(
+            have == want or (axis in self.free and have >= 1) for axis, (have, want) in enumerate(zip(shape, self.shape)))
 
 
 @dataclass(frozen=True)
@@ -125,6 +139,18 @@ class PendingSum:
         return [(delta, scale)]
 
 
+class PendingNorm:
+    """A branch output (float32 [N, W] or a K-split stack) whose NORM is not yet added to the residual: `norm` is the
+    norm part (an RMS norm) that stands on the branch's output.  `row_add` (float32 [W] or None) is added to every row
+    besides.  The next norm of the residual takes it in the same kernel: resid += norm(branch) + row_add, then the
+    normed sum."""
+
+    __slots__ = ("branch", "norm", "row_add")
+
+    def __init__(self, branch, norm, row_add=None):
+        self.branch, self.norm, self.row_add = branch, norm, row_add
+
+
 MIXERS: dict[str, type] = {}
 FEED_FORWARDS: dict[str, type] = {}
 NORMS: dict[str, type] = {}
@@ -134,6 +160,8 @@ EMBEDDINGS: dict[str, type] = {}
 HEADS: dict[str, type] = {}
 PASS_ENTRIES: dict[str, type] = {}
 JOINS: dict[str, type] = {}       # how a sublayer's result joins the residual (a layer lists them as further roles)
+SIDES: dict[str, type] = {}         # further inputs a layer takes per token
+SIDE_TABLES: dict[str, type] = {}   # where those come from (`ModelConfig.side_table`)
 RESIDUALS: dict[str, type] = {}   # a residual that is not one row a token (`ModelConfig.residual`)
 
 _CATEGORIES = {
@@ -142,6 +170,8 @@ _CATEGORIES = {
     "pass_entry": PASS_ENTRIES,
     "join": JOINS,
     "residual": RESIDUALS,
+    "side": SIDES,
+    "side_table": SIDE_TABLES,
     "mixer": MIXERS,
     "feed_forward": FEED_FORWARDS,
     "norm": NORMS,
@@ -152,7 +182,7 @@ _CATEGORIES = {
 
 def register_part(category: str, kind: str, cls: type) -> type:
     """Adds a part class; `category` is one of mixer, feed_forward, norm, position, block,
-    embedding, head, pass_entry, join, residual."""
+    embedding, head, pass_entry, join, residual, side, side_table."""
     _CATEGORIES[category][kind] = cls
     return cls
 

@@ -12,13 +12,17 @@ gets the rounded residual a branch reads from the kernel that made the sum.
 (shrike/models/qwen.py:147-150); the feed-forward may be absent.  The residual `resid` is float32; a branch output
 is handed on as `delta` and added by the next norm kernel.
 
+`SandwichBlock`: a norm on both sides of every sublayer, x += out_norm(mixer(norm(x))), x += out_norm(ffn(norm(x))), and
+optionally a further input per token, x += side_norm(side(x)).  A sublayer's output travels on as a `PendingNorm`, and
+the kernel that adds its norm to the residual also norms the sum for the next sublayer.
+
 When the kernels offer a native issue of whole layers (`ops.layer_program()`) and the four parts
 are ones it serves, the layer's launches are issued by one native call instead of part by part:
 the same kernels with the same arguments in the same order, without the interpreter between them."""
 
 from __future__ import annotations
 
-from .base import PendingSum, register_part
+from .base import PendingNorm, PendingSum, register_part
 
 
 class PreNormBlock:
@@ -113,6 +117,32 @@ class ParallelBlock:
         return resid, PendingSum(PendingSum.of(mixed) + PendingSum.of(fed))
 
 
+class SandwichBlock:
+    capture_safe = True
+
+    def __init__(self, mixer, mixer_norm, mixer_out_norm, feed_forward=None, feed_forward_norm=None,
+                 feed_forward_out_norm=None, side=None, side_norm=None):
+        if len({part is None for part in (feed_forward, feed_forward_norm, feed_forward_out_norm)}) != 1:
+            raise ValueError("a feed-forward and its two norms come together")
+        if (side is None) != (side_norm is None):
+            raise ValueError("a side input and its norm come together")
+        self.mixer, self.mixer_norm, self.mixer_out_norm = mixer, mixer_norm, mixer_out_norm
+        self.feed_forward, self.feed_forward_norm, self.feed_forward_out_norm = feed_forward, feed_forward_norm, feed_forward_out_norm
+        self.side, self.side_norm = side, side_norm
+
+    def forward(self, resid, delta, ctx, run):
+        hidden = self.mixer_norm.add_norm(resid, delta)
+        pending = PendingNorm(self.mixer.forward(hidden, ctx, run), self.mixer_out_norm)
+        if self.feed_forward is not None:
+            hidden = self.feed_forward_norm.add_norm(resid, pending)
+            pending = PendingNorm(self.feed_forward.forward(hidden, ctx), self.feed_forward_out_norm)
+        if self.side is not None:   # it reads the residual itself: the pending norm joins it first
+            hidden = pending.norm.norm_add(resid, pending.branch)
+            pending = PendingNorm(self.side.forward(hidden, ctx), self.side_norm)
+        return resid, pending
+
+
 register_part("block", "pre_norm", PreNormBlock)
+register_part("block", "sandwich", SandwichBlock)
 register_part("block", "parallel", ParallelBlock)
 register_part("block", "branch_norm", BranchNormBlock)

@@ -13,7 +13,7 @@ from __future__ import annotations
 
 import torch
 
-from .base import ParamSpec, PendingSum, register_part
+from .base import ParamSpec, PendingNorm, PendingSum, register_part
 
 
 class TokenEmbedding:
@@ -75,6 +75,11 @@ class PassEntry:
     def forward(self, resid, delta, ctx, number: int):
         if not 0 <= number < self.spec.passes:
             raise ValueError(f"pass {number} of {self.spec.passes}")
+        if isinstance(delta, PendingNorm):
+            if not self.mix and (number == 0 or self._kept is None) and delta.row_add is None:
+                # step[t] alone: it joins the residual in the kernel that adds the pending norm
+                return resid, PendingNorm(delta.branch, delta.norm, self.step[number])
+            raise NotImplementedError("a pending norm meets a pass entry that adds more than its own vector")
         terms = PendingSum.of(delta)
         if self.mix:
             # x <- Win [x ; e] + step[t]: the pending sums are added, the residual and the kept embedding are laid

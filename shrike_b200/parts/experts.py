@@ -13,7 +13,9 @@ sum.  Nothing depends on which experts the tokens chose, so a step's launches ar
 every batch of a shape and can be replayed.  Options of the spec: `scoring` "sigmoid" (an expert's score
 is the sigmoid of its own logit), `renormalise` False (the chosen keep their scores), `weight_on` "input" (an expert
 runs on weight * x: gate and up are linear in x, so the activation kernel forms act(w gate) * (w up) from the same
-product).  The price is arithmetic: every expert's columns are
+product), `correction` (a learned number per expert is added to the scores where experts are chosen, not where they are
+weighted), `groups` (only the experts of the best groups of neighbours can be chosen), `limit` / `shared_limit` (the clamped
+activation's clamp).  The price is arithmetic: every expert's columns are
 computed for every token, experts / top times what the chosen ones alone would take; in decoding,
 where the experts' weights are read once whatever the routing, it costs nothing.
 """
@@ -31,6 +33,8 @@ class RoutedExperts:
     @staticmethod
     def parameters(spec) -> dict[str, ParamSpec]:
         params = {"router.weight": ParamSpec((spec.experts, spec.width), "matrix")}
+        if getattr(spec, "correction", False):
+            params["router.correction"] = ParamSpec((spec.experts,), "choice")
         sizes = [(f"experts.{e}", spec.intermediate) for e in range(spec.experts)]
         if spec.shared_intermediate is not None:
             sizes.append(("shared", spec.shared_intermediate))
@@ -48,6 +52,9 @@ class RoutedExperts:
         if spec.shared_intermediate is not None:
             names.append("shared")
         self.router = tensors.pop("router.weight").to(torch.float32).contiguous()   # the router works in 32-bit
+        self.correction = None
+        if getattr(spec, "correction", False):
+            self.correction = tensors.pop("router.correction").to(torch.float32).contiguous()
         self.shared_gate = None
         if spec.shared_intermediate is not None and spec.shared_gate:
             self.shared_gate = tensors.pop("shared_gate.weight").to(torch.float32).reshape(-1).contiguous()
@@ -64,12 +71,16 @@ class RoutedExperts:
         share = rt.buffer("expert_share", (n, self.columns), torch.float32)
         ops.route_top(x, self.router, self.shared_gate, share, spec.top, spec.renorm_eps,
                       **({"scoring": spec.scoring} if getattr(spec, "scoring", "softmax") != "softmax" else {}),
-                      **({"renormalise": False} if not getattr(spec, "renormalise", True) else {}))
+                      **({"renormalise": False} if not getattr(spec, "renormalise", True) else {}),
+                      **({"correction": self.correction} if self.correction is not None else {}),
+                      **({"groups": spec.groups} if getattr(spec, "groups", None) is not None else {}))
         gate_up = rt.buffer("experts_gate_up", (n, 2 * self.inter), rt.act_dtype)
         ops.linear(x, self.w_gate_up, gate_up)
         act = rt.buffer("experts_act", (n, self.inter), rt.act_dtype)
         ops.act_mul_blocks(gate_up, share, act, spec.experts, spec.intermediate, spec.activation,
-                           **({"weight_on": "input"} if getattr(spec, "weight_on", "output") == "input" else {}))
+                           **({"weight_on": "input"} if getattr(spec, "weight_on", "output") == "input" else {}),
+                           **({"limit": spec.limit} if getattr(spec, "limit", None) is not None else {}),
+                           **({"shared_limit": spec.shared_limit} if getattr(spec, "shared_limit", None) is not None else {}))
         delta = rt.buffer("ffn_delta", (n, spec.width), torch.float32)
         return ops.linear(act, self.w_down, delta, allow_partials=True)
 

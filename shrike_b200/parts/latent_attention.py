@@ -200,10 +200,13 @@ class RotaryLatentAttention:
             heads, 1, padded, spec.scale, spec.window, attended,
             max_q_len=ctx.max_q_len, max_ctx_len=ctx.max_ctx_len, min_q_len=ctx.min_q_len, q_lens=ctx.q_lens,
         )
-        raised = rt.buffer("latent_up", (n, self.out_width), torch.float32)
-        ops.head_linear(attended, self.w_up, raised, heads)
         out = rt.buffer("latent_gated", (n, self.out_width), rt.act_dtype)
-        ops.norm_gate(raised, fused if self.gated else None, self.gate_at, None, spec.eps, out)
+        if self.gated:
+            raised = rt.buffer("latent_up", (n, self.out_width), torch.float32)
+            ops.head_linear(attended, self.w_up, raised, heads)
+            ops.norm_gate(raised, fused, self.gate_at, None, spec.eps, out)
+        else:   # nothing is multiplied in: the heads' outputs leave the product in the engine's type
+            ops.head_linear(attended, self.w_up, out, heads)
         delta = rt.buffer("mixer_delta", (n, spec.width), torch.float32)
         return ops.linear(out, self.w_o, delta, allow_partials=True)
 

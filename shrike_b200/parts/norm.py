@@ -9,7 +9,8 @@ costs no pass of its own.
 Two ways of sitting in a layer.  Before a branch (`add_norm`): the pending branch output is added to
 the residual and the sum is normed.  On a branch's output (`norm_add`): the branch output is normed
 and THAT is added to the residual, x += norm(branch(x)); what the next branch reads is then the
-residual itself, which `norm_add` returns in the activation type.  `LayerNorm` is
+residual itself, which `norm_add` returns in the activation type.  On both sides: the branch's output waits as a
+`PendingNorm`, and the next `add_norm` adds its norm to the residual and norms the sum in the same kernel.  `LayerNorm` is
 (x - mean) / sqrt(var + eps) * w + b with the variance as the mean squared deviation, in 32-bit.
 """
 
@@ -17,7 +18,7 @@ from __future__ import annotations
 
 import torch
 
-from .base import ParamSpec, PendingSum, register_part
+from .base import ParamSpec, PendingNorm, PendingSum, register_part
 
 
 class RMSNorm:
@@ -38,11 +39,19 @@ class RMSNorm:
 
     def add_norm(self, resid, delta, out_name="normed"):
         out = self.runtime.buffer(out_name, (resid.shape[0], self.spec.width), self.runtime.act_dtype)
-        self.ops.add_rmsnorm(resid, delta, self.weight, self.spec.eps, out)
+        if isinstance(delta, PendingNorm):
+            self.ops.norm_join(resid, delta.branch, delta.norm.weight, delta.norm.spec.eps, delta.row_add, self.weight,
+                               self.spec.eps, out)
+        else:
+            self.ops.add_rmsnorm(resid, delta, self.weight, self.spec.eps, out)
         return out
 
     def gather_norm(self, resid, delta, rows, out_name="normed_rows"):
         out = self.runtime.buffer(out_name, (rows.shape[0], self.spec.width), self.runtime.act_dtype)
+        if isinstance(delta, PendingNorm):
+            self.ops.norm_join(resid, delta.branch, delta.norm.weight, delta.norm.spec.eps, delta.row_add, self.weight,
+                               self.spec.eps, out, rows=rows)
+            return out
         self.ops.gather_add_rmsnorm(resid, delta, rows, self.weight, self.spec.eps, out)
         return out
 

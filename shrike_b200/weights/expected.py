@@ -29,6 +29,10 @@ def expected_tensors(config: ModelConfig) -> dict[str, ParamSpec]:
         entry = config.pass_entry
         for local, param in part_class("pass_entry", entry.kind).parameters(entry).items():
             table[names.pass_entry_name(local)] = param
+    if config.side_table is not None:
+        side = config.side_table
+        for local, param in part_class("side_table", side.kind).parameters(side).items():
+            table[names.side_table_name(local)] = param
     norm = config.final_norm
     for local, param in part_class("norm", norm.kind).parameters(norm).items():
         table[names.final_norm_name(local)] = param

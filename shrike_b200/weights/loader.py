@@ -83,7 +83,7 @@ def load_weights(model_dir, config: ModelConfig, engine_dtype: torch.dtype, devi
     wrong = [
         (name, expected[name].shape, where[name].shape(name))
         for name in expected
-        if name in where and tuple(where[name].shape(name)) != tuple(expected[name].shape)
+        if name in where and not expected[name].fits(where[name].shape(name))
     ]
     if missing or unexpected or wrong or duplicates:
         raise WeightError(model_dir, missing, unexpected, wrong, duplicates)

@@ -37,10 +37,16 @@ def random_tensor(name: str, spec, seed: int, device="cpu", dtype=torch.float32)
         values = 1.0 + 0.1 * values
     elif spec.init == "around_zero":
         values = 0.1 * values
-    elif spec.init == "sink":
+    elif spec.init in ("sink", "side_table"):
         pass
     elif spec.init == "conv":            # taps of a short convolution: of the order of one, so that every tap counts
         values = 0.4 * values
+    elif spec.init == "decay_rate":      # the logarithm of a decay's rate
+        values = 0.5 * values
+    elif spec.init == "decay_bias":      # softplus of it: steps from about 0.01 to 1, slow and quick decays side by side
+        values = values - 3.0
+    elif spec.init == "choice":          # what a router's choice is corrected by, of the order of the scores' differences
+        values = 0.01 * values
     elif spec.init == "unit_interval":   # a bound inside (0, 1)
         values = torch.sigmoid(values)
     elif spec.init == "stream_mix":      # [S, S]: near the identity, so that the streams stay apart

@@ -128,18 +128,34 @@ class EmulatedOps:
             held[:, D * Dv: D * Dv + D] = z
             held[:, D * Dv + D] = m
 
-    def route_top(self, x, router, shared_gate, weights, top, renorm_eps, scoring="softmax", renormalise=True):
+    def route_top(self, x, router, shared_gate, weights, top, renorm_eps, scoring="softmax", renormalise=True,
+                  correction=None, groups=None):
         logits = x.float() @ router.T
         scores = torch.sigmoid(logits) if scoring == "sigmoid" else torch.softmax(logits, -1)
-        _, chosen = torch.topk(logits, top, -1)   # the logits order the experts as either score does
+        choice = logits if correction is None and groups is None else scores   # the logits order the experts as either score does
+        if correction is not None:
+            choice = choice + correction
+        if groups is not None:
+            count, keep = groups
+            best = choice.view(x.shape[0], count, -1).amax(-1)
+            shut = torch.ones_like(best, dtype=torch.bool).scatter_(1, best.topk(keep, -1).indices, False)
+            choice = choice.masked_fill(shut.repeat_interleave(router.shape[0] // count, 1), float("-inf"))
+        _, chosen = torch.topk(choice, top, -1)
         best = scores.gather(1, chosen)
         weights.zero_()
         weights[:, : router.shape[0]].scatter_(1, chosen, best / (best.sum(-1, keepdim=True) + renorm_eps) if renormalise else best)
         if weights.shape[1] > router.shape[0]:
             weights[:, -1] = 1.0 if shared_gate is None else torch.sigmoid(x.float() @ shared_gate)
 
-    def act_mul_blocks(self, gate_up, weights, out, experts, each, activation="silu", limit=None, weight_on="output"):
+    def act_mul_blocks(self, gate_up, weights, out, experts, each, activation="silu", limit=None, weight_on="output",
+                       shared_limit=None):
         inter = out.shape[1]
+        if shared_limit is not None and shared_limit != limit:
+            wide = torch.empty_like(out)
+            self.act_mul_blocks(gate_up, weights, wide, experts, each, activation, shared_limit, weight_on)
+            self.act_mul_blocks(gate_up, weights, out, experts, each, activation, limit, weight_on)
+            out[:, experts * each:] = wide[:, experts * each:]
+            return
         column = torch.arange(inter)
         block = torch.where(column < experts * each, column // each, torch.full_like(column, experts))
         plain = torch.empty(out.shape, dtype=torch.float32)
@@ -433,12 +449,82 @@ class EmulatedOps:
                 out[t] = torch.einsum("hdv,hd->hv", S, q).reshape(-1)
             state[slot][:, : D * Dv] = S.reshape(H, -1)
 
-    def head_rms(self, x, weight, eps, out, heads):
+    def head_rms(self, x, weight, eps, out, heads, gate_source=None, gate_at=0):
         shaped = x.float().view(x.shape[0], heads, -1)
         normed = shaped / torch.sqrt(shaped.pow(2).mean(-1, keepdim=True) + eps)
         if weight is not None:
             normed = normed * weight
-        out.copy_(normed.reshape(x.shape).to(out.dtype))
+        normed = normed.reshape(x.shape)
+        if gate_source is not None:
+            gates = gate_source.sum(0) if gate_source.dim() == 3 else gate_source
+            normed = normed * torch.sigmoid(gates[:, gate_at: gate_at + x.shape[1]])
+        out.copy_(normed.to(out.dtype))
+
+    def norm_join(self, resid, branch, branch_weight, branch_eps, row_add, weight, eps, out, rows=None):
+        x = resid if rows is None else resid[rows.long()]
+        y = branch.float().sum(0) if branch.dim() == 3 else branch.float()
+        y = y if rows is None else y[rows.long()]
+        x = x + self._norm(y, branch_weight, None, branch_eps, False)
+        if row_add is not None:
+            x = x + row_add
+        if rows is None:
+            resid.copy_(x)
+        out.copy_(self._norm(x, weight, None, eps, False).to(out.dtype))
+
+    def side_gate(self, gate, table, ids, previous, first, dim, out):
+        gate = gate.sum(0) if gate.dim() == 3 else gate
+        ids = ids.long()
+        if previous is not None and (ids < 0).any():
+            ids = torch.where(ids < 0, previous.long()[(-1 - ids).clamp(min=0, max=previous.numel() - 1)], ids)
+        g = gate[:, :dim].float()
+        act = 0.5 * g * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (g + 0.044715 * g ** 3)))
+        out.zero_()
+        out[:, :dim] = (act * table[ids, first: first + dim].float()).to(out.dtype)
+
+    def linear_act(self, x, w, out, activation="relu2"):
+        assert activation == "relu2"
+        z = torch.empty(out.shape, dtype=out.dtype)
+        self.linear(x, w, z)
+        out.copy_(torch.relu(z.float()).pow(2).to(out.dtype))
+
+    def delta_prep(self, fused, taps, conv_state, q_start, state_slot, seq_of_token, mixed, beta, low, num_seqs, num_heads,
+                   num_kv_heads, dim, vdim, beta_at, low_at, unit_eps, longest=0):
+        if fused.dim() == 3:
+            fused = fused.sum(0)
+        n, qk = fused.shape[0], num_kv_heads * dim
+        channels = 2 * qk + num_heads * vdim
+        conv = torch.empty_like(fused)
+        self.short_conv(fused, None, taps, conv_state, q_start, state_slot, seq_of_token, conv, num_seqs, channels)
+        conv = conv[:, :channels] * torch.sigmoid(conv[:, :channels])
+        unit = lambda t: t / torch.sqrt(t.pow(2).sum(-1, keepdim=True) + unit_eps)  # noqa: E731
+        mixed[:, :qk] = (unit(conv[:, :qk].view(n, num_kv_heads, dim)) * dim ** -0.5).view(n, qk)
+        mixed[:, qk: 2 * qk] = unit(conv[:, qk: 2 * qk].view(n, num_kv_heads, dim)).view(n, qk)
+        mixed[:, 2 * qk:] = conv[:, 2 * qk:]
+        beta.copy_(torch.sigmoid(fused[:, beta_at: beta_at + num_heads]))
+        low.copy_(fused[:, low_at: low_at + low.shape[1]].to(low.dtype))
+
+    def delta_scan(self, mixed, beta, gates, rate, bias, state, q_start, state_slot, out, num_seqs, num_heads, num_kv_heads,
+                   dim, vdim, q_lens=None):
+        if gates.dim() == 3:
+            gates = gates.sum(0)
+        n, qk, share = mixed.shape[0], num_kv_heads * dim, num_heads // num_kv_heads
+        step = torch.nn.functional.softplus(gates[:, : num_heads * dim] + bias, threshold=60.0).view(n, num_heads, dim)
+        g = torch.exp(-rate[None, :, None] * step)
+        q = mixed[:, :qk].view(n, num_kv_heads, dim).repeat_interleave(share, 1)
+        k = mixed[:, qk: 2 * qk].view(n, num_kv_heads, dim).repeat_interleave(share, 1)
+        v = mixed[:, 2 * qk:].view(n, num_heads, vdim)
+        out.zero_()
+        for s in range(num_seqs):
+            slot = int(state_slot[s])
+            if slot < 0:
+                continue
+            held = state[slot][:, : dim * vdim].reshape(num_heads, dim, vdim).clone()
+            for t in range(int(q_start[s]), int(q_start[s + 1])):
+                held = g[t, :, :, None] * held
+                u = beta[t, :, None] * (v[t] - torch.einsum("hdv,hd->hv", held, k[t]))
+                held = held + k[t, :, :, None] * u[:, None, :]
+                out[t] = torch.einsum("hdv,hd->hv", held, q[t]).reshape(-1)
+            state[slot][:, : dim * vdim] = held.reshape(num_heads, -1)
 
     def silu_mul(self, gate_up, out):
         self.act_mul(gate_up, out)
