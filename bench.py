@@ -477,7 +477,7 @@ def run_mixed(args) -> dict:
 
     torch.cuda.set_device(0)
     design = getattr(args, "arch", "qwen2")   # the same workload on another decoder at the same widths
-    sadodra = design in ("sadodra", "vupitar", "kavedra", "setotar")
+    sadodra = design in ("sadodra", "vupitar", "kavedra", "setotar", "nulazen")
     if sadodra:
         from shrike_b200.shapes import shape_config
 
@@ -729,6 +729,74 @@ def run_case(args) -> dict:
             torch.cuda.synchronize()
             times.append(start.elapsed_time(stop) * 1e3)
         work = {"bytes": tokens * h * (2 * count * 4 + 2 * 4 + 2)}
+    elif args.case in ("delta_scan", "delta_scan_single"):
+        # the delta rule with a decay per key channel at the 7B-width shape (28 heads of 128 x 128): one prompt of
+        # --prefill-tokens tokens, or --batch sequences one token each
+        single = args.case.endswith("_single")
+        seqs, q_len = (tokens, 1) if single else (1, args.prefill_tokens)
+        n = seqs * q_len
+        mixed = torch.randn(n, 3 * heads * d, device=dev)
+        mixed[:, : 2 * heads * d] = torch.nn.functional.normalize(mixed[:, : 2 * heads * d].view(n, 2 * heads, d), dim=-1).view(n, -1)
+        beta, gates = torch.rand(n, heads, device=dev), torch.randn(n, 2 * heads * d, device=dev) - 3.0
+        rate, bias = torch.ones(heads, device=dev), torch.zeros(heads * d, device=dev)
+        state = torch.zeros(seqs, heads, d * d, device=dev)
+        q_start = torch.arange(seqs + 1, dtype=torch.int32, device=dev) * q_len
+        slots = torch.arange(seqs, dtype=torch.int32, device=dev)
+        out = torch.empty(n, heads * d, device=dev)
+        for _ in range(6):
+            keep_busy()
+            start.record()
+            ops.delta_scan(mixed, beta, gates, rate, bias, state, q_start, slots, out, seqs, heads, heads, d, d, q_lens=[q_len] * seqs)
+            stop.record()
+            torch.cuda.synchronize()
+            times.append(start.elapsed_time(stop) * 1e3)
+        # a token and head: dim x vdim each of the decay (1 flop), S^T k, k u^T and S^T q (2 flops a multiply-add)
+        work = {"bytes": seqs * heads * d * d * 4 * 2 + n * heads * (5 * d + 1) * 4} if single else {"flops": 7.0 * n * heads * d * d}
+    elif args.case == "delta_prep":
+        # --batch tokens of one sequence, q, k and v of 28 heads of 128 behind four taps, beta and two low-rank rows of 128
+        channels = 3 * heads * d
+        total = channels + heads + 2 * 128 + 4
+        fused = torch.randn(tokens, total, device=dev)
+        taps = torch.randn(channels, 4, device=dev)
+        state = torch.zeros(1, 3, channels, device=dev)
+        q_start = torch.tensor([0, tokens], dtype=torch.int32, device=dev)
+        zeros = torch.zeros(tokens, dtype=torch.int32, device=dev)
+        mixed, beta = torch.empty(tokens, channels, device=dev), torch.empty(tokens, heads, device=dev)
+        low = torch.empty(tokens, 256, device=dev, dtype=torch.bfloat16)
+        for _ in range(6):
+            keep_busy()
+            start.record()
+            ops.delta_prep(fused, taps, state, q_start, zeros[:1], zeros, mixed, beta, low, 1, heads, heads, d, d, channels,
+                           channels + heads, 1e-6, longest=tokens)
+            stop.record()
+            torch.cuda.synchronize()
+            times.append(start.elapsed_time(stop) * 1e3)
+        work = {"bytes": tokens * (total * 4 + channels * 4 + heads * 4 + 256 * 2)}
+    elif args.case == "norm_join":
+        resid, branch = torch.randn(tokens, h, device=dev), torch.randn(tokens, h, device=dev)
+        weight = torch.ones(h, device=dev)
+        out = torch.empty(tokens, h, device=dev, dtype=torch.bfloat16)
+        for _ in range(6):
+            keep_busy()
+            start.record()
+            ops.norm_join(resid, branch, weight, 1e-6, None, weight, 1e-6, out)
+            stop.record()
+            torch.cuda.synchronize()
+            times.append(start.elapsed_time(stop) * 1e3)
+        work = {"bytes": tokens * h * (4 + 4 + 4 + 2)}
+    elif args.case == "head_rms":
+        # --batch rows of 28 heads of 128 with an output gate from a fused product
+        x, gates = torch.randn(tokens, heads * d, device=dev), torch.randn(tokens, 2 * heads * d, device=dev)
+        weight = torch.ones(d, device=dev)
+        out = torch.empty(tokens, heads * d, device=dev, dtype=torch.bfloat16)
+        for _ in range(6):
+            keep_busy()
+            start.record()
+            ops.head_rms(x, weight, 1e-6, out, heads, gate_source=gates, gate_at=heads * d)
+            stop.record()
+            torch.cuda.synchronize()
+            times.append(start.elapsed_time(stop) * 1e3)
+        work = {"bytes": tokens * heads * d * (4 + 4 + 2)}
     elif args.case == "short_conv":
         # --batch tokens of one sequence, the fused q | k | v projection of the 7B-width shape, four taps
         channels = (heads + 2 * kv) * d
@@ -915,7 +983,7 @@ def run_timeline(args) -> dict:
 
 
 def run_design(args) -> dict:
-    """A design (--arch sadodra, the default here, vupitar, kavedra or setotar; the last also beside Vupitar) beside the Qwen2 decoder of the same widths, layer count and vocabulary (the
+    """A design (--arch sadodra, the default here, vupitar, kavedra, setotar or nulazen; the last two also beside the designs they are closest to) beside the Qwen2 decoder of the same widths, layer count and vocabulary (the
     closest model this engine serves), random weights: one 2,048-token prompt in one step, and decoding
     at --batch sequences of --context tokens, device-timed through the step function and the sampling
     kernel; for each, the kernels of one step by the time they take (CUPTI activity records).
@@ -1050,14 +1118,15 @@ def run_design(args) -> dict:
     sampler.start()
     t0 = time.perf_counter()
     results = [measure(f"{design.capitalize()} at Qwen2.5-{args.design.upper()} widths", ours)]
-    if design == "setotar":
-        # the design it is closest to among those served: attention beside a recurrent memory in one layer, routed experts
-        likeness = dict(shape_config(f"vupitar-{args.design}"))
+    # the designs it is closest to among those served: Setotar to Vupitar (attention beside a recurrent memory in one layer,
+    # routed experts); Nulazen to Kavedra (latent attention, a linear recurrence) and for its experts to Vupitar
+    for like in {"setotar": ("vupitar",), "nulazen": ("kavedra", "vupitar")}.get(design, ()):
+        likeness = dict(shape_config(f"{like}-{args.design}"))
         if args.layers:
             loop = likeness.get("loop")
             extra = (loop["stop"] - loop["start"]) * (loop["times"] - 1) if loop else 0
             likeness["layers"] = likeness["layers"][: max(args.layers - extra, loop["stop"] if loop else 1)]
-        results.append(measure(f"Vupitar at Qwen2.5-{args.design.upper()} widths", likeness))
+        results.append(measure(f"{like.capitalize()} at Qwen2.5-{args.design.upper()} widths", likeness))
     results.append(measure(f"Qwen2.5-{args.design.upper()} shape", theirs))
     sampler.stop()
     return {"case": "design", "design": design.capitalize(), "closest": "Qwen2ForCausalLM", "dtype": "bf16",
@@ -1088,7 +1157,7 @@ def main():
     parser.add_argument("--context", type=int, default=1024, help="tokens each sequence holds when decoding is timed")
     parser.add_argument("--workload", default="decode", choices=["decode", "mixed"],
                         help="decode: the headline line; mixed: 64 requests through the scheduler at 1.5B shape")
-    parser.add_argument("--arch", default="qwen2", choices=["qwen2", "sadodra", "vupitar", "kavedra", "setotar"],
+    parser.add_argument("--arch", default="qwen2", choices=["qwen2", "sadodra", "vupitar", "kavedra", "setotar", "nulazen"],
                         help="--workload mixed: the decoder the 64 requests run on (all at Qwen2.5-1.5B widths); "
                              "--case design: the design that is set beside the Qwen2 decoder (default there: sadodra)")
     parser.add_argument("--num-blocks", type=int, default=0, help="cache pages for --workload mixed (few pages force preemption)")
@@ -1103,7 +1172,8 @@ def main():
                              "one key/value head of 256 whose keys are its values; with _sink: a sink in every softmax), "
                              "branch_norm, tanh_norm, head_prep, matrix_memory (a prompt of --prefill-tokens), matrix_memory_single, "
                              "decay_scan (a prompt of --prefill-tokens), decay_scan_single, latent_rope_store, gated_scan, gated_scan_single, "
-                             "stream_norm, short_conv, attention_single_kept, attention_portions_kept; "
+                             "stream_norm, short_conv, delta_scan (a prompt of --prefill-tokens), delta_scan_single, delta_prep, norm_join, head_rms, "
+                             "attention_single_kept, attention_portions_kept; "
                              "--batch gives tokens / sequences / rows.  timeline: per-kernel "
                              "times inside one captured decode step (--layers, default 6).  design: the Sadodra decoder "
                              "beside the Qwen2 decoder of equal widths (--design), prefill and decode")

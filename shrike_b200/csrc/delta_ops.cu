@@ -5,7 +5,9 @@
 //                gates in the engine's type
 //   delta_scan   per head S <- diag(g) S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q over the batch's new tokens,
 //                with g = exp(-rate softplus(z + bias)) from a second product's columns z; the state is read from and
-//                left in the request's slot.  The walk goes token by token with the state in registers.
+//                left in the request's slot.  Single tokens and short portions walk token by token with the state in
+//                registers; longer ones go eight tokens at a time (`delta_local`, `delta_blocks`), the same sums in another
+//                order.
 //
 // Everything that enters the recurrence, and the state, is float32.  A product may come as a stack of K-split partial
 // sums, which are added on the fly.
@@ -13,13 +15,12 @@
 
 namespace delta {
 
-__device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
-
 // log(1 + e^z) without overflow; for small e^z it keeps the digits of e^z
 __device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 // ------------------------------------------------------------------------------------------------ delta_prep
-constexpr int TILE = 8;       // tokens a warp takes together: a projected value is read once for all taps
+constexpr int TILE = 8;       // tokens a warp takes together in a prompt: a projected value is read once for all taps
+constexpr int REST = 128;     // beta and low-rank columns a warp takes
 constexpr int MAX_TAPS = 32;
 
 struct PrepArgs {
@@ -39,24 +40,59 @@ struct PrepArgs {
   int keep;               // 1: a batch of single tokens, whose states this kernel updates itself
 };
 
-// T: the number of taps (1 to 4; 0: any number, values read again per tap).  VEC channels a thread.
-// A warp takes a head (of q, k or v) and TILE tokens; the tokens' values and the T - 1 before them are read first.
-template <typename TO, int T, int VEC>
+// SiLU in the activation type's accuracy: a bfloat16 engine takes the hardware exponential and reciprocal
+template <typename TO> __device__ __forceinline__ float silu_for(float z);
+template <> __device__ __forceinline__ float silu_for<float>(float z) { return z / (1.0f + expf(-z)); }
+template <> __device__ __forceinline__ float silu_for<__nv_bfloat16>(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
+
+template <int VEC>
+__device__ __forceinline__ void load_projected(const PrepArgs& a, bool stacked, int token, int c, float (&v)[VEC]) {
+  const float* at = a.fused + static_cast<size_t>(token) * a.total + c;
+  if constexpr (VEC == 4) {
+    if (stacked) sum_partials4(at, a.stride, a.partials, v);
+    else load4<float>(at, v);
+  } else {
+    v[0] = stacked ? sum_partials(at, a.stride, a.partials) : at[0];
+  }
+}
+
+// The projected value `back` tokens before a sequence's first new one: from its slot, or zero.
+template <int VEC>
+__device__ __forceinline__ void load_held(const PrepArgs& a, int slot, int taps, int back, int c, float (&v)[VEC]) {
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) v[e] = 0.f;
+  if (slot < 0 || slot >= a.num_slots) return;
+  const float* at = a.state + (static_cast<size_t>(slot) * (taps - 1) + (taps - 1 - back)) * a.channels + c;
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) v[e] = at[e];
+}
+
+// T: the number of taps (1 to 4; 0: any number, whose values are read again per tap).  VEC channels a thread, `Tile`
+// tokens a warp: 1 where tokens are few (the product may then be a stack of partial sums), else TILE, whose values are
+// read together and walked with the taps' window in registers.  A warp takes one head (of q, k or v).
+template <typename TO, int T, int VEC, int Tile>
 __global__ void __launch_bounds__(128) delta_prep_kernel(const PrepArgs a) {
   let_dependents_start();
-  wait_for_previous();
+  constexpr bool STACKED = Tile == 1;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int unit = blockIdx.y * 4 + warp;
-  const int first = blockIdx.x * TILE, here = min(TILE, a.n - first);
+  const int first = blockIdx.x * Tile, here = min(Tile, a.n - first);
   const int units = 2 * a.kv_heads + a.heads;
-  if (unit > units) return;
-  if (unit == units) {   // beta and the low-rank rows, column by column
+  const int seq_of = lane < here ? a.seq_of_token[first + lane] : -1;   // the step's metadata: no kernel writes it
+  wait_for_previous();
+  if (unit >= units) {   // beta and the low-rank rows
+    const int begin = (unit - units) * REST, end = min(a.heads + a.low_width, begin + REST);
     for (int t = 0; t < here; ++t) {
       const float* row = a.fused + static_cast<size_t>(first + t) * a.total;
-      for (int c = lane; c < a.heads; c += 32)
-        a.beta[static_cast<size_t>(first + t) * a.heads + c] = 1.0f / (1.0f + expf(-sum_partials(row + a.beta_at + c, a.stride, a.partials)));
-      TO* low = static_cast<TO*>(a.low) + static_cast<size_t>(first + t) * a.low_width;
-      for (int c = lane; c < a.low_width; c += 32) low[c] = from_float<TO>(sum_partials(row + a.low_at + c, a.stride, a.partials));
+#pragma unroll
+      for (int i = 0; i < REST / 32; ++i) {
+        const int c = begin + lane + 32 * i;
+        if (c >= end) continue;
+        const float* at = row + (c < a.heads ? a.beta_at + c : a.low_at + c - a.heads);
+        const float z = STACKED ? sum_partials(at, a.stride, a.partials) : at[0];
+        if (c < a.heads) a.beta[static_cast<size_t>(first + t) * a.heads + c] = 1.0f / (1.0f + expf(-z));
+        else static_cast<TO*>(a.low)[static_cast<size_t>(first + t) * a.low_width + c - a.heads] = from_float<TO>(z);
+      }
     }
     return;
   }
@@ -64,117 +100,114 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const PrepArgs a) {
   const int size = normed ? a.dim : a.vdim;
   const int channel0 = normed ? unit * a.dim : 2 * a.kv_heads * a.dim + (unit - 2 * a.kv_heads) * a.vdim;
   const int taps = T > 0 ? T : a.taps_count;
-  constexpr int HALO = T > 1 ? T - 1 : 0;
-  float squares[TILE];
-#pragma unroll
-  for (int t = 0; t < TILE; ++t) squares[t] = 0.f;
-  // where each token stands in its sequence, and its sequence's slot
-  int index[TILE], slot[TILE];
-#pragma unroll
-  for (int t = 0; t < TILE; ++t) {
-    index[t] = 0;
-    slot[t] = -1;
-    if (t < here) {
-      const int seq = a.seq_of_token[first + t];
-      index[t] = first + t - a.q_start[seq];
-      const int s = a.state_slot[seq];
-      slot[t] = s >= 0 && s < a.num_slots ? s : -1;
-    }
-  }
   const int groups = size / VEC;
-  for (int g = lane; g < groups; g += 32) {
-    const int c = channel0 + g * VEC;
-    const auto projected = [&](int token, float (&v)[VEC]) {
-      const float* at = a.fused + static_cast<size_t>(token) * a.total + c;
-      if constexpr (VEC == 4) sum_partials4(at, a.stride, a.partials, v);
-      else v[0] = sum_partials(at, a.stride, a.partials);
-    };
-    float x[TILE + HALO][VEC];
+  const int seq0 = __shfl_sync(0xffffffffu, seq_of, 0);
+  const int index0 = first - a.q_start[seq0];   // where the tile's first token stands in its sequence's portion
+  float squares[Tile], y[Tile][VEC];
+#pragma unroll
+  for (int t = 0; t < Tile; ++t) squares[t] = 0.f;
+  const bool single = groups <= 32;   // a head's channels are one round of the warp: they stay in registers
+  for (int g0 = 0; g0 < groups; g0 += 32) {
+    const int g = g0 + lane;
+    const bool active = g < groups;
+    const int c = channel0 + (active ? g : 0) * VEC;
+    float x[Tile][VEC];
+#pragma unroll
+    for (int t = 0; t < Tile; ++t) load_projected<VEC>(a, STACKED, first + min(t, here - 1), c, x[t]);
+    float w[T > 0 ? T : 1][VEC], window[T > 1 ? T - 1 : 1][VEC];   // window[i]: i + 1 tokens back
     if constexpr (T > 0) {
 #pragma unroll
-      for (int i = 0; i < TILE + HALO; ++i) {
-        const int token = first + i - HALO;
-        if (token >= 0 && i - HALO < here) projected(token, x[i]);
-        else {
+      for (int e = 0; e < VEC; ++e)
 #pragma unroll
-          for (int e = 0; e < VEC; ++e) x[i][e] = 0.f;
-        }
+        for (int j = 0; j < T; ++j) w[j][e] = a.taps[static_cast<size_t>(c + e) * T + j];
+      const int slot = a.state_slot[seq0];
+#pragma unroll
+      for (int i = 0; i < T - 1; ++i) {
+        if (i + 1 <= index0) load_projected<VEC>(a, STACKED, first - i - 1, c, window[i]);
+        else load_held<VEC>(a, slot, taps, i + 1 - index0, c, window[i]);
       }
     }
-    float w[T > 0 ? T : 1][VEC];
-    if constexpr (T > 0) {
+    int seq = seq0;
 #pragma unroll
-      for (int j = 0; j < T; ++j)
+    for (int t = 0; t < Tile; ++t) {
+      if (t < here) {
+        const int now = Tile > 1 ? __shfl_sync(0xffffffffu, seq_of, t) : seq0;
+        float acc[VEC];
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) w[j][e] = a.taps[static_cast<size_t>(c + e) * T + j];
-    }
+        for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
+        if constexpr (T > 0) {
+          if (Tile > 1 && now != seq) {   // another sequence begins here: its window comes from its slot
+            const int slot = a.state_slot[now];
 #pragma unroll
-    for (int t = 0; t < TILE; ++t) {
-      if (t >= here) continue;
-      float acc[VEC];
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
-      const auto held = [&](int back, int e) {   // the projected value `back` tokens before the sequence's first new one
-        return slot[t] >= 0 ? a.state[(static_cast<size_t>(slot[t]) * (taps - 1) + (taps - 1 - back)) * a.channels + c + e] : 0.f;
-      };
-      if constexpr (T > 0) {
-#pragma unroll
-        for (int j = 0; j < T; ++j) {
-          const int lag = T - 1 - j;
+            for (int i = 0; i < T - 1; ++i) load_held<VEC>(a, slot, taps, i + 1, c, window[i]);
+          }
 #pragma unroll
           for (int e = 0; e < VEC; ++e) {
-            const float u = lag <= index[t] ? x[t + j][e] : held(lag - index[t], e);   // x[t + HALO - lag] is x[t + j]
-            acc[e] = __fmaf_rn(w[j][e], u, acc[e]);
+#pragma unroll
+            for (int j = 0; j < T - 1; ++j) acc[e] = __fmaf_rn(w[j][e], window[T - 2 - j][e], acc[e]);
+            acc[e] = __fmaf_rn(w[T - 1][e], x[t][e], acc[e]);
+#pragma unroll
+            for (int i = T - 2; i > 0; --i) window[i][e] = window[i - 1][e];
+            if (T > 1) window[0][e] = x[t][e];
+          }
+        } else {
+          const int index = first + t - a.q_start[now], slot = a.state_slot[now];
+          for (int j = 0; j < taps; ++j) {
+            const int lag = taps - 1 - j;
+            float u[VEC];
+            if (lag <= index) load_projected<VEC>(a, STACKED, first + t - lag, c, u);
+            else load_held<VEC>(a, slot, taps, lag - index, c, u);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) acc[e] = __fmaf_rn(a.taps[static_cast<size_t>(c + e) * taps + j], u[e], acc[e]);
           }
         }
-      } else {
-        for (int j = 0; j < taps; ++j) {
-          const int lag = taps - 1 - j;
-          float u[VEC];
-          if (lag <= index[t]) projected(first + t - lag, u);
-          else {
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) u[e] = held(lag - index[t], e);
-          }
-#pragma unroll
-          for (int e = 0; e < VEC; ++e) acc[e] = __fmaf_rn(a.taps[static_cast<size_t>(c + e) * taps + j], u[e], acc[e]);
-        }
-      }
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) {
-        acc[e] = silu(acc[e]);
-        squares[t] = __fmaf_rn(acc[e], acc[e], squares[t]);
-      }
-      float* dst = a.mixed + static_cast<size_t>(first + t) * a.channels + c;
-      if constexpr (VEC == 4) store4<float>(dst, acc);
-      else dst[0] = acc[0];
-      if (a.keep && slot[t] >= 0 && taps > 1) {   // a sequence's one token: its state moves up by one
-        float* state = a.state + static_cast<size_t>(slot[t]) * (taps - 1) * a.channels + c;
-        float newest[VEC];
-        projected(first + t, newest);
+        seq = now;
 #pragma unroll
         for (int e = 0; e < VEC; ++e) {
-          for (int i = 0; i + 1 < taps - 1; ++i) state[static_cast<size_t>(i) * a.channels + e] = state[static_cast<size_t>(i + 1) * a.channels + e];
-          state[static_cast<size_t>(taps - 2) * a.channels + e] = newest[e];
+          y[t][e] = silu_for<TO>(acc[e]);
+          if (active) squares[t] = __fmaf_rn(y[t][e], y[t][e], squares[t]);
+        }
+        if (!(single && normed) && active) {
+          float* dst = a.mixed + static_cast<size_t>(first + t) * a.channels + c;
+          if constexpr (VEC == 4) store4<float>(dst, y[t]);
+          else dst[0] = y[t][0];
+        }
+        if (Tile == 1 && a.keep && active && taps > 1) {   // a sequence's one token: its state moves up by one
+          const int slot = a.state_slot[seq0];
+          if (slot >= 0 && slot < a.num_slots) {
+            float* state = a.state + static_cast<size_t>(slot) * (taps - 1) * a.channels + c;
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+              for (int i = 0; i + 1 < taps - 1; ++i)
+                state[static_cast<size_t>(i) * a.channels + e] = state[static_cast<size_t>(i + 1) * a.channels + e];
+              state[static_cast<size_t>(taps - 2) * a.channels + e] = x[t][e];
+            }
+          }
         }
       }
     }
   }
   if (!normed) return;
-  float gain[TILE];
+  float gain[Tile];
 #pragma unroll
-  for (int t = 0; t < TILE; ++t) {
+  for (int t = 0; t < Tile; ++t) {
     gain[t] = 1.0f / sqrtf(warp_sum(squares[t]) + a.unit_eps);
     if (unit < a.kv_heads) gain[t] *= a.q_scale;
   }
-  for (int g = lane; g < groups; g += 32) {   // what this very thread stored
+  for (int g = lane; g < groups; g += 32) {
 #pragma unroll
-    for (int t = 0; t < TILE; ++t) {
+    for (int t = 0; t < Tile; ++t) {
       if (t >= here) continue;
       float* dst = a.mixed + static_cast<size_t>(first + t) * a.channels + channel0 + g * VEC;
       float v[VEC];
-      if constexpr (VEC == 4) load4<float>(dst, v);
-      else v[0] = dst[0];
+      if (single) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[e] = y[t][e];
+      } else if constexpr (VEC == 4) {   // what this very thread stored
+        load4<float>(dst, v);
+      } else {
+        v[0] = dst[0];
+      }
 #pragma unroll
       for (int e = 0; e < VEC; ++e) v[e] *= gain[t];
       if constexpr (VEC == 4) store4<float>(dst, v);
@@ -200,6 +233,7 @@ struct ScanArgs {
   float* out;             // [N][H Dv]
   int heads, kv_heads, dim, vdim, channels, head_stride, num_slots;
   int lanes, cols;        // lanes of a warp that share a thread's columns; columns of a CTA
+  int skip_from;          // > 0: sequences that bring at least so many tokens are served elsewhere
 };
 
 // One CTA owns `cols` value columns of one head's state for one sequence and walks its tokens in order with the state in
@@ -226,6 +260,7 @@ __global__ void __launch_bounds__(128, 4) delta_walk_kernel(const ScanArgs a) {
   const int head = blockIdx.y, seq = blockIdx.z, col0 = blockIdx.x * cols;
   const int cols_here = min(cols, a.vdim - col0);
   const int first = a.q_start[seq], length = a.q_start[seq + 1] - first;
+  if (a.skip_from > 0 && length >= a.skip_from) return;
   const int slot = a.state_slot[seq];
   const size_t out_width = static_cast<size_t>(a.heads) * a.vdim;
   if (slot < 0 || slot >= a.num_slots) {   // a padding row: zeros out, nothing kept
@@ -359,17 +394,420 @@ __global__ void __launch_bounds__(128, 4) delta_walk_kernel(const ScanArgs a) {
   }
 }
 
+// ------------------------------------------------------------------------------------------------ blocks of tokens
+// Longer portions go BLOCK tokens at a time.  With tokens 1 .. B of a block, P_t = g_1 ... g_t and F_t = g_(t+1) ... g_B
+// (per key channel, products of decays, never a quotient), S the state before the block and
+//
+//   A[t][s]  = sum_d k_t k_s g_(s+1) ... g_t  (s < t)        a_t = S^T (P_t k_t)
+//   Aq[t][s] = the same with q_t              (s <= t)       c_t = S^T (P_t q_t)
+//
+// the rule's u_t = beta_t (v_t - a_t - sum_(s<t) A[t][s] u_s) is U = T (V - a) with T = (I + diag(beta) A)^-1 diag(beta),
+// lower triangular, and with d_s = v_s - a_s
+//
+//   o_t = c_t + sum_(s<=t) M[t][s] d_s,  M = Aq T          S <- P_B S + sum_s K_s d_s^T,  K_s = sum_(t>=s) T[t][s] F_t k_t
+//
+// `delta_local` forms P_t k_t, P_t q_t, K_s, P_B and M of every block and value head by itself; `delta_blocks` walks a
+// sequence's blocks with the state in registers: one reduction over the rows, one barrier and one update per BLOCK
+// tokens instead of per token, three multiply-adds a state element and token.
+constexpr int BLOCK = 8;
+
+struct BlockArgs {
+  ScanArgs s;
+  float* records;   // [blocks][head_count][record]: P_t k_t [B][Dp] | P_t q_t [B][Dp] | K_s [B][Dp] | P_B [Dp] | M [B][B]
+  int record, padded_dim;   // padded_dim: rows rounded up to what the lanes hold, zeros behind the head's own
+  int num_seqs, from;       // sequences that bring at least `from` tokens run here
+  int blocks;               // of the whole batch
+  int head0, head_count;    // the heads this launch serves
+};
+
+__host__ __device__ __forceinline__ int record_floats(int padded_dim) { return (3 * BLOCK + 1) * padded_dim + BLOCK * BLOCK; }
+
+// Blocks of sequence `seq`; a warp sums them over the sequences before one.
+__device__ __forceinline__ int blocks_of(const BlockArgs& a, int seq) {
+  const int length = a.s.q_start[seq + 1] - a.s.q_start[seq];
+  return length >= a.from ? (length + BLOCK - 1) / BLOCK : 0;
+}
+
+// The sum of `count` (a power of two times 1) values over 2 * `OFFSET` lanes, transposed: every step halves the values a
+// lane holds, so that lane g of them ends with the sums of values g * n .. g * n + n - 1, n = COUNT / lanes (at least one).
+template <int COUNT, int OFFSET>
+struct FoldLanes {
+  static __device__ __forceinline__ void run(float* v, int lane) {
+    if constexpr (OFFSET > 0) {
+      constexpr int HALF = COUNT / 2;
+      const bool upper = lane & OFFSET;
+#pragma unroll
+      for (int i = 0; i < HALF; ++i) {
+        const float send = upper ? v[i] : v[i + HALF], keep = upper ? v[i + HALF] : v[i];
+        v[i] = keep + __shfl_xor_sync(0xffffffffu, send, OFFSET);
+      }
+      FoldLanes<HALF, OFFSET / 2>::run(v, lane);
+    }
+  }
+};
+
+// grid (blocks, heads / 4): a warp a block and value head.
+__global__ void __launch_bounds__(128) delta_local_kernel(const BlockArgs a) {
+  __shared__ float shared_w[4][BLOCK * BLOCK], shared_t[4][BLOCK * BLOCK];
+  let_dependents_start();
+  wait_for_previous();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int block = blockIdx.x, local_head = blockIdx.y * 4 + warp;
+  if (local_head >= a.head_count) return;
+  const int head = a.head0 + local_head;
+  // the block's sequence: lanes count 32 sequences at a time
+  int before = 0, seq = -1, within = 0;
+  for (int base = 0; base < a.num_seqs && seq < 0; base += 32) {
+    const int mine = base + lane < a.num_seqs ? blocks_of(a, base + lane) : 0;
+    int total = mine;
+#pragma unroll
+    for (int offset = 1; offset < 32; offset <<= 1) {
+      const int other = __shfl_up_sync(0xffffffffu, total, offset);
+      if (lane >= offset) total += other;
+    }
+    const unsigned hit = __ballot_sync(0xffffffffu, block < before + total && mine > 0);
+    if (hit) {
+      const int owner = __ffs(hit) - 1;
+      seq = base + owner;
+      within = block - before - __shfl_sync(0xffffffffu, total - mine, owner);
+    }
+    before += __shfl_sync(0xffffffffu, total, 31);
+  }
+  if (seq < 0) return;
+  const ScanArgs& s = a.s;
+  const int first = s.q_start[seq] + within * BLOCK, here = min(BLOCK, s.q_start[seq + 1] - first);
+  const int D = s.dim, Dp = a.padded_dim;
+  const int group = head / (s.heads / s.kv_heads);
+  const int q_col = group * D, k_col = (s.kv_heads + group) * D;
+  const float rate = s.rate[head];
+  float* record = a.records + (static_cast<size_t>(block) * a.head_count + local_head) * a.record;
+  float* pk = record;
+  float* pq = record + BLOCK * Dp;
+  float* kk = record + 2 * BLOCK * Dp;
+  float* whole = record + 3 * BLOCK * Dp;
+  float pair[BLOCK * BLOCK];   // [t][s], s < t: A;  [s][t], s <= t: Aq
+#pragma unroll
+  for (int i = 0; i < BLOCK * BLOCK; ++i) pair[i] = 0.f;
+  for (int d = lane; d < Dp; d += 32) {
+    float g[BLOCK], k[BLOCK], q[BLOCK];
+    const bool row = d < D;
+    const float shift = row ? s.bias[head * D + d] : 0.f;
+#pragma unroll
+    for (int t = 0; t < BLOCK; ++t) {
+      const bool real = row && t < here;
+      const float* at = s.mixed + static_cast<size_t>(first + (t < here ? t : 0)) * s.channels;
+      k[t] = real ? at[k_col + d] : 0.f;
+      q[t] = real ? at[q_col + d] : 0.f;
+      g[t] = real ? s.gates[static_cast<size_t>(first + t) * s.gate_width + head * D + d] : 0.f;
+    }
+    if (s.partials > 1) {
+#pragma unroll
+      for (int t = 0; t < BLOCK; ++t)
+        if (row && t < here) g[t] = sum_partials(s.gates + static_cast<size_t>(first + t) * s.gate_width + head * D + d, s.stride, s.partials);
+    }
+#pragma unroll
+    for (int t = 0; t < BLOCK; ++t) g[t] = row && t < here ? expf(-rate * softplus(g[t] + shift)) : (row ? 1.f : 0.f);
+#pragma unroll
+    for (int from = 0; from < BLOCK; ++from) {
+      float w = k[from];
+      pair[from * BLOCK + from] = __fmaf_rn(w, q[from], pair[from * BLOCK + from]);
+#pragma unroll
+      for (int t = from + 1; t < BLOCK; ++t) {
+        w *= g[t];
+        pair[t * BLOCK + from] = __fmaf_rn(w, k[t], pair[t * BLOCK + from]);
+        pair[from * BLOCK + t] = __fmaf_rn(w, q[t], pair[from * BLOCK + t]);
+      }
+      kk[from * Dp + d] = w;   // F k: the key as it stands at the block's end
+    }
+    float p = 1.f;
+#pragma unroll
+    for (int t = 0; t < BLOCK; ++t) {
+      p *= g[t];
+      pk[t * Dp + d] = p * k[t];
+      pq[t * Dp + d] = p * q[t];
+    }
+    whole[d] = p;
+  }
+  FoldLanes<BLOCK * BLOCK, 16>::run(pair, lane);
+  float* w = shared_w[warp];
+  float* solved = shared_t[warp];
+  w[2 * lane] = pair[0];
+  w[2 * lane + 1] = pair[1];
+  __syncwarp();
+  if (lane < BLOCK) {   // column `lane` of T by forward substitution
+    float column[BLOCK];
+#pragma unroll
+    for (int t = 0; t < BLOCK; ++t) {
+      float v = t == lane ? 1.f : 0.f;
+#pragma unroll
+      for (int r = 0; r < t; ++r) v = __fmaf_rn(-w[t * BLOCK + r], column[r], v);   // column[r] is 0 above the diagonal
+      const float beta = t < here ? s.beta[static_cast<size_t>(first + t) * s.heads + head] : 0.f;
+      column[t] = beta * v;
+      solved[t * BLOCK + lane] = column[t];
+    }
+  }
+  __syncwarp();
+  float* m = whole + Dp;
+#pragma unroll
+  for (int i = lane; i < BLOCK * BLOCK; i += 32) {
+    const int t = i / BLOCK, c = i % BLOCK;
+    float v = 0.f;
+    for (int r = c; r <= t; ++r) v = __fmaf_rn(w[r * BLOCK + t], solved[r * BLOCK + c], v);
+    m[i] = v;
+  }
+  for (int d = lane; d < Dp; d += 32) {   // what this very thread stored, through T
+    float end[BLOCK];
+#pragma unroll
+    for (int t = 0; t < BLOCK; ++t) end[t] = kk[t * Dp + d];
+#pragma unroll
+    for (int c = 0; c < BLOCK; ++c) {
+      float v = 0.f;
+#pragma unroll
+      for (int t = c; t < BLOCK; ++t) v = __fmaf_rn(solved[t * BLOCK + c], end[t], v);
+      kk[c * Dp + d] = v;
+    }
+  }
+}
+
+// Two float32 multiply-adds in one instruction.
+__device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
+  unsigned long long d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ unsigned long long mul2(unsigned long long a, unsigned long long b) {
+  unsigned long long d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ unsigned long long pack2(float lo, float hi) {
+  unsigned long long d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+  return d;
+}
+__device__ __forceinline__ float2 unpack2(unsigned long long v) {
+  float2 f;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(v));
+  return f;
+}
+__device__ __forceinline__ void copy16(void* shared, const void* global) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(static_cast<unsigned>(__cvta_generic_to_shared(shared))), "l"(global) : "memory");
+}
+__device__ __forceinline__ void copy4(void* shared, const void* global) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(static_cast<unsigned>(__cvta_generic_to_shared(shared))), "l"(global) : "memory");
+}
+
+constexpr int STAGES = 3;
+
+// grid (slices, heads, sequences): a CTA owns `cols` value columns of one head's state for one sequence.  A thread holds
+// rows 4 g .. 4 g + 3 and the same LANES * 4 further on of four neighbouring columns (LANES lanes cover the head's rows).
+template <int LANES>
+__global__ void __launch_bounds__(128) delta_blocks_kernel(const BlockArgs a) {
+  extern __shared__ __align__(16) float blocks_shared[];
+  constexpr int C = 4, CHUNKS = 2, PAIRS = 2 * CHUNKS;   // eight rows a thread as four pairs
+  constexpr int N = BLOCK * C, OWN = N / LANES > 0 ? N / LANES : 1;
+  const ScanArgs& s = a.s;
+  let_dependents_start();
+  wait_for_previous();
+  const int local_head = blockIdx.y, head = a.head0 + local_head, seq = blockIdx.z, cols = s.cols, col0 = blockIdx.x * cols;
+  const int first = s.q_start[seq], length = s.q_start[seq + 1] - first;
+  if (length < a.from) return;   // the token-by-token walk serves it
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane % LANES, team = lane / LANES;
+  const int j = (warp * (32 / LANES) + team) * C;   // the first of this thread's columns among the CTA's
+  const int cols_here = min(cols, s.vdim - col0);
+  const int slot = s.state_slot[seq];
+  const size_t out_width = static_cast<size_t>(s.heads) * s.vdim;
+  float* out = s.out + static_cast<size_t>(first) * out_width + head * s.vdim + col0;
+  if (slot < 0 || slot >= s.num_slots) {
+    for (int t = 0; t < length; ++t)
+      for (int c = threadIdx.x; c < cols_here; c += blockDim.x) out[t * out_width + c] = 0.f;
+    return;
+  }
+  int base = 0;   // the sequence's first block
+  for (int other = lane; other < seq; other += 32) base += blocks_of(a, other);
+#pragma unroll
+  for (int offset = 16; offset > 0; offset >>= 1) base += __shfl_xor_sync(0xffffffffu, base, offset);
+  const int Dp = a.padded_dim;
+  const int blocks = (length + BLOCK - 1) / BLOCK;
+  const int stage_floats = a.record + BLOCK * cols;
+  float* team_values = blocks_shared + STAGES * stage_floats + (warp * (32 / LANES) + team) * 2 * N;   // d, then c, of this team's columns
+  const int v_col = 2 * s.kv_heads * s.dim + head * s.vdim + col0;
+  const bool wide_v = ((v_col | s.channels | s.vdim) & 3) == 0 && (reinterpret_cast<uintptr_t>(s.mixed) & 15) == 0;
+  const auto stage = [&](int block) {   // asks for a block's record and the CTA's columns of v
+    if (block < blocks) {
+      float* at = blocks_shared + (block % STAGES) * stage_floats;
+      const float* record = a.records + (static_cast<size_t>(base + block) * a.head_count + local_head) * a.record;
+      for (int i = threadIdx.x * 4; i < a.record; i += blockDim.x * 4) copy16(at + i, record + i);
+      float* v = at + a.record;
+      const int here = min(BLOCK, length - block * BLOCK);
+      const float* from = s.mixed + static_cast<size_t>(first + block * BLOCK) * s.channels + v_col;
+      if (wide_v) {
+        for (int i = threadIdx.x; i < BLOCK * cols / 4; i += blockDim.x) {
+          const int t = i / (cols / 4), c = (i - t * (cols / 4)) * 4;
+          if (t < here && c < cols_here) copy16(v + t * cols + c, from + static_cast<size_t>(t) * s.channels + c);
+          else *reinterpret_cast<float4*>(v + t * cols + c) = make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+      } else {
+        for (int i = threadIdx.x; i < BLOCK * cols; i += blockDim.x) {
+          const int t = i / cols, c = i - t * cols;
+          if (t < here && c < cols_here) copy4(v + i, from + static_cast<size_t>(t) * s.channels + c);
+          else v[i] = 0.f;
+        }
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+#pragma unroll
+  for (int i = 0; i < STAGES - 1; ++i) stage(i);
+  float* state = s.state + (static_cast<size_t>(slot) * s.heads + head) * s.head_stride;
+  const bool wide = (s.vdim & 3) == 0;
+  unsigned long long S[C][PAIRS];
+  {
+    float row[2][C];
+#pragma unroll
+    for (int p = 0; p < PAIRS; ++p) {
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int d = (p / 2) * 4 * LANES + 4 * g + (p & 1) * 2 + h;
+        const float* at = state + static_cast<size_t>(d) * s.vdim + col0 + j;
+#pragma unroll
+        for (int c = 0; c < C; ++c) row[h][c] = 0.f;
+        if (d < s.dim) {
+          if (wide) {
+            if (j < cols_here) load4<float>(at, row[h]);
+          } else {
+#pragma unroll
+            for (int c = 0; c < C; ++c)
+              if (j + c < cols_here) row[h][c] = at[c];
+          }
+        }
+      }
+#pragma unroll
+      for (int c = 0; c < C; ++c) S[c][p] = pack2(row[0][c], row[1][c]);
+    }
+  }
+  for (int block = 0; block < blocks; ++block) {
+    asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
+    __syncthreads();   // the block's record is there, and everyone is done with the stage that is filled next
+    stage(block + STAGES - 1);
+    const float* at = blocks_shared + (block % STAGES) * stage_floats;
+    const ulonglong2* rows = reinterpret_cast<const ulonglong2*>(at) + g;   // row r: + r * Dp / 4; chunk: + LANES
+    const int pitch = Dp / 4;
+    const float* v = at + a.record;
+    float sum[2][N];   // a_t, then c_t, of this thread's rows; t * C + c
+#pragma unroll
+    for (int which = 0; which < 2; ++which) {
+#pragma unroll
+      for (int t = 0; t < BLOCK; ++t) {
+        unsigned long long acc[C];
+#pragma unroll
+        for (int chunk = 0; chunk < CHUNKS; ++chunk) {
+          const ulonglong2 x = rows[(which * BLOCK + t) * pitch + chunk * LANES];
+#pragma unroll
+          for (int c = 0; c < C; ++c) {
+            acc[c] = chunk == 0 ? mul2(S[c][0], x.x) : fma2(S[c][2 * chunk], x.x, acc[c]);
+            acc[c] = fma2(S[c][2 * chunk + 1], x.y, acc[c]);
+          }
+        }
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+          const float2 f = unpack2(acc[c]);
+          sum[which][t * C + c] = f.x + f.y;
+        }
+      }
+      FoldLanes<N, LANES / 2>::run(sum[which], lane);
+      // this lane holds the sums g * OWN .. of its team's N; d_t = v_t - a_t
+#pragma unroll
+      for (int i = 0; i < OWN; ++i) {
+        const int at_value = g * OWN + i, t = at_value / C, c = at_value % C;
+        team_values[which * N + at_value] = which == 0 ? v[t * cols + j + c] - sum[0][i] : sum[1][i];
+      }
+    }
+    __syncwarp();
+    const float* decay = at + 3 * BLOCK * Dp;
+#pragma unroll
+    for (int chunk = 0; chunk < CHUNKS; ++chunk) {
+      const ulonglong2 x = *(reinterpret_cast<const ulonglong2*>(decay) + g + chunk * LANES);
+#pragma unroll
+      for (int c = 0; c < C; ++c) {
+        S[c][2 * chunk] = mul2(S[c][2 * chunk], x.x);
+        S[c][2 * chunk + 1] = mul2(S[c][2 * chunk + 1], x.y);
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < BLOCK; ++t) {
+      const float4 d = *reinterpret_cast<const float4*>(team_values + t * C);
+      const unsigned long long dd[C] = {pack2(d.x, d.x), pack2(d.y, d.y), pack2(d.z, d.z), pack2(d.w, d.w)};
+#pragma unroll
+      for (int chunk = 0; chunk < CHUNKS; ++chunk) {
+        const ulonglong2 x = rows[(2 * BLOCK + t) * pitch + chunk * LANES];
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+          S[c][2 * chunk] = fma2(x.x, dd[c], S[c][2 * chunk]);
+          S[c][2 * chunk + 1] = fma2(x.y, dd[c], S[c][2 * chunk + 1]);
+        }
+      }
+    }
+    const float* m = decay + Dp;
+    const int here = min(BLOCK, length - block * BLOCK);
+#pragma unroll
+    for (int i = 0; i < (N + LANES - 1) / LANES; ++i) {
+      const int at_value = g + i * LANES, t = at_value / C, c = at_value % C;
+      if (at_value < N && t < here && j + c < cols_here) {
+        float o = team_values[N + at_value];
+#pragma unroll
+        for (int r = 0; r < BLOCK; r += 4) {
+          const float4 row = *reinterpret_cast<const float4*>(m + t * BLOCK + r);
+          o = __fmaf_rn(row.x, team_values[r * C + c], o);
+          o = __fmaf_rn(row.y, team_values[(r + 1) * C + c], o);
+          o = __fmaf_rn(row.z, team_values[(r + 2) * C + c], o);
+          o = __fmaf_rn(row.w, team_values[(r + 3) * C + c], o);
+        }
+        out[static_cast<size_t>(block * BLOCK + t) * out_width + j + c] = o;
+      }
+    }
+    __syncwarp();   // the team's values are used up before the next block overwrites them
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+#pragma unroll
+  for (int p = 0; p < PAIRS; ++p) {
+    float2 row[C];
+#pragma unroll
+    for (int c = 0; c < C; ++c) row[c] = unpack2(S[c][p]);
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int d = (p / 2) * 4 * LANES + 4 * g + (p & 1) * 2 + h;
+      if (d >= s.dim) continue;
+      float* at = state + static_cast<size_t>(d) * s.vdim + col0 + j;
+      float four[C];
+#pragma unroll
+      for (int c = 0; c < C; ++c) four[c] = h == 0 ? row[c].x : row[c].y;
+      if (wide) {
+        if (j < cols_here) store4<float>(at, four);
+      } else {
+#pragma unroll
+        for (int c = 0; c < C; ++c)
+          if (j + c < cols_here) at[c] = four[c];
+      }
+    }
+  }
+}
+
 }  // namespace delta
 
 // =========================================================================================== launchers
 using namespace delta;
 
-// `longest`: the most new tokens a sequence of the batch brings; 1: the kernel also moves every sequence's convolution
-// state up by its token, otherwise the caller updates the states afterwards (shrike_short_conv_keep).
+extern "C" int shrike_short_conv_keep(const float* fused, int partials, long long stride, int total, float* state,
+                                      const int* q_start, const int* state_slot, int channels, int taps_count, int num_seqs,
+                                      int num_slots, cudaStream_t stream);
+
+// `longest`: the most new tokens a sequence of the batch brings (0: not known).  A batch of up to 64 single tokens has its
+// convolution states moved up by the kernel itself, otherwise a second launch updates them.
 SHRIKE_API int shrike_delta_prep(const float* fused, int partials, long long stride, int total, const float* taps, float* state,
                                  const int* q_start, const int* state_slot, const int* seq_of_token, float* mixed, float* beta,
                                  void* low, int dtype, int n, int heads, int kv_heads, int dim, int vdim, int taps_count,
-                                 int beta_at, int low_at, int low_width, int num_slots, float unit_eps, float q_scale,
+                                 int beta_at, int low_at, int low_width, int num_seqs, int num_slots, float unit_eps, float q_scale,
                                  int longest, cudaStream_t stream) {
   if (n <= 0) return SHRIKE_OK;
   if (heads < 1 || kv_heads < 1 || heads % kv_heads || dim < 1 || vdim < 1 || taps_count < 1 || taps_count > MAX_TAPS || partials < 1)
@@ -381,12 +819,19 @@ SHRIKE_API int shrike_delta_prep(const float* fused, int partials, long long str
                 longest == 1 ? 1 : 0};
   const bool vec = dim % 4 == 0 && vdim % 4 == 0 && total % 4 == 0 && stride % 4 == 0 &&
                    (reinterpret_cast<uintptr_t>(fused) | reinterpret_cast<uintptr_t>(mixed)) % 16 == 0;
-  const int units = 2 * kv_heads + heads + 1;
-  const dim3 grid(static_cast<unsigned>((n + TILE - 1) / TILE), static_cast<unsigned>((units + 3) / 4));
+  const bool few = n <= 64 || partials > 1;   // a warp a token and head; otherwise TILE tokens a warp
+  const int units = 2 * kv_heads + heads + (heads + low_width + REST - 1) / REST;
+  const int tile = few ? 1 : TILE;
+  const dim3 grid(static_cast<unsigned>((n + tile - 1) / tile), static_cast<unsigned>((units + 3) / 4));
   if (grid.y > 65535) return SHRIKE_BAD_ARGUMENT;
-#define SHRIKE_PREP(TO, T, V) launch_dependent(delta_prep_kernel<TO, T, V>, grid, 128, 0, stream, a)
-#define SHRIKE_PREP_TAPS(TO, V)                   \
-  do {                                            \
+  if (longest == 1 && !few) a.keep = 0;
+#define SHRIKE_PREP(TO, T, V)                                                                     \
+  do {                                                                                            \
+    if (few) launch_dependent(delta_prep_kernel<TO, T, V, 1>, grid, 128, 0, stream, a);           \
+    else launch_dependent(delta_prep_kernel<TO, T, V, TILE>, grid, 128, 0, stream, a);            \
+  } while (0)
+#define SHRIKE_PREP_TAPS(TO, V)                      \
+  do {                                               \
     if (taps_count == 1) SHRIKE_PREP(TO, 1, V);      \
     else if (taps_count == 2) SHRIKE_PREP(TO, 2, V); \
     else if (taps_count == 3) SHRIKE_PREP(TO, 3, V); \
@@ -398,7 +843,11 @@ SHRIKE_API int shrike_delta_prep(const float* fused, int partials, long long str
   else return SHRIKE_BAD_ARGUMENT;
 #undef SHRIKE_PREP_TAPS
 #undef SHRIKE_PREP
-  return shrike_launch_status();
+  const int status = shrike_launch_status();
+  if (status != SHRIKE_OK || taps_count == 1 || a.keep) return status;
+  // only after every token has read the old states
+  return shrike_short_conv_keep(fused, partials, stride, total, state, q_start, state_slot, channels, taps_count, num_seqs,
+                                num_slots, stream);
 }
 
 // How a walk is laid out for heads of dim x vdim: R rows of C columns a thread, the lanes that share those columns.
@@ -415,10 +864,22 @@ static inline bool delta_shape(int dim, int vdim, DeltaShape* shape) {
   return shape->smem <= static_cast<size_t>(shrike_device().max_smem);
 }
 
+// Scratch floats of one head of one block of BLOCK tokens; 0: heads of this size walk token by token.
+SHRIKE_API int shrike_delta_scan_record(int dim) {
+  DeltaShape shape;
+  if (dim > 256 || !delta_shape(dim, 4, &shape)) return 0;
+  return record_floats(shape.lanes * shape.rows);
+}
+SHRIKE_API int shrike_delta_scan_block() { return BLOCK; }
+
+// Sequences that bring at least `from` tokens (0: none) run in blocks, for which the caller holds `records`
+// (blocks x head_count x shrike_delta_scan_record floats, `blocks` = the sum of ceil(length / BLOCK) over them); heads are
+// then served `head_count` at a time.  `shorter`: whether the batch has sequences below `from`.
 SHRIKE_API int shrike_delta_scan(const float* mixed, const float* beta, const float* gates, int partials, long long stride,
                                  int gate_width, const float* rate, const float* bias, float* state, const int* q_start,
                                  const int* state_slot, float* out, int num_seqs, int heads, int kv_heads, int dim, int vdim,
-                                 int head_stride, int num_slots, cudaStream_t stream) {
+                                 int head_stride, int num_slots, int from, int shorter, float* records, int blocks,
+                                 int head_count, cudaStream_t stream) {
   if (num_seqs <= 0) return SHRIKE_OK;
   if (heads < 1 || heads > 65535 || num_seqs > 65535 || kv_heads < 1 || heads % kv_heads || dim < 1 || vdim < 1 || partials < 1 ||
       head_stride < dim * vdim || gate_width < heads * dim)
@@ -427,10 +888,41 @@ SHRIKE_API int shrike_delta_scan(const float* mixed, const float* beta, const fl
   DeltaShape shape;
   if (!delta_shape(dim, vdim, &shape)) return SHRIKE_BAD_ARGUMENT;   // heads of more than 1,024 rows
   ScanArgs a = {mixed, beta, gates, stride, partials, gate_width, rate, bias, state, q_start, state_slot, out,
-                heads, kv_heads, dim, vdim, 2 * kv_heads * dim + heads * vdim, head_stride, num_slots, shape.lanes, shape.cols};
-  void (*kernel)(ScanArgs) = shape.rows == 8 ? delta_walk_kernel<8, 4> : delta_walk_kernel<32, 1>;
-  if (shape.smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shape.smem));
-  const dim3 grid(static_cast<unsigned>((vdim + shape.cols - 1) / shape.cols), heads, num_seqs);
-  launch_dependent(kernel, grid, static_cast<unsigned>(shape.threads), shape.smem, stream, a);
+                heads, kv_heads, dim, vdim, 2 * kv_heads * dim + heads * vdim, head_stride, num_slots, shape.lanes, shape.cols, 0};
+  const bool in_blocks = from > 0 && records != nullptr && blocks > 0 && head_count > 0 && shape.rows == 8;
+  const unsigned slices = static_cast<unsigned>((vdim + shape.cols - 1) / shape.cols);
+  if (!in_blocks || shorter) {
+    a.skip_from = in_blocks ? from : 0;
+    void (*kernel)(ScanArgs) = shape.rows == 8 ? delta_walk_kernel<8, 4> : delta_walk_kernel<32, 1>;
+    if (shape.smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shape.smem));
+    launch_dependent(kernel, dim3(slices, heads, num_seqs), static_cast<unsigned>(shape.threads), shape.smem, stream, a);
+  }
+  if (in_blocks) {
+    BlockArgs b = {};
+    b.s = a;
+    b.records = records;
+    b.padded_dim = shape.lanes * shape.rows;
+    b.record = record_floats(b.padded_dim);
+    b.num_seqs = num_seqs; b.from = from; b.blocks = blocks;
+    void (*kernel)(BlockArgs) = nullptr;
+    switch (shape.lanes) {
+      case 1: kernel = delta_blocks_kernel<1>; break;
+      case 2: kernel = delta_blocks_kernel<2>; break;
+      case 4: kernel = delta_blocks_kernel<4>; break;
+      case 8: kernel = delta_blocks_kernel<8>; break;
+      case 16: kernel = delta_blocks_kernel<16>; break;
+      default: kernel = delta_blocks_kernel<32>; break;
+    }
+    const int teams = shape.threads / shape.lanes;
+    const size_t smem = (static_cast<size_t>(STAGES) * (b.record + BLOCK * shape.cols) + static_cast<size_t>(teams) * 2 * BLOCK * 4) * sizeof(float);
+    if (smem > static_cast<size_t>(shrike_device().max_smem)) return SHRIKE_BAD_ARGUMENT;
+    if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    for (int head0 = 0; head0 < heads; head0 += head_count) {
+      b.head0 = head0;
+      b.head_count = min(head_count, heads - head0);
+      launch_dependent(delta_local_kernel, dim3(static_cast<unsigned>(blocks), static_cast<unsigned>((b.head_count + 3) / 4)), 128, 0, stream, b);
+      launch_dependent(kernel, dim3(slices, b.head_count, num_seqs), static_cast<unsigned>(shape.threads), smem, stream, b);
+    }
+  }
   return shrike_launch_status();
 }

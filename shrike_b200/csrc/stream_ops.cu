@@ -498,8 +498,13 @@ __global__ void __launch_bounds__(256) gated_scan_carry_kernel(const ScanArgs a)
 }
 
 // ------------------------------------------------------------------------------------------------ head_rms
-// A warp a head; VEC = 4: 16-byte accesses.  `gates` (may be null): the result is multiplied by the sigmoid of column
-// gate_at + (head, element) of a fused projection ([partials][N][gate_width]).
+// A warp two heads; VEC = 4: 16-byte accesses.  `gates` (may be null): the result is multiplied by the sigmoid of column
+// gate_at + (head, element) of a fused projection ([partials][N][gate_width]).  A head of up to 32 groups stays in
+// registers, its gates' loads in flight with its own.
+template <typename TO> __device__ __forceinline__ float sigmoid_for(float z);
+template <> __device__ __forceinline__ float sigmoid_for<float>(float z) { return 1.0f / (1.0f + expf(-z)); }
+template <> __device__ __forceinline__ float sigmoid_for<__nv_bfloat16>(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
+
 template <typename TO, int VEC>
 __global__ void __launch_bounds__(128) head_rms_kernel(const float* __restrict__ x, const float* __restrict__ weight,
                                                        TO* __restrict__ out, int n, int heads, int size, float eps,
@@ -507,37 +512,56 @@ __global__ void __launch_bounds__(128) head_rms_kernel(const float* __restrict__
                                                        int gate_width, int gate_at) {
   let_dependents_start();
   wait_for_previous();
+  constexpr int UNITS = 2;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const long long unit = static_cast<long long>(blockIdx.x) * 4 + warp;
-  if (unit >= static_cast<long long>(n) * heads) return;
-  const float* row = x + unit * size;
+  const long long unit0 = (static_cast<long long>(blockIdx.x) * 4 + warp) * UNITS, units = static_cast<long long>(n) * heads;
   const int groups = size / VEC;
-  const float* gate_row = gates != nullptr ? gates + (unit / heads) * gate_width + gate_at + (unit % heads) * size : nullptr;
-  float squares = 0.f;
-  for (int g = lane; g < groups; g += 32) {
-    float v[VEC];
-    if constexpr (VEC == 4) load4<float>(row + g * 4, v);
-    else v[0] = row[g];
+  const bool single = groups <= 32;
+  float v[UNITS][VEC], z[UNITS][VEC], squares[UNITS];
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) squares = __fmaf_rn(v[e], v[e], squares);
+  for (int u = 0; u < UNITS; ++u) {
+    squares[u] = 0.f;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v[u][e] = z[u][e] = 0.f;
+    const long long unit = unit0 + u;
+    if (unit >= units) continue;
+    const float* row = x + unit * size;
+    for (int g = lane; g < groups; g += 32) {
+      if constexpr (VEC == 4) load4<float>(row + g * 4, v[u]);
+      else v[u][0] = row[g];
+      if (single && gates != nullptr) {
+        const float* gate = gates + (unit / heads) * gate_width + gate_at + (unit % heads) * size + g * VEC;
+        if constexpr (VEC == 4) sum_partials4(gate, stride, partials, z[u]);
+        else z[u][0] = sum_partials(gate, stride, partials);
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) squares[u] = __fmaf_rn(v[u][e], v[u][e], squares[u]);
+    }
   }
-  const float r = rsqrtf(warp_sum(squares) / static_cast<float>(size) + eps);
-  for (int g = lane; g < groups; g += 32) {
-    float v[VEC], z[VEC] = {};
-    if constexpr (VEC == 4) {
-      load4<float>(row + g * 4, v);
-      if (gate_row != nullptr) sum_partials4(gate_row + g * 4, stride, partials, z);
-    } else {
-      v[0] = row[g];
-      if (gate_row != nullptr) z[0] = sum_partials(gate_row + g, stride, partials);
-    }
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) {
-      v[e] = v[e] * r * (weight != nullptr ? weight[g * VEC + e] : 1.f);
-      if (gate_row != nullptr) v[e] = v[e] / (1.0f + expf(-z[e]));
+  for (int u = 0; u < UNITS; ++u) {
+    const long long unit = unit0 + u;
+    if (unit >= units) continue;
+    const float r = rsqrtf(warp_sum(squares[u]) / static_cast<float>(size) + eps);
+    for (int g = lane; g < groups; g += 32) {
+      if (!single) {
+        if constexpr (VEC == 4) load4<float>(x + unit * size + g * 4, v[u]);
+        else v[u][0] = x[unit * size + g];
+        if (gates != nullptr) {
+          const float* gate = gates + (unit / heads) * gate_width + gate_at + (unit % heads) * size + g * VEC;
+          if constexpr (VEC == 4) sum_partials4(gate, stride, partials, z[u]);
+          else z[u][0] = sum_partials(gate, stride, partials);
+        }
+      }
+      float w[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        w[e] = v[u][e] * r * (weight != nullptr ? weight[g * VEC + e] : 1.f);
+        if (gates != nullptr) w[e] *= sigmoid_for<TO>(z[u][e]);
+      }
+      if constexpr (VEC == 4) store4<TO>(out + unit * size + g * 4, w);
+      else out[unit * size + g] = from_float<TO>(w[0]);
     }
-    if constexpr (VEC == 4) store4<TO>(out + unit * size + g * 4, v);
-    else out[unit * size + g] = from_float<TO>(v[0]);
   }
 }
 
@@ -707,7 +731,7 @@ SHRIKE_API int shrike_head_rms(const float* x, const float* weight, void* out, i
   if (heads < 1 || size < 1 || partials < 1) return SHRIKE_BAD_ARGUMENT;
   if (gates != nullptr && (gate_at < 0 || gate_at + heads * size > gate_width)) return SHRIKE_BAD_ARGUMENT;
   const long long units = static_cast<long long>(n) * heads;
-  const long long blocks = (units + 3) / 4;
+  const long long blocks = (units + 7) / 8;
   if (blocks > 0x7fffffffLL) return SHRIKE_BAD_ARGUMENT;
   const bool vec = size % 4 == 0 && (reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out)) % 16 == 0 &&
                    (gates == nullptr || (reinterpret_cast<uintptr_t>(gates) % 16 == 0 && gate_at % 4 == 0 && gate_width % 4 == 0 && stride % 4 == 0));

@@ -129,6 +129,7 @@ class CudaOps:
         self._memory_scratch = None   # what the matrix memory's chunk kernels hand from one launch to the next
         self._decay_scratch = None    # the same for the decayed linear attention: a state per run of tokens
         self._scan_scratch = None     # the gated recurrence's runs of tokens: each run's state, decay and first index
+        self._delta_scratch = None    # the delta rule's blocks of tokens: what the walk over them reads
         self.portion_splits = 0  # 0: the kernel library's rule; n: that many key splits for portions (tests)
         self.generation = 0      # grows when the scratch moves
         self._held_stream = None
@@ -188,8 +189,11 @@ class CudaOps:
         lib.shrike_plain_act.argtypes = [_P, _I, _LL, _I, _P]
         lib.shrike_side_gate.argtypes = [_P, _I, _LL, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _P, _I, _P]
         lib.shrike_short_conv_keep.argtypes = [_P, _I, _LL, _I, _P, _P, _P, _I, _I, _I, _I, _P]
-        lib.shrike_delta_prep.argtypes = [_P, _I, _LL, _I, _P, _P, _P, _P, _P, _P, _P, _P] + [_I] * 11 + [_F, _F, _I, _P]
-        lib.shrike_delta_scan.argtypes = [_P, _P, _P, _I, _LL, _I, _P, _P, _P, _P, _P, _P] + [_I] * 7 + [_P]
+        lib.shrike_delta_prep.argtypes = [_P, _I, _LL, _I, _P, _P, _P, _P, _P, _P, _P, _P] + [_I] * 12 + [_F, _F, _I, _P]
+        lib.shrike_delta_scan.argtypes = [_P, _P, _P, _I, _LL, _I, _P, _P, _P, _P, _P, _P] + [_I] * 9 + [_P, _I, _I, _P]
+        lib.shrike_delta_scan_record.argtypes = [_I]
+        lib.shrike_delta_scan_record.restype = _I
+        lib.shrike_delta_scan_block.restype = _I
         for name in ("shrike_decay_scan", "shrike_norm_gate", "shrike_latent_rope_store", "shrike_concat_cast",
                      "shrike_stream_norm", "shrike_short_conv", "shrike_gated_scan", "shrike_head_rms",
                      "shrike_head_prep_norms", "shrike_route_top_scores", "shrike_act_mul_blocks_at",
@@ -1179,17 +1183,15 @@ class CudaOps:
             raise KernelError(f"delta_prep: taps {tuple(taps.shape)}, q, k and v {tuple(mixed.shape)}")
         if count > 1 and tuple(conv_state.shape[1:]) != (count - 1, channels):
             raise KernelError("delta_prep: conv_state [slots, T - 1, channels]")
-        self.launches += 1
+        self.launches += 1 if count == 1 or (longest == 1 and n <= 64) else 2
         _check(self.core.shrike_delta_prep(
             _ptr(fused), partials, stride, total, _ptr(taps), _ptr(conv_state), _ptr(q_start), _ptr(state_slot),
             _ptr(seq_of_token), _ptr(mixed), _ptr(beta), _ptr(low), self.code, n, num_heads, num_kv_heads, dim, vdim, count,
-            beta_at, low_at, low.shape[1], conv_state.shape[0], unit_eps, float(dim) ** -0.5, int(longest), self._stream()),
-            "delta_prep")
-        if count > 1 and longest != 1:   # only after every token has read the old state
-            self.launches += 1
-            _check(self.core.shrike_short_conv_keep(_ptr(fused), partials, stride, total, _ptr(conv_state), _ptr(q_start),
-                                                    _ptr(state_slot), channels, count, num_seqs, conv_state.shape[0],
-                                                    self._stream()), "short_conv")
+            beta_at, low_at, low.shape[1], num_seqs, conv_state.shape[0], unit_eps, float(dim) ** -0.5, int(longest),
+            self._stream()), "delta_prep")
+
+    DELTA_BLOCKS_FROM = 16            # a sequence that brings at least this many tokens goes eight tokens at a time
+    DELTA_SCRATCH_FLOATS = 64 << 20   # at most 256 MiB of what the blocks hand to the walk: heads take turns beyond
 
     def delta_scan(self, mixed, beta, gates, rate, bias, state, q_start, state_slot, out, num_seqs, num_heads, num_kv_heads,
                    dim, vdim, q_lens=None):
@@ -1197,18 +1199,34 @@ class CudaOps:
         `delta_prep` leaves it): S <- diag(g) S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q, with g =
         exp(-rate[h] softplus(z + bias)), z column h dim + d of `gates` ([N, at least H dim] float32 or a K-split stack).
         `state` float32 [slots, H, at least dim * vdim, a multiple of four] is read and left updated for the slots
-        `state_slot` names (-1: zeros out, nothing kept); `out` float32 [N, H * vdim]."""
+        `state_slot` names (-1: zeros out, nothing kept); `out` float32 [N, H * vdim].  `q_lens` (the batch's lengths, host):
+        longer portions go eight tokens at a time, with the same result up to the order of the sums; without it every
+        sequence walks token by token."""
         for name, tensor in (("q, k and v", mixed), ("beta", beta), ("gates", gates), ("rate", rate), ("bias", bias),
                              ("state", state), ("scan output", out)):
             _dense(tensor, torch.float32, name)
         partials, stride = self._stack(gates)
         if state.dim() != 3 or state.shape[1] != num_heads or state.shape[2] < dim * vdim or bias.numel() != num_heads * dim:
             raise KernelError(f"state {tuple(state.shape)} does not fit {num_heads} heads of {dim} x {vdim}")
-        self.launches += 1
+        blocks, records, head_count, shorter = 0, None, 0, True
+        record = self.core.shrike_delta_scan_record(dim) if q_lens is not None and max(q_lens) >= self.DELTA_BLOCKS_FROM else 0
+        if record:
+            size = self.core.shrike_delta_scan_block()
+            blocks = sum(-(-length // size) for length in q_lens if length >= self.DELTA_BLOCKS_FROM)
+            shorter = min(q_lens) < self.DELTA_BLOCKS_FROM
+            turns = -(-num_heads * blocks * record // self.DELTA_SCRATCH_FLOATS)
+            head_count = max(1, -(-num_heads // turns))
+            need = blocks * head_count * record
+            if self._delta_scratch is None or self._delta_scratch.numel() < need:
+                self._delta_scratch = torch.empty(max(need, 1 << 20), dtype=torch.float32, device=self.device)
+                self.generation += 1
+            records = self._delta_scratch
+        self.launches += int(shorter) + (2 * -(-num_heads // head_count) if blocks else 0)
         _check(self.core.shrike_delta_scan(
             _ptr(mixed), _ptr(beta), _ptr(gates), partials, stride, gates.shape[-1], _ptr(rate), _ptr(bias), _ptr(state),
             _ptr(q_start), _ptr(state_slot), _ptr(out), num_seqs, num_heads, num_kv_heads, dim, vdim, state.shape[2],
-            state.shape[0], self._stream()), "delta_scan")
+            state.shape[0], self.DELTA_BLOCKS_FROM if blocks else 0, int(shorter), _ptr(records), blocks, head_count,
+            self._stream()), "delta_scan")
 
     def sample(self, logits, temperature, top_p, seeds, out):
         _dense(logits, torch.float32, "logits")
