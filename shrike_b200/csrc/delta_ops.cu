@@ -428,20 +428,26 @@ __device__ __forceinline__ int blocks_of(const BlockArgs& a, int seq) {
   return length >= a.from ? (length + BLOCK - 1) / BLOCK : 0;
 }
 
-// The sum of `count` (a power of two times 1) values over 2 * `OFFSET` lanes, transposed: every step halves the values a
-// lane holds, so that lane g of them ends with the sums of values g * n .. g * n + n - 1, n = COUNT / lanes (at least one).
+// The sums of COUNT values over 2 * OFFSET lanes, transposed: every step halves the values a lane holds, so that lane g of
+// L ends with the sums of values g * n .. g * n + n - 1, n = COUNT / L; where the lanes outnumber the values, lanes that
+// differ in the lowest bits end with the same one.
 template <int COUNT, int OFFSET>
 struct FoldLanes {
   static __device__ __forceinline__ void run(float* v, int lane) {
     if constexpr (OFFSET > 0) {
-      constexpr int HALF = COUNT / 2;
-      const bool upper = lane & OFFSET;
+      if constexpr (COUNT > 1) {
+        constexpr int HALF = COUNT / 2;
+        const bool upper = lane & OFFSET;
 #pragma unroll
-      for (int i = 0; i < HALF; ++i) {
-        const float send = upper ? v[i] : v[i + HALF], keep = upper ? v[i + HALF] : v[i];
-        v[i] = keep + __shfl_xor_sync(0xffffffffu, send, OFFSET);
+        for (int i = 0; i < HALF; ++i) {
+          const float send = upper ? v[i] : v[i + HALF], keep = upper ? v[i + HALF] : v[i];
+          v[i] = keep + __shfl_xor_sync(0xffffffffu, send, OFFSET);
+        }
+        FoldLanes<HALF, OFFSET / 2>::run(v, lane);
+      } else {
+        v[0] += __shfl_xor_sync(0xffffffffu, v[0], OFFSET);
+        FoldLanes<1, OFFSET / 2>::run(v, lane);
       }
-      FoldLanes<HALF, OFFSET / 2>::run(v, lane);
     }
   }
 };
@@ -449,8 +455,7 @@ struct FoldLanes {
 // grid (blocks, heads / 4): a warp a block and value head.
 __global__ void __launch_bounds__(128) delta_local_kernel(const BlockArgs a) {
   __shared__ float shared_w[4][BLOCK * BLOCK], shared_t[4][BLOCK * BLOCK];
-  let_dependents_start();
-  wait_for_previous();
+  wait_for_previous();   // the walk may start only when this kernel is nearly done: see the end
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int block = blockIdx.x, local_head = blockIdx.y * 4 + warp;
   if (local_head >= a.head_count) return;
@@ -567,6 +572,9 @@ __global__ void __launch_bounds__(128) delta_local_kernel(const BlockArgs a) {
       kk[c * Dp + d] = v;
     }
   }
+  // (a CTA that leaves counts as having let its dependents start.)  A walk launched while these CTAs still fill the
+  // device would be packed onto the few SMs that free up first, several of its long-running CTAs to an SM.
+  let_dependents_start();
 }
 
 // Two float32 multiply-adds in one instruction.
@@ -600,12 +608,16 @@ __device__ __forceinline__ void copy4(void* shared, const void* global) {
 constexpr int STAGES = 3;
 
 // grid (slices, heads, sequences): a CTA owns `cols` value columns of one head's state for one sequence.  A thread holds
-// rows 4 g .. 4 g + 3 and the same LANES * 4 further on of four neighbouring columns (LANES lanes cover the head's rows).
-template <int LANES>
-__global__ void __launch_bounds__(128) delta_blocks_kernel(const BlockArgs a) {
+// rows 4 g .. 4 g + 3 (with CHUNKS 2 also the same LANES * 4 further on) of four neighbouring columns; LANES lanes, a
+// team, cover the head's rows.  Register c of a lane is column c ^ turn of the team's four, `turn` the lane's top two bits:
+// adding up over those lanes then needs no selection, every step keeps the first half of the columns and sends the other.
+template <int LANES, int CHUNKS>
+__global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(const BlockArgs a) {
   extern __shared__ __align__(16) float blocks_shared[];
-  constexpr int C = 4, CHUNKS = 2, PAIRS = 2 * CHUNKS;   // eight rows a thread as four pairs
-  constexpr int N = BLOCK * C, OWN = N / LANES > 0 ? N / LANES : 1;
+  constexpr int C = 4, PAIRS = 2 * CHUNKS, N = BLOCK * C;
+  constexpr int COLUMN_LANES = LANES >= C ? C : LANES;   // lanes the columns are shared out over, then the tokens
+  constexpr int TOKEN_LANES = LANES / COLUMN_LANES;
+  constexpr int OWN_COLUMNS = C / COLUMN_LANES, OWN_TOKENS = BLOCK / TOKEN_LANES;
   const ScanArgs& s = a.s;
   let_dependents_start();
   wait_for_previous();
@@ -613,7 +625,8 @@ __global__ void __launch_bounds__(128) delta_blocks_kernel(const BlockArgs a) {
   const int first = s.q_start[seq], length = s.q_start[seq + 1] - first;
   if (length < a.from) return;   // the token-by-token walk serves it
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane % LANES, team = lane / LANES;
-  const int j = (warp * (32 / LANES) + team) * C;   // the first of this thread's columns among the CTA's
+  const int j = (warp * (32 / LANES) + team) * C;   // the first of the team's columns among the CTA's
+  const int turn = COLUMN_LANES == 4 ? g / TOKEN_LANES : (COLUMN_LANES == 2 ? 2 * g : 0);
   const int cols_here = min(cols, s.vdim - col0);
   const int slot = s.state_slot[seq];
   const size_t out_width = static_cast<size_t>(s.heads) * s.vdim;
@@ -660,41 +673,25 @@ __global__ void __launch_bounds__(128) delta_blocks_kernel(const BlockArgs a) {
 #pragma unroll
   for (int i = 0; i < STAGES - 1; ++i) stage(i);
   float* state = s.state + (static_cast<size_t>(slot) * s.heads + head) * s.head_stride;
-  const bool wide = (s.vdim & 3) == 0;
   unsigned long long S[C][PAIRS];
-  {
-    float row[2][C];
 #pragma unroll
-    for (int p = 0; p < PAIRS; ++p) {
+  for (int p = 0; p < PAIRS; ++p)
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const int d = (p / 2) * 4 * LANES + 4 * g + (p & 1) * 2 + h;
-        const float* at = state + static_cast<size_t>(d) * s.vdim + col0 + j;
-#pragma unroll
-        for (int c = 0; c < C; ++c) row[h][c] = 0.f;
-        if (d < s.dim) {
-          if (wide) {
-            if (j < cols_here) load4<float>(at, row[h]);
-          } else {
-#pragma unroll
-            for (int c = 0; c < C; ++c)
-              if (j + c < cols_here) row[h][c] = at[c];
-          }
-        }
-      }
-#pragma unroll
-      for (int c = 0; c < C; ++c) S[c][p] = pack2(row[0][c], row[1][c]);
+    for (int c = 0; c < C; ++c) {
+      const int d = (p / 2) * 4 * LANES + 4 * g + (p & 1) * 2, column = j + (c ^ turn);
+      const float* at = state + static_cast<size_t>(d) * s.vdim + col0 + column;
+      const bool mine = column < cols_here;
+      S[c][p] = pack2(mine && d < s.dim ? at[0] : 0.f, mine && d + 1 < s.dim ? at[s.vdim] : 0.f);
     }
-  }
+  const int pitch = Dp / 4;
   for (int block = 0; block < blocks; ++block) {
     asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
     __syncthreads();   // the block's record is there, and everyone is done with the stage that is filled next
     stage(block + STAGES - 1);
     const float* at = blocks_shared + (block % STAGES) * stage_floats;
-    const ulonglong2* rows = reinterpret_cast<const ulonglong2*>(at) + g;   // row r: + r * Dp / 4; chunk: + LANES
-    const int pitch = Dp / 4;
+    const ulonglong2* rows = reinterpret_cast<const ulonglong2*>(at) + g;   // row r: + r * pitch; chunk: + LANES
     const float* v = at + a.record;
-    float sum[2][N];   // a_t, then c_t, of this thread's rows; t * C + c
+    float sum[2][N];   // a_t, then c_t, of this thread's rows: [column][token]
 #pragma unroll
     for (int which = 0; which < 2; ++which) {
 #pragma unroll
@@ -712,15 +709,24 @@ __global__ void __launch_bounds__(128) delta_blocks_kernel(const BlockArgs a) {
 #pragma unroll
         for (int c = 0; c < C; ++c) {
           const float2 f = unpack2(acc[c]);
-          sum[which][t * C + c] = f.x + f.y;
+          sum[which][c * BLOCK + t] = f.x + f.y;
         }
       }
-      FoldLanes<N, LANES / 2>::run(sum[which], lane);
-      // this lane holds the sums g * OWN .. of its team's N; d_t = v_t - a_t
 #pragma unroll
-      for (int i = 0; i < OWN; ++i) {
-        const int at_value = g * OWN + i, t = at_value / C, c = at_value % C;
-        team_values[which * N + at_value] = which == 0 ? v[t * cols + j + c] - sum[0][i] : sum[1][i];
+      for (int half = N / 2, offset = LANES / 2; half >= OWN_COLUMNS * BLOCK && offset > 0; half /= 2, offset /= 2)
+#pragma unroll
+        for (int i = 0; i < half; ++i) sum[which][i] += __shfl_xor_sync(0xffffffffu, sum[which][i + half], offset);
+      // this lane holds its columns' sums, shared with TOKEN_LANES - 1 others: d_t = v_t - a_t of its own tokens
+#pragma unroll
+      for (int i = 0; i < OWN_COLUMNS; ++i) {
+        FoldLanes<BLOCK, TOKEN_LANES / 2>::run(sum[which] + i * BLOCK, lane);
+        const int c = turn + i;
+#pragma unroll
+        for (int k = 0; k < OWN_TOKENS; ++k) {
+          const int t = g % TOKEN_LANES * OWN_TOKENS + k;
+          const float total = sum[which][i * BLOCK + k];
+          team_values[which * N + c * BLOCK + t] = which == 0 ? v[t * cols + j + c] - total : total;
+        }
       }
     }
     __syncwarp();
@@ -734,10 +740,19 @@ __global__ void __launch_bounds__(128) delta_blocks_kernel(const BlockArgs a) {
         S[c][2 * chunk + 1] = mul2(S[c][2 * chunk + 1], x.y);
       }
     }
+    float d[C][BLOCK];
+#pragma unroll
+    for (int c = 0; c < C; ++c)
+#pragma unroll
+      for (int t = 0; t < BLOCK; t += 4) {
+        const float4 four = *reinterpret_cast<const float4*>(team_values + (c ^ turn) * BLOCK + t);
+        d[c][t] = four.x; d[c][t + 1] = four.y; d[c][t + 2] = four.z; d[c][t + 3] = four.w;
+      }
 #pragma unroll
     for (int t = 0; t < BLOCK; ++t) {
-      const float4 d = *reinterpret_cast<const float4*>(team_values + t * C);
-      const unsigned long long dd[C] = {pack2(d.x, d.x), pack2(d.y, d.y), pack2(d.z, d.z), pack2(d.w, d.w)};
+      unsigned long long dd[C];
+#pragma unroll
+      for (int c = 0; c < C; ++c) dd[c] = pack2(d[c][t], d[c][t]);
 #pragma unroll
       for (int chunk = 0; chunk < CHUNKS; ++chunk) {
         const ulonglong2 x = rows[(2 * BLOCK + t) * pitch + chunk * LANES];
@@ -754,14 +769,15 @@ __global__ void __launch_bounds__(128) delta_blocks_kernel(const BlockArgs a) {
     for (int i = 0; i < (N + LANES - 1) / LANES; ++i) {
       const int at_value = g + i * LANES, t = at_value / C, c = at_value % C;
       if (at_value < N && t < here && j + c < cols_here) {
-        float o = team_values[N + at_value];
+        float o = team_values[N + c * BLOCK + t];
 #pragma unroll
         for (int r = 0; r < BLOCK; r += 4) {
           const float4 row = *reinterpret_cast<const float4*>(m + t * BLOCK + r);
-          o = __fmaf_rn(row.x, team_values[r * C + c], o);
-          o = __fmaf_rn(row.y, team_values[(r + 1) * C + c], o);
-          o = __fmaf_rn(row.z, team_values[(r + 2) * C + c], o);
-          o = __fmaf_rn(row.w, team_values[(r + 3) * C + c], o);
+          const float4 four = *reinterpret_cast<const float4*>(team_values + c * BLOCK + r);
+          o = __fmaf_rn(row.x, four.x, o);
+          o = __fmaf_rn(row.y, four.y, o);
+          o = __fmaf_rn(row.z, four.z, o);
+          o = __fmaf_rn(row.w, four.w, o);
         }
         out[static_cast<size_t>(block * BLOCK + t) * out_width + j + c] = o;
       }
@@ -770,27 +786,17 @@ __global__ void __launch_bounds__(128) delta_blocks_kernel(const BlockArgs a) {
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
 #pragma unroll
-  for (int p = 0; p < PAIRS; ++p) {
-    float2 row[C];
+  for (int p = 0; p < PAIRS; ++p)
 #pragma unroll
-    for (int c = 0; c < C; ++c) row[c] = unpack2(S[c][p]);
-#pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      const int d = (p / 2) * 4 * LANES + 4 * g + (p & 1) * 2 + h;
-      if (d >= s.dim) continue;
-      float* at = state + static_cast<size_t>(d) * s.vdim + col0 + j;
-      float four[C];
-#pragma unroll
-      for (int c = 0; c < C; ++c) four[c] = h == 0 ? row[c].x : row[c].y;
-      if (wide) {
-        if (j < cols_here) store4<float>(at, four);
-      } else {
-#pragma unroll
-        for (int c = 0; c < C; ++c)
-          if (j + c < cols_here) at[c] = four[c];
+    for (int c = 0; c < C; ++c) {
+      const int d = (p / 2) * 4 * LANES + 4 * g + (p & 1) * 2, column = j + (c ^ turn);
+      float* at = state + static_cast<size_t>(d) * s.vdim + col0 + column;
+      const float2 two = unpack2(S[c][p]);
+      if (column < cols_here) {
+        if (d < s.dim) at[0] = two.x;
+        if (d + 1 < s.dim) at[s.vdim] = two.y;
       }
     }
-  }
 }
 
 }  // namespace delta
@@ -904,24 +910,43 @@ SHRIKE_API int shrike_delta_scan(const float* mixed, const float* beta, const fl
     b.padded_dim = shape.lanes * shape.rows;
     b.record = record_floats(b.padded_dim);
     b.num_seqs = num_seqs; b.from = from; b.blocks = blocks;
+    // Four rows a thread where the walks are few (twice the warps hide each other's waits), eight where there are enough
+    // of them (half the adding up over lanes); a head of more than 128 rows takes eight.
+    const int sms = shrike_device().sm_count;
+    const long long quarters = static_cast<long long>((vdim + 31) / 32) * min(head_count, heads) * num_seqs;   // CTAs of 32 columns
+    const int chunks = b.padded_dim > 128 || quarters > 2 * sms ? 2 : 1;
+    const int lanes = b.padded_dim / (4 * chunks);
+    const int per_warp = 32 / lanes * 4;
+    const int warps = max(1, min(chunks == 2 ? 4 : 8, (vdim + per_warp - 1) / per_warp));
+    b.s.cols = per_warp * warps;
+    const unsigned block_slices = static_cast<unsigned>((vdim + b.s.cols - 1) / b.s.cols);
     void (*kernel)(BlockArgs) = nullptr;
-    switch (shape.lanes) {
-      case 1: kernel = delta_blocks_kernel<1>; break;
-      case 2: kernel = delta_blocks_kernel<2>; break;
-      case 4: kernel = delta_blocks_kernel<4>; break;
-      case 8: kernel = delta_blocks_kernel<8>; break;
-      case 16: kernel = delta_blocks_kernel<16>; break;
-      default: kernel = delta_blocks_kernel<32>; break;
+#define SHRIKE_DELTA_BLOCKS(L) kernel = chunks == 2 ? delta_blocks_kernel<L, 2> : delta_blocks_kernel<L, 1>
+    switch (lanes) {
+      case 1: SHRIKE_DELTA_BLOCKS(1); break;
+      case 2: SHRIKE_DELTA_BLOCKS(2); break;
+      case 4: SHRIKE_DELTA_BLOCKS(4); break;
+      case 8: SHRIKE_DELTA_BLOCKS(8); break;
+      case 16: SHRIKE_DELTA_BLOCKS(16); break;
+      default: SHRIKE_DELTA_BLOCKS(32); break;
     }
-    const int teams = shape.threads / shape.lanes;
-    const size_t smem = (static_cast<size_t>(STAGES) * (b.record + BLOCK * shape.cols) + static_cast<size_t>(teams) * 2 * BLOCK * 4) * sizeof(float);
-    if (smem > static_cast<size_t>(shrike_device().max_smem)) return SHRIKE_BAD_ARGUMENT;
+#undef SHRIKE_DELTA_BLOCKS
+    const int teams = warps * 32 / lanes;
+    size_t smem = (static_cast<size_t>(STAGES) * (b.record + BLOCK * b.s.cols) + static_cast<size_t>(teams) * 2 * BLOCK * 4) * sizeof(float);
+    const size_t most = static_cast<size_t>(shrike_device().max_smem);
+    if (smem > most) return SHRIKE_BAD_ARGUMENT;
+    // The walk's CTAs are few and run long: each asks for so much shared memory that they spread evenly over the SMs
+    // instead of being packed where there is room first.
+    const long long ctas = static_cast<long long>(block_slices) * min(head_count, heads) * num_seqs;
+    const long long per_sm = (ctas + sms - 1) / sms;
+    const size_t fair = most / static_cast<size_t>(per_sm) - 2048;
+    if (per_sm <= 8 && fair > smem) smem = fair;
     if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
     for (int head0 = 0; head0 < heads; head0 += head_count) {
       b.head0 = head0;
       b.head_count = min(head_count, heads - head0);
       launch_dependent(delta_local_kernel, dim3(static_cast<unsigned>(blocks), static_cast<unsigned>((b.head_count + 3) / 4)), 128, 0, stream, b);
-      launch_dependent(kernel, dim3(slices, b.head_count, num_seqs), static_cast<unsigned>(shape.threads), smem, stream, b);
+      launch_dependent(kernel, dim3(block_slices, b.head_count, num_seqs), static_cast<unsigned>(warps * 32), smem, stream, b);
     }
   }
   return shrike_launch_status();
