@@ -234,6 +234,7 @@ struct ScanArgs {
   int heads, kv_heads, dim, vdim, channels, head_stride, num_slots;
   int lanes, cols;        // lanes of a warp that share a thread's columns; columns of a CTA
   int skip_from;          // > 0: sequences that bring at least so many tokens are served elsewhere
+  int early_state;        // 1: no kernel still running writes the states: they are read before the wait
 };
 
 // One CTA owns `cols` value columns of one head's state for one sequence and walks its tokens in order with the state in
@@ -245,7 +246,7 @@ template <int R, int C>
 __global__ void __launch_bounds__(128, 4) delta_walk_kernel(const ScanArgs a) {
   extern __shared__ __align__(16) float delta_shared[];
   let_dependents_start();
-  wait_for_previous();
+  if (!a.early_state) wait_for_previous();
   const int D = a.dim, lanes = a.lanes, cols = a.cols;
   constexpr int PITCH = R + 4;
   const int padded = lanes * PITCH;
@@ -260,10 +261,14 @@ __global__ void __launch_bounds__(128, 4) delta_walk_kernel(const ScanArgs a) {
   const int head = blockIdx.y, seq = blockIdx.z, col0 = blockIdx.x * cols;
   const int cols_here = min(cols, a.vdim - col0);
   const int first = a.q_start[seq], length = a.q_start[seq + 1] - first;
-  if (a.skip_from > 0 && length >= a.skip_from) return;
+  if (a.skip_from > 0 && length >= a.skip_from) {
+    if (a.early_state) wait_for_previous();   // every CTA waits before it leaves
+    return;
+  }
   const int slot = a.state_slot[seq];
   const size_t out_width = static_cast<size_t>(a.heads) * a.vdim;
   if (slot < 0 || slot >= a.num_slots) {   // a padding row: zeros out, nothing kept
+    if (a.early_state) wait_for_previous();
     if (g == 0)
       for (int t = 0; t < length; ++t)
 #pragma unroll
@@ -290,6 +295,7 @@ __global__ void __launch_bounds__(128, 4) delta_walk_kernel(const ScanArgs a) {
 #pragma unroll
     for (int c = 0; c < C; ++c) S[c][r] = d < D && j + c < cols_here ? at[c] : 0.f;
   }
+  if (a.early_state) wait_for_previous();
   // rows past the head's own are zero in q, k and the decays: the state's rows there stay zero
   const int extra = lanes * R - D;
   for (int i = threadIdx.x; i < STAGED * extra; i += blockDim.x) {
@@ -880,12 +886,13 @@ SHRIKE_API int shrike_delta_scan_block() { return BLOCK; }
 
 // Sequences that bring at least `from` tokens (0: none) run in blocks, for which the caller holds `records`
 // (blocks x head_count x shrike_delta_scan_record floats, `blocks` = the sum of ceil(length / BLOCK) over them); heads are
-// then served `head_count` at a time.  `shorter`: whether the batch has sequences below `from`.
+// then served `head_count` at a time.  `early_state` 1: the caller knows that whatever kernel wrote the states has finished
+// (an earlier step, not merely an earlier launch), so that the walk may read them while the kernel before it runs.  `shorter`: whether the batch has sequences below `from`.
 SHRIKE_API int shrike_delta_scan(const float* mixed, const float* beta, const float* gates, int partials, long long stride,
                                  int gate_width, const float* rate, const float* bias, float* state, const int* q_start,
                                  const int* state_slot, float* out, int num_seqs, int heads, int kv_heads, int dim, int vdim,
                                  int head_stride, int num_slots, int from, int shorter, float* records, int blocks,
-                                 int head_count, cudaStream_t stream) {
+                                 int head_count, int early_state, cudaStream_t stream) {
   if (num_seqs <= 0) return SHRIKE_OK;
   if (heads < 1 || heads > 65535 || num_seqs > 65535 || kv_heads < 1 || heads % kv_heads || dim < 1 || vdim < 1 || partials < 1 ||
       head_stride < dim * vdim || gate_width < heads * dim)
@@ -894,7 +901,7 @@ SHRIKE_API int shrike_delta_scan(const float* mixed, const float* beta, const fl
   DeltaShape shape;
   if (!delta_shape(dim, vdim, &shape)) return SHRIKE_BAD_ARGUMENT;   // heads of more than 1,024 rows
   ScanArgs a = {mixed, beta, gates, stride, partials, gate_width, rate, bias, state, q_start, state_slot, out,
-                heads, kv_heads, dim, vdim, 2 * kv_heads * dim + heads * vdim, head_stride, num_slots, shape.lanes, shape.cols, 0};
+                heads, kv_heads, dim, vdim, 2 * kv_heads * dim + heads * vdim, head_stride, num_slots, shape.lanes, shape.cols, 0, early_state};
   const bool in_blocks = from > 0 && records != nullptr && blocks > 0 && head_count > 0 && shape.rows == 8;
   const unsigned slices = static_cast<unsigned>((vdim + shape.cols - 1) / shape.cols);
   if (!in_blocks || shorter) {

@@ -190,7 +190,7 @@ class CudaOps:
         lib.shrike_side_gate.argtypes = [_P, _I, _LL, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _P, _I, _P]
         lib.shrike_short_conv_keep.argtypes = [_P, _I, _LL, _I, _P, _P, _P, _I, _I, _I, _I, _P]
         lib.shrike_delta_prep.argtypes = [_P, _I, _LL, _I, _P, _P, _P, _P, _P, _P, _P, _P] + [_I] * 12 + [_F, _F, _I, _P]
-        lib.shrike_delta_scan.argtypes = [_P, _P, _P, _I, _LL, _I, _P, _P, _P, _P, _P, _P] + [_I] * 9 + [_P, _I, _I, _P]
+        lib.shrike_delta_scan.argtypes = [_P, _P, _P, _I, _LL, _I, _P, _P, _P, _P, _P, _P] + [_I] * 9 + [_P, _I, _I, _I, _P]
         lib.shrike_delta_scan_record.argtypes = [_I]
         lib.shrike_delta_scan_record.restype = _I
         lib.shrike_delta_scan_block.restype = _I
@@ -1194,14 +1194,15 @@ class CudaOps:
     DELTA_SCRATCH_FLOATS = 64 << 20   # at most 256 MiB of what the blocks hand to the walk: heads take turns beyond
 
     def delta_scan(self, mixed, beta, gates, rate, bias, state, q_start, state_slot, out, num_seqs, num_heads, num_kv_heads,
-                   dim, vdim, q_lens=None):
+                   dim, vdim, q_lens=None, early_state=False):
         """The delta rule over the batch's new tokens, per value head h with q/k head h // (H / G) of `mixed` (as
         `delta_prep` leaves it): S <- diag(g) S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q, with g =
         exp(-rate[h] softplus(z + bias)), z column h dim + d of `gates` ([N, at least H dim] float32 or a K-split stack).
         `state` float32 [slots, H, at least dim * vdim, a multiple of four] is read and left updated for the slots
         `state_slot` names (-1: zeros out, nothing kept); `out` float32 [N, H * vdim].  `q_lens` (the batch's lengths, host):
         longer portions go eight tokens at a time, with the same result up to the order of the sums; without it every
-        sequence walks token by token."""
+        sequence walks token by token.  `early_state`: the states were last written by an earlier step (whose kernels have
+        finished), not merely by an earlier launch; single tokens then read them while the kernel before this one runs."""
         for name, tensor in (("q, k and v", mixed), ("beta", beta), ("gates", gates), ("rate", rate), ("bias", bias),
                              ("state", state), ("scan output", out)):
             _dense(tensor, torch.float32, name)
@@ -1226,7 +1227,7 @@ class CudaOps:
             _ptr(mixed), _ptr(beta), _ptr(gates), partials, stride, gates.shape[-1], _ptr(rate), _ptr(bias), _ptr(state),
             _ptr(q_start), _ptr(state_slot), _ptr(out), num_seqs, num_heads, num_kv_heads, dim, vdim, state.shape[2],
             state.shape[0], self.DELTA_BLOCKS_FROM if blocks else 0, int(shorter), _ptr(records), blocks, head_count,
-            self._stream()), "delta_scan")
+            int(bool(early_state)), self._stream()), "delta_scan")
 
     def sample(self, logits, temperature, top_p, seeds, out):
         _dense(logits, torch.float32, "logits")

@@ -125,7 +125,8 @@ class ChannelDelta:
         gates = ops.linear(low, self.w_gates, gates, allow_partials=True)
         scanned = rt.buffer("memory_num", (n, self.out_width), torch.float32)
         ops.delta_scan(mixed, beta, gates, self.rate, self.bias, ctx.storage.state[run.cache], ctx.q_start, ctx.state_slot,
-                       scanned, ctx.num_seqs, spec.num_heads, spec.num_kv_heads, spec.head_dim, spec.value_dim, q_lens=ctx.q_lens)
+                       scanned, ctx.num_seqs, spec.num_heads, spec.num_kv_heads, spec.head_dim, spec.value_dim, q_lens=ctx.q_lens,
+                       early_state=True)   # a run's state is its own: only earlier steps wrote it
         out = rt.buffer("memory_out", (n, self.out_width), rt.act_dtype)
         ops.head_rms(scanned, self.norm_weight, spec.eps, out, spec.num_heads, gate_source=gates, gate_at=self.gate_at)
         delta = rt.buffer("memory_delta", (n, spec.width), torch.float32)

@@ -504,7 +504,7 @@ class EmulatedOps:
         low.copy_(fused[:, low_at: low_at + low.shape[1]].to(low.dtype))
 
     def delta_scan(self, mixed, beta, gates, rate, bias, state, q_start, state_slot, out, num_seqs, num_heads, num_kv_heads,
-                   dim, vdim, q_lens=None):
+                   dim, vdim, q_lens=None, early_state=False):
         if gates.dim() == 3:
             gates = gates.sum(0)
         n, qk, share = mixed.shape[0], num_kv_heads * dim, num_heads // num_kv_heads
