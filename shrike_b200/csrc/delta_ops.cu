@@ -426,7 +426,7 @@ struct BlockArgs {
   int head0, head_count;    // the heads this launch serves
 };
 
-__host__ __device__ __forceinline__ int record_floats(int padded_dim) { return (3 * BLOCK + 1) * padded_dim + BLOCK * BLOCK; }
+__host__ __device__ constexpr int record_floats(int padded_dim) { return (3 * BLOCK + 1) * padded_dim + BLOCK * BLOCK; }
 
 // Blocks of sequence `seq`; a warp sums them over the sequences before one.
 __device__ __forceinline__ int blocks_of(const BlockArgs& a, int seq) {
@@ -624,6 +624,7 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
   constexpr int COLUMN_LANES = LANES >= C ? C : LANES;   // lanes the columns are shared out over, then the tokens
   constexpr int TOKEN_LANES = LANES / COLUMN_LANES;
   constexpr int OWN_COLUMNS = C / COLUMN_LANES, OWN_TOKENS = BLOCK / TOKEN_LANES;
+  constexpr int Dp = 4 * LANES * CHUNKS, RECORD = record_floats(Dp), PITCH = LANES * CHUNKS;
   const ScanArgs& s = a.s;
   let_dependents_start();
   wait_for_previous();
@@ -646,25 +647,30 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
   for (int other = lane; other < seq; other += 32) base += blocks_of(a, other);
 #pragma unroll
   for (int offset = 16; offset > 0; offset >>= 1) base += __shfl_xor_sync(0xffffffffu, base, offset);
-  const int Dp = a.padded_dim;
   const int blocks = (length + BLOCK - 1) / BLOCK;
-  const int stage_floats = a.record + BLOCK * cols;
+  const int stage_floats = RECORD + BLOCK * cols;
   float* team_values = blocks_shared + STAGES * stage_floats + (warp * (32 / LANES) + team) * 2 * N;   // d, then c, of this team's columns
   const int v_col = 2 * s.kv_heads * s.dim + head * s.vdim + col0;
   const bool wide_v = ((v_col | s.channels | s.vdim) & 3) == 0 && (reinterpret_cast<uintptr_t>(s.mixed) & 15) == 0;
+  // a thread's 16-byte piece of the CTA's columns of v, the same in every block (narrow heads have more pieces than threads)
+  const int pieces = BLOCK * cols / 4, piece_t = static_cast<int>(threadIdx.x) / (cols / 4), piece_c = (static_cast<int>(threadIdx.x) - piece_t * (cols / 4)) * 4;
+  const bool one_piece = wide_v && pieces <= static_cast<int>(blockDim.x);
+  const float* next_record = a.records + (static_cast<size_t>(base) * a.head_count + local_head) * RECORD + threadIdx.x * 4;
+  const size_t record_step = static_cast<size_t>(a.head_count) * RECORD;
+  int fill = 0;   // the stage that is filled next
   const auto stage = [&](int block) {   // asks for a block's record and the CTA's columns of v
     if (block < blocks) {
-      float* at = blocks_shared + (block % STAGES) * stage_floats;
-      const float* record = a.records + (static_cast<size_t>(base + block) * a.head_count + local_head) * a.record;
-      for (int i = threadIdx.x * 4; i < a.record; i += blockDim.x * 4) copy16(at + i, record + i);
-      float* v = at + a.record;
+      float* at = blocks_shared + fill * stage_floats;
+#pragma unroll 4
+      for (int i = threadIdx.x * 4, k = 0; i < RECORD; i += blockDim.x * 4, k += blockDim.x * 4) copy16(at + i, next_record + k);
+      next_record += record_step;
+      float* v = at + RECORD;
       const int here = min(BLOCK, length - block * BLOCK);
       const float* from = s.mixed + static_cast<size_t>(first + block * BLOCK) * s.channels + v_col;
-      if (wide_v) {
-        for (int i = threadIdx.x; i < BLOCK * cols / 4; i += blockDim.x) {
-          const int t = i / (cols / 4), c = (i - t * (cols / 4)) * 4;
-          if (t < here && c < cols_here) copy16(v + t * cols + c, from + static_cast<size_t>(t) * s.channels + c);
-          else *reinterpret_cast<float4*>(v + t * cols + c) = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (one_piece) {
+        if (static_cast<int>(threadIdx.x) < pieces) {
+          if (piece_t < here && piece_c < cols_here) copy16(v + piece_t * cols + piece_c, from + static_cast<size_t>(piece_t) * s.channels + piece_c);
+          else *reinterpret_cast<float4*>(v + piece_t * cols + piece_c) = make_float4(0.f, 0.f, 0.f, 0.f);
         }
       } else {
         for (int i = threadIdx.x; i < BLOCK * cols; i += blockDim.x) {
@@ -674,6 +680,7 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
         }
       }
     }
+    fill = fill + 1 == STAGES ? 0 : fill + 1;
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
 #pragma unroll
@@ -689,14 +696,15 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
       const bool mine = column < cols_here;
       S[c][p] = pack2(mine && d < s.dim ? at[0] : 0.f, mine && d + 1 < s.dim ? at[s.vdim] : 0.f);
     }
-  const int pitch = Dp / 4;
+  int taken = 0;   // the stage of the block at hand
   for (int block = 0; block < blocks; ++block) {
     asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
     __syncthreads();   // the block's record is there, and everyone is done with the stage that is filled next
     stage(block + STAGES - 1);
-    const float* at = blocks_shared + (block % STAGES) * stage_floats;
-    const ulonglong2* rows = reinterpret_cast<const ulonglong2*>(at) + g;   // row r: + r * pitch; chunk: + LANES
-    const float* v = at + a.record;
+    const float* at = blocks_shared + taken * stage_floats;
+    taken = taken + 1 == STAGES ? 0 : taken + 1;
+    const ulonglong2* rows = reinterpret_cast<const ulonglong2*>(at) + g;   // row r: + r * PITCH; chunk: + LANES
+    const float* v = at + RECORD;
     float sum[2][N];   // a_t, then c_t, of this thread's rows: [column][token]
 #pragma unroll
     for (int which = 0; which < 2; ++which) {
@@ -705,7 +713,7 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
         unsigned long long acc[C];
 #pragma unroll
         for (int chunk = 0; chunk < CHUNKS; ++chunk) {
-          const ulonglong2 x = rows[(which * BLOCK + t) * pitch + chunk * LANES];
+          const ulonglong2 x = rows[(which * BLOCK + t) * PITCH + chunk * LANES];
 #pragma unroll
           for (int c = 0; c < C; ++c) {
             acc[c] = chunk == 0 ? mul2(S[c][0], x.x) : fma2(S[c][2 * chunk], x.x, acc[c]);
@@ -718,21 +726,24 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
           sum[which][c * BLOCK + t] = f.x + f.y;
         }
       }
+    }
 #pragma unroll
-      for (int half = N / 2, offset = LANES / 2; half >= OWN_COLUMNS * BLOCK && offset > 0; half /= 2, offset /= 2)
+    for (int half = N / 2, offset = LANES / 2; half >= OWN_COLUMNS * BLOCK && offset > 0; half /= 2, offset /= 2)
 #pragma unroll
-        for (int i = 0; i < half; ++i) sum[which][i] += __shfl_xor_sync(0xffffffffu, sum[which][i + half], offset);
-      // this lane holds its columns' sums, shared with TOKEN_LANES - 1 others: d_t = v_t - a_t of its own tokens
+      for (int i = 0; i < half; ++i)
 #pragma unroll
-      for (int i = 0; i < OWN_COLUMNS; ++i) {
-        FoldLanes<BLOCK, TOKEN_LANES / 2>::run(sum[which] + i * BLOCK, lane);
-        const int c = turn + i;
+        for (int which = 0; which < 2; ++which) sum[which][i] += __shfl_xor_sync(0xffffffffu, sum[which][i + half], offset);
+    // this lane holds its columns' sums, shared with TOKEN_LANES - 1 others: d_t = v_t - a_t of its own tokens
 #pragma unroll
-        for (int k = 0; k < OWN_TOKENS; ++k) {
-          const int t = g % TOKEN_LANES * OWN_TOKENS + k;
-          const float total = sum[which][i * BLOCK + k];
-          team_values[which * N + c * BLOCK + t] = which == 0 ? v[t * cols + j + c] - total : total;
-        }
+    for (int i = 0; i < OWN_COLUMNS; ++i) {
+      FoldLanes<BLOCK, TOKEN_LANES / 2>::run(sum[0] + i * BLOCK, lane);
+      FoldLanes<BLOCK, TOKEN_LANES / 2>::run(sum[1] + i * BLOCK, lane);
+      const int c = turn + i;
+#pragma unroll
+      for (int k = 0; k < OWN_TOKENS; ++k) {
+        const int t = g % TOKEN_LANES * OWN_TOKENS + k;
+        team_values[c * BLOCK + t] = v[t * cols + j + c] - sum[0][i * BLOCK + k];
+        team_values[N + c * BLOCK + t] = sum[1][i * BLOCK + k];
       }
     }
     __syncwarp();
@@ -761,7 +772,7 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
       for (int c = 0; c < C; ++c) dd[c] = pack2(d[c][t], d[c][t]);
 #pragma unroll
       for (int chunk = 0; chunk < CHUNKS; ++chunk) {
-        const ulonglong2 x = rows[(2 * BLOCK + t) * pitch + chunk * LANES];
+        const ulonglong2 x = rows[(2 * BLOCK + t) * PITCH + chunk * LANES];
 #pragma unroll
         for (int c = 0; c < C; ++c) {
           S[c][2 * chunk] = fma2(x.x, dd[c], S[c][2 * chunk]);
@@ -924,7 +935,11 @@ SHRIKE_API int shrike_delta_scan(const float* mixed, const float* beta, const fl
     const int chunks = b.padded_dim > 128 || quarters > 2 * sms ? 2 : 1;
     const int lanes = b.padded_dim / (4 * chunks);
     const int per_warp = 32 / lanes * 4;
-    const int warps = max(1, min(chunks == 2 ? 4 : 8, (vdim + per_warp - 1) / per_warp));
+    int warps = max(1, min(chunks == 2 ? 4 : 8, (vdim + per_warp - 1) / per_warp));
+    // few heads: narrower CTAs, as many as there are SMs for
+    while (warps > 2 && warps % 2 == 0 &&
+           static_cast<long long>((vdim + per_warp * warps - 1) / (per_warp * warps)) * min(head_count, heads) * num_seqs * 2 <= sms)
+      warps /= 2;
     b.s.cols = per_warp * warps;
     const unsigned block_slices = static_cast<unsigned>((vdim + b.s.cols - 1) / b.s.cols);
     void (*kernel)(BlockArgs) = nullptr;
