@@ -1191,7 +1191,7 @@ class CudaOps:
             self._stream()), "delta_prep")
 
     DELTA_BLOCKS_FROM = 16            # a sequence that brings at least this many tokens goes eight tokens at a time
-    DELTA_SCRATCH_FLOATS = 64 << 20   # at most 256 MiB of what the blocks hand to the walk: heads take turns beyond
+    DELTA_SCRATCH_FLOATS = 128 << 20   # at most 512 MiB of what the blocks hand to the walk: heads take turns beyond
 
     def delta_scan(self, mixed, beta, gates, rate, bias, state, q_start, state_slot, out, num_seqs, num_heads, num_kv_heads,
                    dim, vdim, q_lens=None, early_state=False):
