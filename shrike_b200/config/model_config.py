@@ -199,6 +199,8 @@ class GatedHeadAttentionSpec(PartSpec):
     softcap: float | None = None
     # `keep_first` n (with a window): the sequence's first n keys stay visible to every later query
     keep_first: int = 0
+    # `element_gate`: the heads' outputs, side by side, are multiplied element by element by sigmoid(Wg x)
+    element_gate: bool = False
     # `own_kv` False: the layer has no key and value projections and attends over the keys and values another
     # layer cached (the run order says whose)
     own_kv: bool = True
@@ -209,6 +211,8 @@ class GatedHeadAttentionSpec(PartSpec):
             raise ConfigError(f"heads={self.num_heads} is not a multiple of kv_heads={self.num_kv_heads}")
         if self.window is not None and self.chunk is not None:
             raise ConfigError("an attention layer has a window or a chunk, not both")
+        if self.head_gate and self.element_gate:
+            raise ConfigError("an attention layer has a gate a head or a gate an element, not both")
         if self.qk_norm not in (False, True, "whole"):
             raise ConfigError(f"qk_norm {self.qk_norm!r}; known: False, True (per head), 'whole'")
         if self.conv is not None and not 1 <= self.conv <= 32:
@@ -374,6 +378,54 @@ class ChannelDeltaSpec(PartSpec):
 
 
 @dataclass(frozen=True)
+class HeadDeltaSpec(PartSpec):
+    """A delta rule with one decay a head (the gated delta rule).  Projections, convolutions, unit vectors and the
+    recurrence are `ChannelDeltaSpec`'s, with g = exp(-exp(A_log) softplus(Wa x + dt_bias)) one number a head (Wa one row
+    a head), and every head's normed output is multiplied by silu(Wg x), Wg of full rank, one number an element."""
+
+    width: int
+    num_heads: int
+    num_kv_heads: int
+    head_dim: int
+    value_dim: int
+    conv: int
+    eps: float
+    unit_eps: float = 1e-6
+    kind: str = field(init=False, default="head_delta")
+
+    def __post_init__(self):
+        if self.num_heads % self.num_kv_heads:
+            raise ConfigError(f"heads={self.num_heads} is not a multiple of kv_heads={self.num_kv_heads}")
+        if not 1 <= self.conv <= 32:
+            raise ConfigError(f"a short convolution has 1 to 32 taps, got {self.conv}")
+
+
+@dataclass(frozen=True)
+class GatedLinearAttentionSpec(PartSpec):
+    """Linear attention whose state decays per key channel by a gate of the token's own.  Per head, from S = 0,
+
+        S_t = diag(a_t) S_(t-1) + k_t v_t^T;   o_t = S_t^T q_t;   a = sigmoid(Wa2 (Wa1 x) + b)^(1/tau) per key channel
+
+    with q = head_dim^(-1/2) Wq x, k = Wk x, v = Wv x.  Every head's o is divided by its root mean square, scaled by one
+    weight of the head's size that all heads share, multiplied by silu(Wg x) and projected.  `decay_rank`, the rows of
+    Wa1, is what a model's tensors say (None); a number here is used for random weights.  Gates, state and recurrence are
+    32-bit."""
+
+    width: int
+    num_heads: int
+    head_dim: int
+    value_dim: int
+    tau: float
+    eps: float
+    decay_rank: int | None = None
+    kind: str = field(init=False, default="gated_linear_attention")
+
+    def __post_init__(self):
+        if not self.tau > 0:
+            raise ConfigError(f"tau must be positive, got {self.tau}")
+
+
+@dataclass(frozen=True)
 class HyperConnectionSpec(PartSpec):
     """How a sublayer's result y joins a residual of `streams` streams x_1 .. x_S, and how the sublayer reads them:
     u = sum_s in[s] x_s is what the sublayer's norm sees; afterwards, all streams at once from the old ones,
@@ -461,7 +513,8 @@ class GatedMLPSpec(PartSpec):
 
 @dataclass(frozen=True)
 class MLPSpec(PartSpec):
-    """Dense feed-forward without a gate: down(act(up(x))).  `activation` "relu2": the square of relu."""
+    """Dense feed-forward without a gate: down(act(up(x))).  `activation` "relu2": the square of relu; "gelu": z (1 + erf(z /
+    sqrt(2))) / 2."""
 
     width: int
     intermediate: int
@@ -496,14 +549,27 @@ class RoutedExpertsSpec(PartSpec):
     shared_limit: float | None = None
     # `correction`: a learned number per expert is added to the scores for the choice; the weights are without it
     correction: bool = False
+    # `gated` False: an expert is down(act(up x)), without a gate (the activations of `MLPSpec`)
+    gated: bool = True
+    # `identity` n: the router has n more outputs behind the experts'; an identity expert's output is the input itself, and
+    # it takes part in scores, choice and weights like the others
+    identity: int = 0
     # `groups` (count, keep): the experts form `count` equal groups of neighbours, a group counts as much as its best
     # expert, and only experts of the best `keep` groups can be chosen
     groups: tuple | None = None
     kind: str = field(init=False, default="routed_experts")
 
     def __post_init__(self):
-        if not 1 <= self.top <= self.experts:
-            raise ConfigError(f"router: top={self.top} must lie in 1..experts={self.experts}")
+        if self.identity < 0:
+            raise ConfigError(f"router: identity={self.identity} must not be negative")
+        if not 1 <= self.top <= self.experts + self.identity:
+            raise ConfigError(f"router: top={self.top} must lie in 1..{self.experts + self.identity}, the router's outputs")
+        if (self.identity or not self.gated) and self.weight_on != "output":
+            raise ConfigError("identity experts and experts without a gate carry their weight on the output")
+        if not self.gated and self.shared_intermediate is not None:
+            raise ConfigError("a shared expert beside experts without a gate is not served")
+        if self.identity and self.groups is not None:
+            raise ConfigError("identity experts do not form groups")
         if self.scoring not in ("softmax", "sigmoid"):
             raise ConfigError(f"router scoring {self.scoring!r}; known: softmax, sigmoid")
         if self.weight_on not in ("output", "input"):
@@ -610,6 +676,7 @@ class LayerSpec:
     feed_forward_norm: PartSpec | None
     block: str = "pre_norm"
     extra: tuple = ()
+    block_options: tuple = ()   # (name, value): constants the block takes besides its parts
 
     def roles(self):
         """(role, category, spec) of every part of the layer; a part the layer leaves out (None, where

@@ -5,12 +5,15 @@
 //                  out = norm(resid[rows]) for a few gathered rows; RMS or layer norm, bias optional
 //   norm_join      resid += norm(branch) (+ a row), then out = norm(resid): the norm on one sublayer's output and
 //                  the norm before the next one from one pass over the row; also on gathered rows
+//   sum_norm       resid += scale * term over up to four pending sums (+ rows of the activation type, a factor each), then
+//                  out = norm(resid): the norm of a block whose branches run side by side; also on gathered rows
 //   qk_norm_store  queries and keys of a fused q|k projection: RMS over the whole projection (all
 //                  heads at once), a position-dependent query temperature, keys into the key pages
 //                  and the keys as projected into the value pages
 //   latent_store   queries, latent and gate of a fused q|latent|gate projection: queries cast,
 //                  the latent RMS-normed into its (one-plane) pages, the gate through a sigmoid
 //   head_scale     x[token, head, :] *= gate[token, head]
+//   element_gate   x[token, head, i] *= sigmoid of the gate's own column of a fused projection
 //
 // Statistics, temperature, sigmoid and the residual sum are float32; a result is rounded once, when
 // it is stored in the activation type.  Inputs that a K-split product left as a stack of partial
@@ -341,6 +344,134 @@ static int launch_norm_join(float* resid, const float* branch, int partials, lon
   return SHRIKE_OK;
 }
 
+// ------------------------------------------------------------ several pending sums, then a norm
+// A pending sum is cut into its slices (the partial sums a K-split product leaves): the kernel adds slice after slice, each
+// times its sum's scale, up to eight loads of a group in flight.
+constexpr int MAX_SLICES = 64;
+
+struct SumNormArgs {
+  float* resid;                      // [*][width]
+  const float* slices[MAX_SLICES];   // each [*][width]
+  float scales[MAX_SLICES];
+  int num_slices;
+  const void* rows_in;               // [*][width] in the activation type, or null: added times row_weight[row * row_stride]
+  const float* row_weight;           // (a row whose factor is zero is not read); may be the array `out` writes when no rows
+  int row_stride;                    // are gathered: a thread reads what it later overwrites
+  float row_scale;
+  const int* rows;                   // null: every row, the residual is rewritten; else out[r] for row rows[r]
+  const float* weight;
+  float eps;
+  void* out;
+  int width;
+};
+
+template <typename TO, int VEC, int PT>
+__global__ void __launch_bounds__(PT == 4 ? 256 : 1024, PT == 4 ? 4 : 1) sum_norm_kernel(const __grid_constant__ SumNormArgs a) {
+  __shared__ float scratch[33];
+  constexpr bool EARLY = PT == 1;
+  let_dependents_start();
+  const int groups = a.width / VEC;
+  float early_w[VEC] = {};
+  if (EARLY && threadIdx.x < groups) {   // a parameter of the model: no kernel writes it
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) early_w[e] = a.weight[threadIdx.x * VEC + e];
+  }
+  wait_for_previous();
+  const int out_row = blockIdx.x;
+  const int row = a.rows != nullptr ? a.rows[out_row] : out_row;
+  const size_t base = static_cast<size_t>(row) * a.width;
+  float* x = a.resid + base;
+  TO* y = static_cast<TO*>(a.out) + static_cast<size_t>(out_row) * a.width;
+  const float factor = a.rows_in != nullptr ? a.row_weight[static_cast<size_t>(row) * a.row_stride] : 0.f;
+  float held[PT][VEC];
+  float squares = 0.f;
+#pragma unroll
+  for (int it = 0; it < PT; ++it) {
+    const int g = threadIdx.x + it * blockDim.x;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) held[it][e] = 0.f;
+    if (g < groups) {
+      const size_t at = base + static_cast<size_t>(g) * VEC;
+      if constexpr (VEC == 4) load4<float>(a.resid + at, held[it]);
+      else held[it][0] = a.resid[at];
+      constexpr int AHEAD = EARLY ? 8 : 4;
+      for (int s0 = 0; s0 < a.num_slices; s0 += AHEAD) {
+        float part[AHEAD][VEC];
+#pragma unroll
+        for (int s = 0; s < AHEAD; ++s)
+          if (s0 + s < a.num_slices) {
+            if constexpr (VEC == 4) load4<float>(a.slices[s0 + s] + at, part[s]);
+            else part[s][0] = a.slices[s0 + s][at];
+          }
+#pragma unroll
+        for (int s = 0; s < AHEAD; ++s)
+          if (s0 + s < a.num_slices) {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) held[it][e] = __fmaf_rn(a.scales[s0 + s], part[s][e], held[it][e]);
+          }
+      }
+      if (factor != 0.f) {
+        float own[VEC];
+        const TO* from = static_cast<const TO*>(a.rows_in) + at;
+        if constexpr (VEC == 4) load4<TO>(from, own);
+        else own[0] = to_float(from[0]);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) held[it][e] = __fmaf_rn(a.row_scale, __fmul_rn(factor, own[e]), held[it][e]);
+      }
+      if (a.rows == nullptr) {
+        if constexpr (VEC == 4) store4<float>(x + static_cast<size_t>(g) * 4, held[it]);
+        else x[g] = held[it][0];
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) squares = fmaf(held[it][e], held[it][e], squares);
+    }
+  }
+  const float scale = 1.0f / sqrtf(block_sum(squares, scratch) / static_cast<float>(a.width) + a.eps);
+#pragma unroll
+  for (int it = 0; it < PT; ++it) {
+    const int g = threadIdx.x + it * blockDim.x;
+    if (g < groups) {
+      float w[VEC], r[VEC];
+      if (EARLY) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) w[e] = early_w[e];
+      } else if constexpr (VEC == 4) {
+        load4<float>(a.weight + g * 4, w);
+      } else {
+        w[0] = a.weight[g];
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) r[e] = __fmul_rn(__fmul_rn(held[it][e], scale), w[e]);
+      if constexpr (VEC == 4) store4<TO>(y + g * 4, r);
+      else y[g] = from_float<TO>(r[0]);
+    }
+  }
+}
+
+template <typename TO>
+static int launch_sum_norm(const SumNormArgs& a, int n, cudaStream_t stream) {
+  uintptr_t addresses = reinterpret_cast<uintptr_t>(a.resid) | reinterpret_cast<uintptr_t>(a.weight) |
+                        reinterpret_cast<uintptr_t>(a.out) | reinterpret_cast<uintptr_t>(a.rows_in);
+  for (int s = 0; s < a.num_slices; ++s) addresses |= reinterpret_cast<uintptr_t>(a.slices[s]);
+  const bool vec = a.width % 4 == 0 && addresses % 16 == 0;
+  const int groups = vec ? a.width / 4 : a.width;
+  const bool few = n <= 256 && groups <= 1024;
+  int threads = ((few ? groups : (groups + 3) / 4) + 31) / 32 * 32;
+  threads = threads < 64 ? 64 : (threads > 1024 ? 1024 : threads);
+  if (static_cast<long long>(threads) * MAX_PER_THREAD < groups) return SHRIKE_BAD_ARGUMENT;
+  const bool four = !few && threads <= 256;
+#define SHRIKE_SUM_NORM_CASE(V)                                                                              \
+  do {                                                                                                       \
+    if (few) launch_dependent(sum_norm_kernel<TO, V, 1>, n, threads, 0, stream, a);                          \
+    else if (four) launch_dependent(sum_norm_kernel<TO, V, 4>, n, threads, 0, stream, a);                    \
+    else launch_dependent(sum_norm_kernel<TO, V, MAX_PER_THREAD>, n, threads, 0, stream, a);                 \
+  } while (0)
+  if (vec) SHRIKE_SUM_NORM_CASE(4);
+  else SHRIKE_SUM_NORM_CASE(1);
+#undef SHRIKE_SUM_NORM_CASE
+  return SHRIKE_OK;
+}
+
 // ------------------------------------------------------------ queries and keys of a q|k projection
 // One block per token.  qk [P][n][H * D + G * D] float32.  The keys as projected (before their norm)
 // are the values.  Heads are stored `padded` (>= D) elements apart, the padding zeroed, so that an
@@ -505,6 +636,41 @@ __global__ void head_scale_kernel(T* __restrict__ x, const float* __restrict__ g
   }
 }
 
+// x [n][heads][padded] in place, elements 0 .. vdim - 1 of every head: x *= sigmoid(z), z column gate_at + h vdim + i of the
+// fused projection's row (a stack of partial sums is added up).  A thread takes VEC elements, blockIdx.y the token.
+template <typename T> __device__ __forceinline__ float element_sigmoid(float z);
+template <> __device__ __forceinline__ float element_sigmoid<float>(float z) { return 1.0f / (1.0f + expf(-z)); }
+// (a bfloat16 result keeps 8 bits: the hardware exponential and reciprocal serve)
+template <> __device__ __forceinline__ float element_sigmoid<__nv_bfloat16>(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
+
+template <typename T, int VEC>
+__global__ void element_gate_kernel(T* __restrict__ x, const float* __restrict__ fused, int partials, long long stride, int total,
+                                    int gate_at, int heads, int vdim, int padded, int n) {
+  let_dependents_start();
+  wait_for_previous();
+  const int per_row = heads * vdim / VEC;
+  for (int token = blockIdx.y; token < n; token += gridDim.y) {
+    T* row = x + static_cast<size_t>(token) * heads * padded;
+    const float* gates = fused + static_cast<size_t>(token) * total + gate_at;
+    for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < per_row; i += gridDim.x * blockDim.x) {
+      const int c = i * VEC, h = c / vdim;
+      T* at = row + static_cast<size_t>(h) * padded + (c - h * vdim);
+      float v[VEC], z[VEC];
+      if constexpr (VEC == 4) {
+        sum_partials4(gates + c, stride, partials, z);
+        load4<T>(at, v);
+      } else {
+        z[0] = sum_partials(gates + c, stride, partials);
+        v[0] = to_float(at[0]);
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[e] *= element_sigmoid<T>(z[e]);
+      if constexpr (VEC == 4) store4<T>(at, v);
+      else at[0] = from_float<T>(v[0]);
+    }
+  }
+}
+
 template <typename TD, typename TO>
 static int launch_norm_rows(float* resid, const void* branch, int partials, long long partial_stride, const int* rows,
                             const float* weight, const float* bias, float eps, int layer_norm, void* out, int n, int width,
@@ -665,5 +831,54 @@ SHRIKE_API int shrike_head_scale(void* x, const float* gate, int dtype, int n, i
   else if (dtype == SHRIKE_BF16)
     launch_dependent(head_scale_kernel<__nv_bfloat16>, grid, 256, 0, stream, static_cast<__nv_bfloat16*>(x), gate, heads, dim, n);
   else return SHRIKE_BAD_ARGUMENT;
+  return shrike_launch_status();
+}
+
+// resid += scales[t] * sum of `partials[t]` slices of data[t] (float32, `strides[t]` elements apart) over the `num_terms`
+// (at most four) pending sums; with `rows_in` (activation type [*][width]) also row_scale * row_weight[row * row_stride] times
+// its row; out = norm(resid) * weight.  rows: null, n rows, the residual rewritten; else out[r] for row rows[r].
+SHRIKE_API int shrike_sum_norm(float* resid, const float* const* data, const int* partials, const long long* strides, const float* scales,
+                               int num_terms, const void* rows_in, const float* row_weight, int row_stride, float row_scale,
+                               const int* rows, const float* weight, float eps, void* out, int out_dtype, int n, int width,
+                               cudaStream_t stream) {
+  using namespace branch;
+  if (n <= 0) return SHRIKE_OK;
+  if (width <= 0 || num_terms < 0 || weight == nullptr || out == nullptr) return SHRIKE_BAD_ARGUMENT;
+  if (rows_in != nullptr && row_weight == nullptr) return SHRIKE_BAD_ARGUMENT;
+  SumNormArgs a = {};
+  a.resid = resid;
+  for (int t = 0; t < num_terms; ++t) {
+    if (partials[t] < 1 || a.num_slices + partials[t] > MAX_SLICES) return SHRIKE_BAD_ARGUMENT;
+    for (int p = 0; p < partials[t]; ++p) {
+      a.slices[a.num_slices] = data[t] + p * strides[t];
+      a.scales[a.num_slices++] = scales[t];
+    }
+  }
+  a.rows_in = rows_in; a.row_weight = row_weight; a.row_stride = row_stride; a.row_scale = row_scale;
+  a.rows = rows; a.weight = weight; a.eps = eps; a.out = out; a.width = width;
+  int status;
+  if (out_dtype == SHRIKE_BF16) status = launch_sum_norm<__nv_bfloat16>(a, n, stream);
+  else if (out_dtype == SHRIKE_F32) status = launch_sum_norm<float>(a, n, stream);
+  else return SHRIKE_BAD_ARGUMENT;
+  if (status != SHRIKE_OK) return status;
+  return shrike_launch_status();
+}
+
+// x [n][heads][padded] in the activation type, in place; see the kernel.
+SHRIKE_API int shrike_element_gate(void* x, const float* fused, int partials, long long stride, int total, int gate_at, int dtype, int n,
+                                   int heads, int vdim, int padded, cudaStream_t stream) {
+  using namespace branch;
+  if (n <= 0) return SHRIKE_OK;
+  if (heads < 1 || vdim < 1 || padded < vdim || partials < 1 || gate_at < 0 || gate_at + heads * vdim > total) return SHRIKE_BAD_ARGUMENT;
+  const bool vec = vdim % 4 == 0 && padded % 4 == 0 && total % 4 == 0 && gate_at % 4 == 0 && stride % 4 == 0 &&
+                   (reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(fused)) % 16 == 0;
+  const int per_row = heads * vdim / (vec ? 4 : 1);
+  const dim3 grid(max(1, min(8, (per_row + 255) / 256)), max(1, min(n, 65535)));
+#define SHRIKE_ELEMENT_GATE(T, V) \
+  launch_dependent(element_gate_kernel<T, V>, grid, 256, 0, stream, static_cast<T*>(x), fused, partials, stride, total, gate_at, heads, vdim, padded, n)
+  if (dtype == SHRIKE_F32) { if (vec) SHRIKE_ELEMENT_GATE(float, 4); else SHRIKE_ELEMENT_GATE(float, 1); }
+  else if (dtype == SHRIKE_BF16) { if (vec) SHRIKE_ELEMENT_GATE(__nv_bfloat16, 4); else SHRIKE_ELEMENT_GATE(__nv_bfloat16, 1); }
+  else return SHRIKE_BAD_ARGUMENT;
+#undef SHRIKE_ELEMENT_GATE
   return shrike_launch_status();
 }

@@ -171,12 +171,17 @@ template <typename T> __device__ __forceinline__ float act_times(int act, float 
   return act == SHRIKE_ACT_GELU_TANH ? gelu_tanh_times<T>(g, u) : silu_times<T>(g, u);
 }
 
-// Activations of an ungated feed-forward: relu2 is max(z, 0)^2, formed in float32 and rounded once.
-enum : int { SHRIKE_PLAIN_NONE = 0, SHRIKE_PLAIN_RELU2 = 1 };
+// Activations of an ungated feed-forward, formed in float32 and rounded once: relu2 is max(z, 0)^2, gelu is
+// z (1 + erf(z / sqrt(2))) / 2.
+enum : int { SHRIKE_PLAIN_NONE = 0, SHRIKE_PLAIN_RELU2 = 1, SHRIKE_PLAIN_GELU = 2 };
+__host__ __device__ __forceinline__ bool known_plain_activation(int act) { return act == SHRIKE_PLAIN_RELU2 || act == SHRIKE_PLAIN_GELU; }
+__device__ __forceinline__ float plain_act_value(int act, float z) {
+  if (act == SHRIKE_PLAIN_GELU) return __fmul_rn(0.5f * z, 1.0f + erff(z * 0.70710678118654752f));
+  const float v = fmaxf(z, 0.f);
+  return __fmul_rn(v, v);
+}
 template <typename T> __device__ __forceinline__ T plain_act(int act, T z) {
-  if (act != SHRIKE_PLAIN_RELU2) return z;
-  const float v = fmaxf(to_float(z), 0.f);
-  return from_float<T>(__fmul_rn(v, v));
+  return act == SHRIKE_PLAIN_NONE ? z : from_float<T>(plain_act_value(act, to_float(z)));
 }
 
 // The first key a query at position `last` sees.  span > 0: the `span` latest keys (a sliding window);

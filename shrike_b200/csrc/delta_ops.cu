@@ -1,13 +1,16 @@
-// Kernels of the delta rule whose state decays per key channel.
+// Kernels of recurrences whose state per head is a matrix that decays by a factor per key channel, or per head, and
+// takes in one outer product a token: the delta rule, and linear attention with gated decays.
 //
 //   delta_prep   a fused projection's q, k and v behind a causal convolution over time per channel and a SiLU, q and k
 //                unit vectors per head (q also scaled), beta's sigmoid, and the low-rank rows of decays and output
 //                gates in the engine's type
-//   delta_scan   per head S <- diag(g) S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q over the batch's new tokens,
-//                with g = exp(-rate softplus(z + bias)) from a second product's columns z; the state is read from and
-//                left in the request's slot.  Single tokens and short portions walk token by token with the state in
-//                registers; longer ones go eight tokens at a time (`delta_local`, `delta_blocks`), the same sums in another
-//                order.
+//   delta_scan   per head S <- diag(g) S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q over the batch's new tokens
+//                (without beta: u = v, plain linear attention), with g = exp(-rate softplus(sign (z + bias))) from a
+//                product's columns z, one a key channel or one a head; the state is read from and left in the request's
+//                slot.  Single tokens and short portions walk token by token with the state in registers; longer ones go
+//                eight tokens at a time (`delta_local`, `delta_blocks`), the same sums in another order.
+//   low_rank     z = A r for the rows r that columns of a fused projection hold: the second half of a low-rank product,
+//                in float32 from the projection on
 //
 // Everything that enters the recurrence, and the state, is float32.  A product may come as a stack of K-split partial
 // sums, which are added on the fly.
@@ -220,29 +223,37 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const PrepArgs a) {
 constexpr int STAGED = 8;   // tokens staged at a time: their loads are in flight together
 
 struct ScanArgs {
-  const float* mixed;     // [N][channels]: q (G D) | k (G D) | v (H Dv)
-  const float* beta;      // [N][H]
-  const float* gates;     // [partials][N][gate_width]: z of head h, channel d at column h D + d
+  const float* mixed;     // [mixed_partials][N][pitch]: q (G D) | k (G D) | v (H Dv) | ..
+  long long mixed_stride;
+  int mixed_partials, pitch;
+  const float* beta;      // [N][H]; null: no delta rule, every token adds k v^T
+  const float* gates;     // [partials][N][gate_width]: z of head h, channel d at column gate_at + h D + d, or gate_at + h
   long long stride;
-  int partials, gate_width;
+  int partials, gate_width, gate_at;
   const float* rate;      // [H]
-  const float* bias;      // [H D]
+  const float* bias;      // [H D], or [H]; null: none
+  float sign, q_scale;
   float* state;           // [slots][H][head_stride]: row d, column j of S at d * Dv + j
   const int* q_start;
   const int* state_slot;
   float* out;             // [N][H Dv]
-  int heads, kv_heads, dim, vdim, channels, head_stride, num_slots;
+  int heads, kv_heads, dim, vdim, head_stride, num_slots;
   int lanes, cols;        // lanes of a warp that share a thread's columns; columns of a CTA
   int skip_from;          // > 0: sequences that bring at least so many tokens are served elsewhere
   int early_state;        // 1: no kernel still running writes the states: they are read before the wait
 };
 
+__device__ __forceinline__ float decay_of(const ScanArgs& a, float rate, float z, float bias) {
+  return expf(-rate * softplus(a.sign * (z + bias)));
+}
+
 // One CTA owns `cols` value columns of one head's state for one sequence and walks its tokens in order with the state in
 // registers: a thread holds R rows of C neighbouring columns, `lanes` neighbouring lanes (a power of two covering the
 // head's rows) share those columns and add up by shuffles; no barrier falls inside the walk.  Tokens are staged STAGED
 // at a time: q, k and the decays of the head (a lane's rows side by side, its run padded by four floats so that the
-// lanes' 16-byte loads fall into different banks), the CTA's columns of v, and beta.
-template <int R, int C>
+// lanes' 16-byte loads fall into different banks), the CTA's columns of v, and beta.  DELTA: the delta rule, else every
+// token adds k v^T; HEAD: one decay a head instead of one a key channel.
+template <int R, int C, bool DELTA, bool HEAD>
 __global__ void __launch_bounds__(128, 4) delta_walk_kernel(const ScanArgs a) {
   extern __shared__ __align__(16) float delta_shared[];
   let_dependents_start();
@@ -254,7 +265,7 @@ __global__ void __launch_bounds__(128, 4) delta_walk_kernel(const ScanArgs a) {
   float* k = q + STAGED * padded;
   float* f = k + STAGED * padded;       // decays
   float* v = f + STAGED * padded;       // [STAGED][cols]
-  float* b = v + STAGED * cols;         // [STAGED]
+  float* b = v + STAGED * cols;         // [STAGED]; one decay a head: those at f[0 .. STAGED)
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int g = lane % lanes;
   const int j = (warp * (32 / lanes) + lane / lanes) * C;
@@ -303,7 +314,7 @@ __global__ void __launch_bounds__(128, 4) delta_walk_kernel(const ScanArgs a) {
     const int at = t * padded + (d / R) * PITCH + d % R;
     q[at] = 0.f;
     k[at] = 0.f;
-    f[at] = 0.f;
+    if (!HEAD) f[at] = 0.f;
   }
   const int group = head / (a.heads / a.kv_heads);
   const int q_col = group * D, k_col = (a.kv_heads + group) * D, v_col = 2 * a.kv_heads * D + head * a.vdim + col0;
@@ -313,18 +324,25 @@ __global__ void __launch_bounds__(128, 4) delta_walk_kernel(const ScanArgs a) {
     __syncthreads();   // the tokens staged before are used up
     for (int i = threadIdx.x; i < here * D; i += blockDim.x) {
       const int t = i / D, d = i - t * D;
-      const float* row = a.mixed + static_cast<size_t>(first + t0 + t) * a.channels;
-      const float z = sum_partials(a.gates + static_cast<size_t>(first + t0 + t) * a.gate_width + head * D + d, a.stride, a.partials);
+      const float* row = a.mixed + static_cast<size_t>(first + t0 + t) * a.pitch;
       const int at = t * padded + (d / R) * PITCH + d % R;
-      q[at] = row[q_col + d];
-      k[at] = row[k_col + d];
-      f[at] = expf(-rate * softplus(z + a.bias[head * D + d]));
+      q[at] = a.q_scale * sum_partials(row + q_col + d, a.mixed_stride, a.mixed_partials);
+      k[at] = sum_partials(row + k_col + d, a.mixed_stride, a.mixed_partials);
+      if (!HEAD) {
+        const float z = sum_partials(a.gates + static_cast<size_t>(first + t0 + t) * a.gate_width + a.gate_at + head * D + d, a.stride, a.partials);
+        f[at] = decay_of(a, rate, z, a.bias != nullptr ? a.bias[head * D + d] : 0.f);
+      }
     }
     for (int i = threadIdx.x; i < here * cols; i += blockDim.x) {
       const int t = i / cols, c = i - t * cols;
-      v[i] = c < cols_here ? a.mixed[static_cast<size_t>(first + t0 + t) * a.channels + v_col + c] : 0.f;
+      v[i] = c < cols_here ? sum_partials(a.mixed + static_cast<size_t>(first + t0 + t) * a.pitch + v_col + c, a.mixed_stride, a.mixed_partials) : 0.f;
     }
-    if (threadIdx.x < here) b[threadIdx.x] = a.beta[static_cast<size_t>(first + t0 + threadIdx.x) * a.heads + head];
+    if (DELTA && threadIdx.x < here) b[threadIdx.x] = a.beta[static_cast<size_t>(first + t0 + threadIdx.x) * a.heads + head];
+    if (HEAD && threadIdx.x >= 16 && threadIdx.x - 16 < here) {   // (a CTA has at least a warp)
+      const int t = threadIdx.x - 16;
+      const float z = sum_partials(a.gates + static_cast<size_t>(first + t0 + t) * a.gate_width + a.gate_at + head, a.stride, a.partials);
+      f[t] = decay_of(a, rate, z, a.bias != nullptr ? a.bias[head] : 0.f);
+    }
     __syncthreads();
     for (int t = 0; t < here; ++t) {
       const float4* f4 = reinterpret_cast<const float4*>(f + t * padded + g * PITCH);
@@ -340,20 +358,22 @@ __global__ void __launch_bounds__(128, 4) delta_walk_kernel(const ScanArgs a) {
       for (int c = 0; c < C; ++c) sum[c] = 0.f;
 #pragma unroll
       for (int r = 0; r < R; r += 4) {
-        const float4 x = f4[r >> 2];
+        const float4 x = HEAD ? make_float4(f[t], f[t], f[t], f[t]) : f4[r >> 2];
         const float keep[4] = {x.x, x.y, x.z, x.w};
 #pragma unroll
         for (int e = 0; e < 4; ++e)
 #pragma unroll
           for (int c = 0; c < C; ++c) {
             S[c][r + e] *= keep[e];
-            sum[c] = __fmaf_rn(S[c][r + e], kk[r + e], sum[c]);
+            if (DELTA) sum[c] = __fmaf_rn(S[c][r + e], kk[r + e], sum[c]);
           }
       }
-      for (int offset = lanes >> 1; offset > 0; offset >>= 1)
+      if (DELTA) {
+        for (int offset = lanes >> 1; offset > 0; offset >>= 1)
 #pragma unroll
-        for (int c = 0; c < C; ++c) sum[c] += __shfl_xor_sync(0xffffffffu, sum[c], offset);
-      const float share = b[t];
+          for (int c = 0; c < C; ++c) sum[c] += __shfl_xor_sync(0xffffffffu, sum[c], offset);
+      }
+      const float share = DELTA ? b[t] : 1.f;
 #pragma unroll
       for (int c = 0; c < C; ++c) sum[c] = share * (v[t * cols + j + c] - sum[c]);   // u
       float read[C];
@@ -414,19 +434,20 @@ __global__ void __launch_bounds__(128, 4) delta_walk_kernel(const ScanArgs a) {
 //
 // `delta_local` forms P_t k_t, P_t q_t, K_s, P_B and M of every block and value head by itself; `delta_blocks` walks a
 // sequence's blocks with the state in registers: one reduction over the rows, one barrier and one update per BLOCK
-// tokens instead of per token, three multiply-adds a state element and token.
+// tokens instead of per token, three multiply-adds a state element and token.  Without the delta rule u_t = v_t: a_t is
+// not needed, T is the identity, M = Aq and K_s = F_s k_s.
 constexpr int BLOCK = 8;
 
 struct BlockArgs {
   ScanArgs s;
-  float* records;   // [blocks][head_count][record]: P_t k_t [B][Dp] | P_t q_t [B][Dp] | K_s [B][Dp] | P_B [Dp] | M [B][B]
+  float* records;   // [blocks][head_count][record]: P_t k_t [B][Dp] (delta rule) | P_t q_t [B][Dp] | K_s [B][Dp] | P_B [Dp] | M [B][B]
   int record, padded_dim;   // padded_dim: rows rounded up to what the lanes hold, zeros behind the head's own
   int num_seqs, from;       // sequences that bring at least `from` tokens run here
   int blocks;               // of the whole batch
   int head0, head_count;    // the heads this launch serves
 };
 
-__host__ __device__ constexpr int record_floats(int padded_dim) { return (3 * BLOCK + 1) * padded_dim + BLOCK * BLOCK; }
+__host__ __device__ constexpr int record_floats(int padded_dim, bool delta) { return ((delta ? 3 : 2) * BLOCK + 1) * padded_dim + BLOCK * BLOCK; }
 
 // Blocks of sequence `seq`; a warp sums them over the sequences before one.
 __device__ __forceinline__ int blocks_of(const BlockArgs& a, int seq) {
@@ -459,6 +480,7 @@ struct FoldLanes {
 };
 
 // grid (blocks, heads / 4): a warp a block and value head.
+template <bool DELTA, bool HEAD>
 __global__ void __launch_bounds__(128) delta_local_kernel(const BlockArgs a) {
   __shared__ float shared_w[4][BLOCK * BLOCK], shared_t[4][BLOCK * BLOCK];
   wait_for_previous();   // the walk may start only when this kernel is nearly done: see the end
@@ -493,31 +515,39 @@ __global__ void __launch_bounds__(128) delta_local_kernel(const BlockArgs a) {
   const float rate = s.rate[head];
   float* record = a.records + (static_cast<size_t>(block) * a.head_count + local_head) * a.record;
   float* pk = record;
-  float* pq = record + BLOCK * Dp;
-  float* kk = record + 2 * BLOCK * Dp;
-  float* whole = record + 3 * BLOCK * Dp;
-  float pair[BLOCK * BLOCK];   // [t][s], s < t: A;  [s][t], s <= t: Aq
+  float* pq = record + (DELTA ? BLOCK * Dp : 0);
+  float* kk = pq + BLOCK * Dp;
+  float* whole = kk + BLOCK * Dp;
+  float pair[BLOCK * BLOCK];   // [t][s], s < t: A (delta rule);  [s][t], s <= t: Aq
 #pragma unroll
   for (int i = 0; i < BLOCK * BLOCK; ++i) pair[i] = 0.f;
-  for (int d = lane; d < Dp; d += 32) {
+  float head_decay = 1.f;   // lane t holds token t's
+  if (HEAD && lane < here) {
+    const float z = sum_partials(s.gates + static_cast<size_t>(first + lane) * s.gate_width + s.gate_at + head, s.stride, s.partials);
+    head_decay = decay_of(s, rate, z, s.bias != nullptr ? s.bias[head] : 0.f);
+  }
+  for (int d = lane; d - lane < Dp; d += 32) {   // every lane takes part in the shuffles; rows past Dp are not stored
     float g[BLOCK], k[BLOCK], q[BLOCK];
-    const bool row = d < D;
-    const float shift = row ? s.bias[head * D + d] : 0.f;
+    const bool row = d < D, kept = d < Dp;
+    const float shift = !HEAD && row && s.bias != nullptr ? s.bias[head * D + d] : 0.f;
 #pragma unroll
     for (int t = 0; t < BLOCK; ++t) {
       const bool real = row && t < here;
-      const float* at = s.mixed + static_cast<size_t>(first + (t < here ? t : 0)) * s.channels;
+      const float* at = s.mixed + static_cast<size_t>(first + (t < here ? t : 0)) * s.pitch;
       k[t] = real ? at[k_col + d] : 0.f;
-      q[t] = real ? at[q_col + d] : 0.f;
-      g[t] = real ? s.gates[static_cast<size_t>(first + t) * s.gate_width + head * D + d] : 0.f;
+      q[t] = real ? s.q_scale * at[q_col + d] : 0.f;
+      if (!HEAD) g[t] = real ? s.gates[static_cast<size_t>(first + t) * s.gate_width + s.gate_at + head * D + d] : 0.f;
     }
-    if (s.partials > 1) {
+    if (!HEAD && s.partials > 1) {
 #pragma unroll
       for (int t = 0; t < BLOCK; ++t)
-        if (row && t < here) g[t] = sum_partials(s.gates + static_cast<size_t>(first + t) * s.gate_width + head * D + d, s.stride, s.partials);
+        if (row && t < here) g[t] = sum_partials(s.gates + static_cast<size_t>(first + t) * s.gate_width + s.gate_at + head * D + d, s.stride, s.partials);
     }
 #pragma unroll
-    for (int t = 0; t < BLOCK; ++t) g[t] = row && t < here ? expf(-rate * softplus(g[t] + shift)) : (row ? 1.f : 0.f);
+    for (int t = 0; t < BLOCK; ++t) {
+      if (HEAD) g[t] = __shfl_sync(0xffffffffu, head_decay, t);
+      else g[t] = row && t < here ? decay_of(s, rate, g[t], shift) : (row ? 1.f : 0.f);
+    }
 #pragma unroll
     for (int from = 0; from < BLOCK; ++from) {
       float w = k[from];
@@ -525,19 +555,19 @@ __global__ void __launch_bounds__(128) delta_local_kernel(const BlockArgs a) {
 #pragma unroll
       for (int t = from + 1; t < BLOCK; ++t) {
         w *= g[t];
-        pair[t * BLOCK + from] = __fmaf_rn(w, k[t], pair[t * BLOCK + from]);
+        if (DELTA) pair[t * BLOCK + from] = __fmaf_rn(w, k[t], pair[t * BLOCK + from]);
         pair[from * BLOCK + t] = __fmaf_rn(w, q[t], pair[from * BLOCK + t]);
       }
-      kk[from * Dp + d] = w;   // F k: the key as it stands at the block's end
+      if (kept) kk[from * Dp + d] = w;   // F k: the key as it stands at the block's end
     }
     float p = 1.f;
 #pragma unroll
     for (int t = 0; t < BLOCK; ++t) {
       p *= g[t];
-      pk[t * Dp + d] = p * k[t];
-      pq[t * Dp + d] = p * q[t];
+      if (DELTA && kept) pk[t * Dp + d] = p * k[t];
+      if (kept) pq[t * Dp + d] = p * q[t];
     }
-    whole[d] = p;
+    if (kept) whole[d] = p;
   }
   FoldLanes<BLOCK * BLOCK, 16>::run(pair, lane);
   float* w = shared_w[warp];
@@ -545,6 +575,16 @@ __global__ void __launch_bounds__(128) delta_local_kernel(const BlockArgs a) {
   w[2 * lane] = pair[0];
   w[2 * lane + 1] = pair[1];
   __syncwarp();
+  float* m = whole + Dp;
+  if (!DELTA) {   // M is Aq as it stands, K_s the decayed keys
+#pragma unroll
+    for (int i = lane; i < BLOCK * BLOCK; i += 32) {
+      const int t = i / BLOCK, c = i % BLOCK;
+      m[i] = c <= t ? w[c * BLOCK + t] : 0.f;
+    }
+    let_dependents_start();
+    return;
+  }
   if (lane < BLOCK) {   // column `lane` of T by forward substitution
     float column[BLOCK];
 #pragma unroll
@@ -558,7 +598,6 @@ __global__ void __launch_bounds__(128) delta_local_kernel(const BlockArgs a) {
     }
   }
   __syncwarp();
-  float* m = whole + Dp;
 #pragma unroll
   for (int i = lane; i < BLOCK * BLOCK; i += 32) {
     const int t = i / BLOCK, c = i % BLOCK;
@@ -617,14 +656,15 @@ constexpr int STAGES = 3;
 // rows 4 g .. 4 g + 3 (with CHUNKS 2 also the same LANES * 4 further on) of four neighbouring columns; LANES lanes, a
 // team, cover the head's rows.  Register c of a lane is column c ^ turn of the team's four, `turn` the lane's top two bits:
 // adding up over those lanes then needs no selection, every step keeps the first half of the columns and sends the other.
-template <int LANES, int CHUNKS>
+template <int LANES, int CHUNKS, bool DELTA>
 __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(const BlockArgs a) {
   extern __shared__ __align__(16) float blocks_shared[];
   constexpr int C = 4, PAIRS = 2 * CHUNKS, N = BLOCK * C;
   constexpr int COLUMN_LANES = LANES >= C ? C : LANES;   // lanes the columns are shared out over, then the tokens
   constexpr int TOKEN_LANES = LANES / COLUMN_LANES;
   constexpr int OWN_COLUMNS = C / COLUMN_LANES, OWN_TOKENS = BLOCK / TOKEN_LANES;
-  constexpr int Dp = 4 * LANES * CHUNKS, RECORD = record_floats(Dp), PITCH = LANES * CHUNKS;
+  constexpr int Dp = 4 * LANES * CHUNKS, RECORD = record_floats(Dp, DELTA), PITCH = LANES * CHUNKS;
+  constexpr int Q_ROW = DELTA ? BLOCK : 0, K_ROW = Q_ROW + BLOCK;   // where a record's P q and K begin, in rows
   const ScanArgs& s = a.s;
   let_dependents_start();
   wait_for_previous();
@@ -651,7 +691,7 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
   const int stage_floats = RECORD + BLOCK * cols;
   float* team_values = blocks_shared + STAGES * stage_floats + (warp * (32 / LANES) + team) * 2 * N;   // d, then c, of this team's columns
   const int v_col = 2 * s.kv_heads * s.dim + head * s.vdim + col0;
-  const bool wide_v = ((v_col | s.channels | s.vdim) & 3) == 0 && (reinterpret_cast<uintptr_t>(s.mixed) & 15) == 0;
+  const bool wide_v = ((v_col | s.pitch | s.vdim) & 3) == 0 && (reinterpret_cast<uintptr_t>(s.mixed) & 15) == 0;
   // a thread's 16-byte piece of the CTA's columns of v, the same in every block (narrow heads have more pieces than threads)
   const int pieces = BLOCK * cols / 4, piece_t = static_cast<int>(threadIdx.x) / (cols / 4), piece_c = (static_cast<int>(threadIdx.x) - piece_t * (cols / 4)) * 4;
   const bool one_piece = wide_v && pieces <= static_cast<int>(blockDim.x);
@@ -666,16 +706,16 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
       next_record += record_step;
       float* v = at + RECORD;
       const int here = min(BLOCK, length - block * BLOCK);
-      const float* from = s.mixed + static_cast<size_t>(first + block * BLOCK) * s.channels + v_col;
+      const float* from = s.mixed + static_cast<size_t>(first + block * BLOCK) * s.pitch + v_col;
       if (one_piece) {
         if (static_cast<int>(threadIdx.x) < pieces) {
-          if (piece_t < here && piece_c < cols_here) copy16(v + piece_t * cols + piece_c, from + static_cast<size_t>(piece_t) * s.channels + piece_c);
+          if (piece_t < here && piece_c < cols_here) copy16(v + piece_t * cols + piece_c, from + static_cast<size_t>(piece_t) * s.pitch + piece_c);
           else *reinterpret_cast<float4*>(v + piece_t * cols + piece_c) = make_float4(0.f, 0.f, 0.f, 0.f);
         }
       } else {
         for (int i = threadIdx.x; i < BLOCK * cols; i += blockDim.x) {
           const int t = i / cols, c = i - t * cols;
-          if (t < here && c < cols_here) copy4(v + i, from + static_cast<size_t>(t) * s.channels + c);
+          if (t < here && c < cols_here) copy4(v + i, from + static_cast<size_t>(t) * s.pitch + c);
           else v[i] = 0.f;
         }
       }
@@ -707,13 +747,13 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
     const float* v = at + RECORD;
     float sum[2][N];   // a_t, then c_t, of this thread's rows: [column][token]
 #pragma unroll
-    for (int which = 0; which < 2; ++which) {
+    for (int which = DELTA ? 0 : 1; which < 2; ++which) {
 #pragma unroll
       for (int t = 0; t < BLOCK; ++t) {
         unsigned long long acc[C];
 #pragma unroll
         for (int chunk = 0; chunk < CHUNKS; ++chunk) {
-          const ulonglong2 x = rows[(which * BLOCK + t) * PITCH + chunk * LANES];
+          const ulonglong2 x = rows[((which == 0 ? 0 : Q_ROW) + t) * PITCH + chunk * LANES];
 #pragma unroll
           for (int c = 0; c < C; ++c) {
             acc[c] = chunk == 0 ? mul2(S[c][0], x.x) : fma2(S[c][2 * chunk], x.x, acc[c]);
@@ -732,22 +772,22 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
 #pragma unroll
       for (int i = 0; i < half; ++i)
 #pragma unroll
-        for (int which = 0; which < 2; ++which) sum[which][i] += __shfl_xor_sync(0xffffffffu, sum[which][i + half], offset);
+        for (int which = DELTA ? 0 : 1; which < 2; ++which) sum[which][i] += __shfl_xor_sync(0xffffffffu, sum[which][i + half], offset);
     // this lane holds its columns' sums, shared with TOKEN_LANES - 1 others: d_t = v_t - a_t of its own tokens
 #pragma unroll
     for (int i = 0; i < OWN_COLUMNS; ++i) {
-      FoldLanes<BLOCK, TOKEN_LANES / 2>::run(sum[0] + i * BLOCK, lane);
+      if constexpr (DELTA) FoldLanes<BLOCK, TOKEN_LANES / 2>::run(sum[0] + i * BLOCK, lane);
       FoldLanes<BLOCK, TOKEN_LANES / 2>::run(sum[1] + i * BLOCK, lane);
       const int c = turn + i;
 #pragma unroll
       for (int k = 0; k < OWN_TOKENS; ++k) {
         const int t = g % TOKEN_LANES * OWN_TOKENS + k;
-        team_values[c * BLOCK + t] = v[t * cols + j + c] - sum[0][i * BLOCK + k];
+        team_values[c * BLOCK + t] = v[t * cols + j + c] - (DELTA ? sum[0][i * BLOCK + k] : 0.f);
         team_values[N + c * BLOCK + t] = sum[1][i * BLOCK + k];
       }
     }
     __syncwarp();
-    const float* decay = at + 3 * BLOCK * Dp;
+    const float* decay = at + (K_ROW + BLOCK) * Dp;
 #pragma unroll
     for (int chunk = 0; chunk < CHUNKS; ++chunk) {
       const ulonglong2 x = *(reinterpret_cast<const ulonglong2*>(decay) + g + chunk * LANES);
@@ -772,7 +812,7 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
       for (int c = 0; c < C; ++c) dd[c] = pack2(d[c][t], d[c][t]);
 #pragma unroll
       for (int chunk = 0; chunk < CHUNKS; ++chunk) {
-        const ulonglong2 x = rows[(2 * BLOCK + t) * PITCH + chunk * LANES];
+        const ulonglong2 x = rows[(K_ROW + t) * PITCH + chunk * LANES];
 #pragma unroll
         for (int c = 0; c < C; ++c) {
           S[c][2 * chunk] = fma2(x.x, dd[c], S[c][2 * chunk]);
@@ -814,6 +854,69 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
         if (d + 1 < s.dim) at[s.vdim] = two.y;
       }
     }
+}
+
+// ------------------------------------------------------------------------------------------------ low_rank
+// z[n][c] = sum_r A[c][r] * x[n][r], x the `rank` columns of a fused projection from `at` on (a stack of partial sums is
+// added up), A [C][padded] in the activation type with zeros behind its rank (16-byte rows).  A thread takes one column of
+// TOK tokens, whose low-rank rows lie in shared memory.
+constexpr int LOW_THREADS = 128;
+
+template <typename T, int TOK>
+__global__ void __launch_bounds__(LOW_THREADS) low_rank_kernel(const float* __restrict__ fused, int partials, long long stride, int total,
+                                                               int at, const T* __restrict__ A, int padded, int rank,
+                                                               float* __restrict__ z, int n, int columns) {
+  extern __shared__ __align__(16) float low_shared[];   // [TOK][padded]
+  let_dependents_start();
+  wait_for_previous();
+  const int first = blockIdx.y * TOK, here = min(TOK, n - first);
+  for (int i = threadIdx.x; i < TOK * padded; i += LOW_THREADS) {
+    const int t = i / padded, r = i - t * padded;
+    low_shared[i] = t < here && r < rank ? sum_partials(fused + static_cast<size_t>(first + t) * total + at + r, stride, partials) : 0.f;
+  }
+  __syncthreads();
+  const int c = blockIdx.x * LOW_THREADS + threadIdx.x;
+  if (c >= columns) return;
+  const T* row = A + static_cast<size_t>(c) * padded;
+  float acc[TOK];
+#pragma unroll
+  for (int t = 0; t < TOK; ++t) acc[t] = 0.f;
+  for (int r = 0; r < padded; r += 8) {
+    float w[8];
+    {
+      float lo[4], hi[4];
+      load4<T>(row + r, lo);
+      load4<T>(row + r + 4, hi);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) { w[e] = lo[e]; w[4 + e] = hi[e]; }
+    }
+#pragma unroll
+    for (int t = 0; t < TOK; ++t) {
+      const float4 x0 = *reinterpret_cast<const float4*>(low_shared + t * padded + r);
+      const float4 x1 = *reinterpret_cast<const float4*>(low_shared + t * padded + r + 4);
+      acc[t] = __fmaf_rn(w[0], x0.x, acc[t]); acc[t] = __fmaf_rn(w[1], x0.y, acc[t]);
+      acc[t] = __fmaf_rn(w[2], x0.z, acc[t]); acc[t] = __fmaf_rn(w[3], x0.w, acc[t]);
+      acc[t] = __fmaf_rn(w[4], x1.x, acc[t]); acc[t] = __fmaf_rn(w[5], x1.y, acc[t]);
+      acc[t] = __fmaf_rn(w[6], x1.z, acc[t]); acc[t] = __fmaf_rn(w[7], x1.w, acc[t]);
+    }
+  }
+#pragma unroll
+  for (int t = 0; t < TOK; ++t)
+    if (t < here) z[static_cast<size_t>(first + t) * columns + c] = acc[t];
+}
+
+template <typename T>
+static void launch_low_rank(const float* fused, int partials, long long stride, int total, int at, const void* A, int padded, int rank,
+                            float* z, int n, int columns, cudaStream_t stream) {
+  const unsigned blocks = static_cast<unsigned>((columns + LOW_THREADS - 1) / LOW_THREADS);
+  const T* a = static_cast<const T*>(A);
+  if (n <= 64) {   // few tokens: one each, so that they fill the device
+    launch_dependent(low_rank_kernel<T, 1>, dim3(blocks, n), LOW_THREADS, padded * sizeof(float), stream, fused, partials, stride,
+                     total, at, a, padded, rank, z, n, columns);
+  } else {
+    launch_dependent(low_rank_kernel<T, 8>, dim3(blocks, (n + 7) / 8), LOW_THREADS, 8 * padded * sizeof(float), stream, fused, partials,
+                     stride, total, at, a, padded, rank, z, n, columns);
+  }
 }
 
 }  // namespace delta
@@ -888,36 +991,47 @@ static inline bool delta_shape(int dim, int vdim, DeltaShape* shape) {
 }
 
 // Scratch floats of one head of one block of BLOCK tokens; 0: heads of this size walk token by token.
-SHRIKE_API int shrike_delta_scan_record(int dim) {
+SHRIKE_API int shrike_delta_scan_record(int dim, int delta) {
   DeltaShape shape;
   if (dim > 256 || !delta_shape(dim, 4, &shape)) return 0;
-  return record_floats(shape.lanes * shape.rows);
+  return record_floats(shape.lanes * shape.rows, delta != 0);
 }
 SHRIKE_API int shrike_delta_scan_block() { return BLOCK; }
 
+// `mixed` (`mixed_partials` slices `mixed_stride` apart, rows of `pitch`): q | k | v; only a walk takes more than one slice.
+// `beta` null: no delta rule.  `gate_each`: 1, one decay a head, or dim, one a key channel (`bias`, where there is one, has
+// heads * gate_each numbers); the decays' columns begin at `gate_at`.
 // Sequences that bring at least `from` tokens (0: none) run in blocks, for which the caller holds `records`
 // (blocks x head_count x shrike_delta_scan_record floats, `blocks` = the sum of ceil(length / BLOCK) over them); heads are
 // then served `head_count` at a time.  `early_state` 1: the caller knows that whatever kernel wrote the states has finished
 // (an earlier step, not merely an earlier launch), so that the walk may read them while the kernel before it runs.  `shorter`: whether the batch has sequences below `from`.
-SHRIKE_API int shrike_delta_scan(const float* mixed, const float* beta, const float* gates, int partials, long long stride,
-                                 int gate_width, const float* rate, const float* bias, float* state, const int* q_start,
+SHRIKE_API int shrike_delta_scan(const float* mixed, int mixed_partials, long long mixed_stride, int pitch, const float* beta,
+                                 const float* gates, int partials, long long stride, int gate_width, int gate_at, int gate_each,
+                                 const float* rate, const float* bias, float sign, float q_scale, float* state, const int* q_start,
                                  const int* state_slot, float* out, int num_seqs, int heads, int kv_heads, int dim, int vdim,
                                  int head_stride, int num_slots, int from, int shorter, float* records, int blocks,
                                  int head_count, int early_state, cudaStream_t stream) {
   if (num_seqs <= 0) return SHRIKE_OK;
   if (heads < 1 || heads > 65535 || num_seqs > 65535 || kv_heads < 1 || heads % kv_heads || dim < 1 || vdim < 1 || partials < 1 ||
-      head_stride < dim * vdim || gate_width < heads * dim)
+      mixed_partials < 1 || head_stride < dim * vdim || (gate_each != 1 && gate_each != dim) || gate_at < 0 ||
+      gate_width < gate_at + heads * gate_each || pitch < 2 * kv_heads * dim + heads * vdim)
     return SHRIKE_BAD_ARGUMENT;
+  const bool delta_rule = beta != nullptr, per_head = gate_each == 1 && dim > 1;
+  if (per_head && !delta_rule) return SHRIKE_BAD_ARGUMENT;   // no design has asked for that pairing
   if (head_stride % 4 || reinterpret_cast<uintptr_t>(state) % 16) return SHRIKE_BAD_ARGUMENT;
   DeltaShape shape;
   if (!delta_shape(dim, vdim, &shape)) return SHRIKE_BAD_ARGUMENT;   // heads of more than 1,024 rows
-  ScanArgs a = {mixed, beta, gates, stride, partials, gate_width, rate, bias, state, q_start, state_slot, out,
-                heads, kv_heads, dim, vdim, 2 * kv_heads * dim + heads * vdim, head_stride, num_slots, shape.lanes, shape.cols, 0, early_state};
+  ScanArgs a = {mixed, mixed_stride, mixed_partials, pitch, beta, gates, stride, partials, gate_width, gate_at, rate, bias, sign, q_scale,
+                state, q_start, state_slot, out, heads, kv_heads, dim, vdim, head_stride, num_slots, shape.lanes, shape.cols, 0, early_state};
   const bool in_blocks = from > 0 && records != nullptr && blocks > 0 && head_count > 0 && shape.rows == 8;
+  if (in_blocks && mixed_partials > 1) return SHRIKE_BAD_ARGUMENT;
   const unsigned slices = static_cast<unsigned>((vdim + shape.cols - 1) / shape.cols);
   if (!in_blocks || shorter) {
     a.skip_from = in_blocks ? from : 0;
-    void (*kernel)(ScanArgs) = shape.rows == 8 ? delta_walk_kernel<8, 4> : delta_walk_kernel<32, 1>;
+    void (*kernel)(ScanArgs);
+    if (!delta_rule) kernel = shape.rows == 8 ? delta_walk_kernel<8, 4, false, false> : delta_walk_kernel<32, 1, false, false>;
+    else if (per_head) kernel = shape.rows == 8 ? delta_walk_kernel<8, 4, true, true> : delta_walk_kernel<32, 1, true, true>;
+    else kernel = shape.rows == 8 ? delta_walk_kernel<8, 4, true, false> : delta_walk_kernel<32, 1, true, false>;
     if (shape.smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(shape.smem));
     launch_dependent(kernel, dim3(slices, heads, num_seqs), static_cast<unsigned>(shape.threads), shape.smem, stream, a);
   }
@@ -926,7 +1040,7 @@ SHRIKE_API int shrike_delta_scan(const float* mixed, const float* beta, const fl
     b.s = a;
     b.records = records;
     b.padded_dim = shape.lanes * shape.rows;
-    b.record = record_floats(b.padded_dim);
+    b.record = record_floats(b.padded_dim, delta_rule);
     b.num_seqs = num_seqs; b.from = from; b.blocks = blocks;
     // Four rows a thread where the walks are few (twice the warps hide each other's waits), eight where there are enough
     // of them (half the adding up over lanes); a head of more than 128 rows takes eight.
@@ -943,7 +1057,9 @@ SHRIKE_API int shrike_delta_scan(const float* mixed, const float* beta, const fl
     b.s.cols = per_warp * warps;
     const unsigned block_slices = static_cast<unsigned>((vdim + b.s.cols - 1) / b.s.cols);
     void (*kernel)(BlockArgs) = nullptr;
-#define SHRIKE_DELTA_BLOCKS(L) kernel = chunks == 2 ? delta_blocks_kernel<L, 2> : delta_blocks_kernel<L, 1>
+#define SHRIKE_DELTA_BLOCKS(L)                                                                                    \
+  kernel = delta_rule ? (chunks == 2 ? delta_blocks_kernel<L, 2, true> : delta_blocks_kernel<L, 1, true>) \
+                      : (chunks == 2 ? delta_blocks_kernel<L, 2, false> : delta_blocks_kernel<L, 1, false>)
     switch (lanes) {
       case 1: SHRIKE_DELTA_BLOCKS(1); break;
       case 2: SHRIKE_DELTA_BLOCKS(2); break;
@@ -967,9 +1083,25 @@ SHRIKE_API int shrike_delta_scan(const float* mixed, const float* beta, const fl
     for (int head0 = 0; head0 < heads; head0 += head_count) {
       b.head0 = head0;
       b.head_count = min(head_count, heads - head0);
-      launch_dependent(delta_local_kernel, dim3(static_cast<unsigned>(blocks), static_cast<unsigned>((b.head_count + 3) / 4)), 128, 0, stream, b);
+      void (*local)(BlockArgs) = !delta_rule ? delta_local_kernel<false, false>
+                                             : (per_head ? delta_local_kernel<true, true> : delta_local_kernel<true, false>);
+      launch_dependent(local, dim3(static_cast<unsigned>(blocks), static_cast<unsigned>((b.head_count + 3) / 4)), 128, 0, stream, b);
       launch_dependent(kernel, dim3(block_slices, b.head_count, num_seqs), static_cast<unsigned>(warps * 32), smem, stream, b);
     }
   }
+  return shrike_launch_status();
+}
+
+// z [N][columns] = the rows of A [columns][padded] (activation type, zeros from `rank` on, `padded` a multiple of 8, rows on
+// 16-byte borders) times the `rank` columns of `fused` from `at` on.
+SHRIKE_API int shrike_low_rank(const float* fused, int partials, long long stride, int total, int at, const void* A, int dtype,
+                               int padded, int rank, float* z, int n, int columns, cudaStream_t stream) {
+  if (n <= 0) return SHRIKE_OK;
+  if (partials < 1 || columns < 1 || rank < 1 || padded < rank || padded % 8 || padded > 1024 || at < 0 || at + rank > total ||
+      reinterpret_cast<uintptr_t>(A) % 16 || n > 8 * 65535)
+    return SHRIKE_BAD_ARGUMENT;
+  if (dtype == SHRIKE_F32) launch_low_rank<float>(fused, partials, stride, total, at, A, padded, rank, z, n, columns, stream);
+  else if (dtype == SHRIKE_BF16) launch_low_rank<__nv_bfloat16>(fused, partials, stride, total, at, A, padded, rank, z, n, columns, stream);
+  else return SHRIKE_BAD_ARGUMENT;
   return shrike_launch_status();
 }

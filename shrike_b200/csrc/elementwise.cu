@@ -412,7 +412,7 @@ static void launch_plain_act(void* x, long long count, int act, cudaStream_t str
 // x (`count` elements) <- act(x), `act` one of SHRIKE_PLAIN_*.
 SHRIKE_API int shrike_plain_act(void* x, int dtype, long long count, int act, cudaStream_t stream) {
   if (count <= 0) return SHRIKE_OK;
-  if (act != SHRIKE_PLAIN_RELU2) return SHRIKE_BAD_ARGUMENT;
+  if (!known_plain_activation(act)) return SHRIKE_BAD_ARGUMENT;
   if (dtype == SHRIKE_F32) launch_plain_act<float>(x, count, act, stream);
   else if (dtype == SHRIKE_BF16) launch_plain_act<__nv_bfloat16>(x, count, act, stream);
   else return SHRIKE_BAD_ARGUMENT;

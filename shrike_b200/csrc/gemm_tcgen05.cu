@@ -342,7 +342,7 @@ SHRIKE_API int shrike_gemm_tc(const void* x, const void* w, const float* bias, v
 // rounded to bfloat16 before the activation; `act` one of SHRIKE_PLAIN_*.
 SHRIKE_API int shrike_gemm_tc_act(const void* x, const void* w, void* out, int tokens, int n, int k, int act, int* status,
                                   cudaStream_t stream) {
-  if (act != SHRIKE_PLAIN_RELU2) return SHRIKE_BAD_ARGUMENT;
+  if (!known_plain_activation(act)) return SHRIKE_BAD_ARGUMENT;
   return launch_gemm_tc(x, w, nullptr, out, SHRIKE_BF16, tokens, n, k, 1, 0, status, stream, 0.f, act);
 }
 

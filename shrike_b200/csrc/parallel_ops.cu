@@ -911,7 +911,8 @@ template <typename T>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 route_top_kernel(const T* __restrict__ x, const float* __restrict__ router, const float* __restrict__ shared_gate,
                  float* __restrict__ weights, int n, int width, int experts, int top, int columns, float renorm_eps,
-                 int sigmoid_scores, int renormalise, const float* __restrict__ correction, int group_count, int group_keep) {
+                 int sigmoid_scores, int renormalise, const float* __restrict__ correction, int group_count, int group_keep,
+                 int identity) {
   extern __shared__ float route_shared[];   // [ROUTE_WARPS][rows] sums of the warps, then [rows] scores in the first row
   let_dependents_start();
   wait_for_previous();
@@ -919,8 +920,11 @@ route_top_kernel(const T* __restrict__ x, const float* __restrict__ router, cons
   const int token = blockIdx.x;
   const T* row = x + static_cast<size_t>(token) * width;
   float* out = weights + static_cast<size_t>(token) * columns;
+  // the last `identity` of the `experts` are identity experts: their weights leave as one sum in the last column
+  const int real = experts - identity;
+  const bool shared_column = columns > real + (identity > 0 ? 1 : 0);
   // rows of the product: the experts, then (when there is one) the shared expert's gate vector
-  const int rows = experts + (columns > experts && shared_gate != nullptr ? 1 : 0);
+  const int rows = experts + (shared_column && shared_gate != nullptr ? 1 : 0);
   const bool wide = (width & 3) == 0 && (reinterpret_cast<uintptr_t>(router) & 15) == 0 &&
                     (shared_gate == nullptr || (reinterpret_cast<uintptr_t>(shared_gate) & 15) == 0) &&
                     (reinterpret_cast<uintptr_t>(x) & 15) == 0;
@@ -984,10 +988,10 @@ route_top_kernel(const T* __restrict__ x, const float* __restrict__ router, cons
   __syncwarp();
   for (int e = lane; e < experts; e += 32) {
     score[e] = score[e] / total;
-    out[e] = 0.f;
+    if (e < real) out[e] = 0.f;
   }
   __syncwarp();
-  float chosen_sum = 0.f;
+  float chosen_sum = 0.f, identity_sum = 0.f;
   if (correction != nullptr || group_count > 0) {
     // the choice goes by score + correction among the experts of the best groups; the weights are the scores.  Rows one
     // and two of the warps' sums are used up: they hold the choice scores and the groups' best.
@@ -1030,8 +1034,9 @@ route_top_kernel(const T* __restrict__ x, const float* __restrict__ router, cons
       if (where < experts) {
         const float weight = score[where];
         chosen_sum += weight;
+        if (where >= real) identity_sum += weight;
         if (lane == 0) {
-          out[where] = weight;
+          if (where < real) out[where] = weight;
           choice[where] = -INFINITY;
         }
       }
@@ -1054,17 +1059,20 @@ route_top_kernel(const T* __restrict__ x, const float* __restrict__ router, cons
     }
     if (sigmoid_scores) mine = 1.0f / (1.0f + expf(-mine));
     chosen_sum += mine;
+    if (where >= real && where < experts) identity_sum += mine;
     if (lane == 0 && where < experts) {
-      out[where] = mine;
+      if (where < real) out[where] = mine;
       score[where] = sigmoid_scores ? -INFINITY : -2.f;
     }
     __syncwarp();
   }
   if (renormalise) {
     const float inv = 1.0f / (chosen_sum + renorm_eps);
-    for (int e = lane; e < experts; e += 32) out[e] = out[e] * inv;
+    for (int e = lane; e < real; e += 32) out[e] = out[e] * inv;
+    identity_sum *= inv;
   }
-  if (columns > experts && lane == 0) out[experts] = shared_gate != nullptr ? 1.0f / (1.0f + expf(-shared_dot)) : 1.f;
+  if (shared_column && lane == 0) out[real] = shared_gate != nullptr ? 1.0f / (1.0f + expf(-shared_dot)) : 1.f;
+  if (identity > 0 && lane == 0) out[columns - 1] = identity_sum;
 }
 
 // ------------------------------------------------------------------------------------------ act_mul_blocks
@@ -1107,6 +1115,46 @@ act_mul_blocks_kernel(const T* __restrict__ gate_up, const float* __restrict__ w
       *reinterpret_cast<Pack*>(o + c) = r;
     }
   }
+}
+
+// ---------------------------------------------------------------------------------------------- act_blocks
+// Experts without a gate: x [N][I] in place, column c of expert c / each: x <- act(x) * the expert's weight for the row.
+// A thread takes VEC columns (one 16-byte access; no group straddles two experts); a column whose expert the row did not
+// choose becomes exactly zero without being read.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+act_blocks_kernel(T* __restrict__ x, const float* __restrict__ weights, int n, int inter, int each, int columns, int act) {
+  let_dependents_start();
+  wait_for_previous();
+  struct alignas(sizeof(T) * VEC) Pack { T v[VEC]; };
+  const int groups = inter / VEC;
+  for (int row = blockIdx.y; row < n; row += gridDim.y) {
+    T* at = x + static_cast<size_t>(row) * inter;
+    const float* w = weights + static_cast<size_t>(row) * columns;
+    for (int group = blockIdx.x * blockDim.x + threadIdx.x; group < groups; group += gridDim.x * blockDim.x) {
+      const float share = w[group * VEC / each];
+      Pack r;
+      if (share == 0.f) {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) r.v[j] = from_float<T>(0.f);
+      } else {
+        r = *reinterpret_cast<const Pack*>(at + group * VEC);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) r.v[j] = from_float<T>(__fmul_rn(plain_act_value(act, to_float(r.v[j])), share));
+      }
+      *reinterpret_cast<Pack*>(at + group * VEC) = r;
+    }
+  }
+}
+
+template <typename T>
+static void launch_act_blocks(void* x, const float* weights, int n, int inter, int each, int columns, int act, cudaStream_t stream) {
+  constexpr int WIDE = 16 / sizeof(T);
+  const bool vec = reinterpret_cast<uintptr_t>(x) % 16 == 0 && each % WIDE == 0;
+  const int groups = vec ? inter / WIDE : inter;
+  const dim3 grid(max(1, min(64, (groups + 255) / 256)), max(1, min(n, 65535)));
+  if (vec) launch_dependent(act_blocks_kernel<T, WIDE>, grid, 256, 0, stream, static_cast<T*>(x), weights, n, inter, each, columns, act);
+  else launch_dependent(act_blocks_kernel<T, 1>, grid, 256, 0, stream, static_cast<T*>(x), weights, n, inter, each, columns, act);
 }
 
 }  // namespace parallel
@@ -1300,12 +1348,16 @@ SHRIKE_API int shrike_matrix_memory_out(const float* numerator, const float* den
 // chosen experts keep their scores as they are.
 // `correction` (float32 [experts], null: none) is added to the scores for the choice alone; `group_count` > 0: equal groups
 // of neighbouring experts, of which only those of the `group_keep` groups with the largest choice score can be chosen.
+// `identity`: the last so many of the `experts` are identity experts; `weights` has no columns for them but one last column
+// with the sum of what the row gives them.
 SHRIKE_API int shrike_route_top_groups(const void* x, int dtype, const float* router, const float* shared_gate, float* weights, int n,
                                        int width, int experts, int top, int columns, float renorm_eps, int sigmoid_scores,
-                                       int renormalise, const float* correction, int group_count, int group_keep,
+                                       int renormalise, const float* correction, int group_count, int group_keep, int identity,
                                        cudaStream_t stream) {
   if (n <= 0) return SHRIKE_OK;
-  if (experts < 1 || top < 1 || top > experts || experts > 1024 || (columns != experts && columns != experts + 1)) return SHRIKE_BAD_ARGUMENT;
+  if (experts < 1 || top < 1 || top > experts || experts > 1024 || identity < 0 || identity >= experts) return SHRIKE_BAD_ARGUMENT;
+  const int least = experts - identity + (identity > 0 ? 1 : 0);
+  if (columns != least && columns != least + 1) return SHRIKE_BAD_ARGUMENT;
   if (group_count > 0 && (experts % group_count || group_keep < 1 || group_keep > group_count || top > group_keep * (experts / group_count)))
     return SHRIKE_BAD_ARGUMENT;
   const unsigned blocks = static_cast<unsigned>(n);
@@ -1313,11 +1365,11 @@ SHRIKE_API int shrike_route_top_groups(const void* x, int dtype, const float* ro
   if (dtype == SHRIKE_F32)
     launch_dependent(route_top_kernel<float>, blocks, ROUTE_WARPS * 32, smem, stream, static_cast<const float*>(x), router,
                      shared_gate, weights, n, width, experts, top, columns, renorm_eps, sigmoid_scores, renormalise, correction,
-                     group_count, group_keep);
+                     group_count, group_keep, identity);
   else if (dtype == SHRIKE_BF16)
     launch_dependent(route_top_kernel<__nv_bfloat16>, blocks, ROUTE_WARPS * 32, smem, stream, static_cast<const __nv_bfloat16*>(x),
                      router, shared_gate, weights, n, width, experts, top, columns, renorm_eps, sigmoid_scores, renormalise, correction,
-                     group_count, group_keep);
+                     group_count, group_keep, identity);
   else return SHRIKE_BAD_ARGUMENT;
   return shrike_launch_status();
 }
@@ -1326,7 +1378,7 @@ SHRIKE_API int shrike_route_top_scores(const void* x, int dtype, const float* ro
                                        int width, int experts, int top, int columns, float renorm_eps, int sigmoid_scores,
                                        int renormalise, cudaStream_t stream) {
   return shrike_route_top_groups(x, dtype, router, shared_gate, weights, n, width, experts, top, columns, renorm_eps, sigmoid_scores,
-                                 renormalise, nullptr, 0, 0, stream);
+                                 renormalise, nullptr, 0, 0, 0, stream);
 }
 
 SHRIKE_API int shrike_route_top(const void* x, int dtype, const float* router, const float* shared_gate, float* weights, int n,
@@ -1376,4 +1428,18 @@ SHRIKE_API int shrike_act_mul_blocks_at(const void* gate_up, const float* weight
 SHRIKE_API int shrike_act_mul_blocks(const void* gate_up, const float* weights, void* out, int dtype, int n, int inter, int experts,
                                      int each, int columns, int act, float limit, cudaStream_t stream) {
   return shrike_act_mul_blocks_at(gate_up, weights, out, dtype, n, inter, experts, each, columns, act, limit, 0, stream);
+}
+
+// x [N][experts * each] in place: the activation of an ungated expert times the expert's weight; `act` one of SHRIKE_PLAIN_*,
+// `weights` [N][columns] as route_top leaves them.
+SHRIKE_API int shrike_act_blocks(void* x, const float* weights, int dtype, int n, int experts, int each, int columns, int act,
+                                 cudaStream_t stream) {
+  if (n <= 0) return SHRIKE_OK;
+  if (experts < 1 || each < 1 || columns < experts || !known_plain_activation(act) ||
+      static_cast<long long>(experts) * each > 0x7fffffffLL)
+    return SHRIKE_BAD_ARGUMENT;
+  if (dtype == SHRIKE_F32) launch_act_blocks<float>(x, weights, n, experts * each, each, columns, act, stream);
+  else if (dtype == SHRIKE_BF16) launch_act_blocks<__nv_bfloat16>(x, weights, n, experts * each, each, columns, act, stream);
+  else return SHRIKE_BAD_ARGUMENT;
+  return shrike_launch_status();
 }

@@ -17,7 +17,7 @@
 //                    portions in three launches over runs of tokens (every run from a zero state and its decay, the
 //                    runs' states carried in order, every run again from the state it starts from).
 //   head_rms         every head of a row over its root mean square, times one weight of the head's size, times the
-//                    sigmoid of columns of a fused projection (optional).
+//                    sigmoid, or the SiLU, of columns of a fused projection (optional).
 //
 // Sums, norms, gates, decays and states are float32; a result is rounded once, when it is stored in the activation type.
 #include <cooperative_groups.h>
@@ -509,7 +509,7 @@ template <typename TO, int VEC>
 __global__ void __launch_bounds__(128) head_rms_kernel(const float* __restrict__ x, const float* __restrict__ weight,
                                                        TO* __restrict__ out, int n, int heads, int size, float eps,
                                                        const float* __restrict__ gates, int partials, long long stride,
-                                                       int gate_width, int gate_at) {
+                                                       int gate_width, int gate_at, int gate_silu) {
   let_dependents_start();
   wait_for_previous();
   constexpr int UNITS = 2;
@@ -557,7 +557,7 @@ __global__ void __launch_bounds__(128) head_rms_kernel(const float* __restrict__
 #pragma unroll
       for (int e = 0; e < VEC; ++e) {
         w[e] = v[u][e] * r * (weight != nullptr ? weight[g * VEC + e] : 1.f);
-        if (gates != nullptr) w[e] *= sigmoid_for<TO>(z[u][e]);
+        if (gates != nullptr) w[e] *= gate_silu ? z[u][e] * sigmoid_for<TO>(z[u][e]) : sigmoid_for<TO>(z[u][e]);
       }
       if constexpr (VEC == 4) store4<TO>(out + unit * size + g * 4, w);
       else out[unit * size + g] = from_float<TO>(w[0]);
@@ -723,10 +723,11 @@ SHRIKE_API int shrike_short_conv_keep(const float* fused, int partials, long lon
   return shrike_launch_status();
 }
 
-// `gates` (null: none): [partials][N][gate_width] float32, `stride` elements between partials; see the kernel.
+// `gates` (null: none): [partials][N][gate_width] float32, `stride` elements between partials; `gate_silu` 1: their SiLU
+// multiplies the heads, not their sigmoid.  See the kernel.
 SHRIKE_API int shrike_head_rms(const float* x, const float* weight, void* out, int dtype, int n, int heads, int size,
                                float eps, const float* gates, int partials, long long stride, int gate_width, int gate_at,
-                               cudaStream_t stream) {
+                               int gate_silu, cudaStream_t stream) {
   if (n <= 0) return SHRIKE_OK;
   if (heads < 1 || size < 1 || partials < 1) return SHRIKE_BAD_ARGUMENT;
   if (gates != nullptr && (gate_at < 0 || gate_at + heads * size > gate_width)) return SHRIKE_BAD_ARGUMENT;
@@ -737,7 +738,7 @@ SHRIKE_API int shrike_head_rms(const float* x, const float* weight, void* out, i
                    (gates == nullptr || (reinterpret_cast<uintptr_t>(gates) % 16 == 0 && gate_at % 4 == 0 && gate_width % 4 == 0 && stride % 4 == 0));
 #define SHRIKE_HEAD_RMS(T, V)                                                                                               \
   launch_dependent(head_rms_kernel<T, V>, static_cast<unsigned>(blocks), 128, 0, stream, x, weight, static_cast<T*>(out), n, heads, \
-                   size, eps, gates, partials, stride, gate_width, gate_at)
+                   size, eps, gates, partials, stride, gate_width, gate_at, gate_silu)
   if (dtype == SHRIKE_F32) { if (vec) SHRIKE_HEAD_RMS(float, 4); else SHRIKE_HEAD_RMS(float, 1); }
   else if (dtype == SHRIKE_BF16) { if (vec) SHRIKE_HEAD_RMS(__nv_bfloat16, 4); else SHRIKE_HEAD_RMS(__nv_bfloat16, 1); }
   else return SHRIKE_BAD_ARGUMENT;

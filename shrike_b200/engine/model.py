@@ -75,7 +75,7 @@ class DecoderModel:
                 cls = part_class(category, spec.kind)
                 built[role] = cls(spec, {local: tensors[names.layer_tensor(index, role, local)]
                                          for local in cls.parameters(spec)}, ops, runtime)
-            self.blocks.append(part_class("block", layer.block)(**built))
+            self.blocks.append(part_class("block", layer.block)(**built, **dict(layer.block_options)))
             if hasattr(self.blocks[-1], "prepare"):
                 self.blocks[-1].prepare()
             parts += [*built.values(), self.blocks[-1]]

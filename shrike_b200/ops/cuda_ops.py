@@ -60,11 +60,15 @@ _LIMITS = {
     "stream_norm": "1 to 8 streams, at most four pending sums, a row that fits an SM's shared memory",
     "short_conv": "1 to 32 taps, at most 65535 sequences, the convolved channels the projection's first columns",
     "gated_scan": "heads of at most 1024 rows, at most 65535 sequences, heads and runs of tokens, the row at least as wide as q, f and v, the state's heads at least dim * vdim floats",
-    "route_top": "at most 1024 experts, 1 <= top <= experts, the weights [N, experts] or [N, experts + 1], groups of equal size that hold enough experts",
+    "route_top": "at most 1024 experts, 1 <= top <= experts, the weights [N, experts] (identity experts sharing one last column) and a column more for a shared expert, groups of equal size that hold enough experts",
     "norm_join": "the row width must be at most 32768 (8192 when it is no multiple of 4)",
     "side_gate": "the gate at least as wide as the token's part, which lies inside the table's rows",
     "delta_prep": "1 to 32 taps, heads a multiple of kv heads, beta and the low-rank columns behind q, k and v inside the row",
-    "delta_scan": "heads of at most 1024 rows, at most 65535 sequences and heads, the state's heads on 16-byte borders and at least dim * vdim floats",
+    "delta_scan": "heads of at most 1024 rows, at most 65535 sequences and heads, the state's heads on 16-byte borders and at least dim * vdim floats, a decay per head only with beta",
+    "low_rank": "a rank of at most 1024, its columns inside the row, the matrix's rows on 16-byte borders",
+    "sum_norm": "the row width must be at most 32768 (8192 when it is no multiple of 4), at most 64 slices in all",
+    "element_gate": "the gate's columns inside the row, the padded head at least as wide as its values",
+    "act_blocks": "an activation the kernels know, a weight column per expert",
     "act_mul_blocks": "experts * each columns at most, the rest the shared expert's, which needs the weights' last column",
     "paged_attention_bf16": "at most 65535 sequences and heads, heads a multiple of kv heads, at most 32 splits",
 }
@@ -179,26 +183,32 @@ class CudaOps:
         lib.shrike_gated_scan.argtypes = [_P, _I, _LL, _I, _P, _P, _P, _P, _P, _P] + [_I] * 7 + [_P, _P, _P, _I, _I, _P]
         lib.shrike_gated_scan_runs.argtypes = [_I, _I, _I]
         lib.shrike_gated_scan_runs.restype = _LL
-        lib.shrike_head_rms.argtypes = [_P, _P, _P, _I, _I, _I, _I, _F, _P, _I, _LL, _I, _I, _P]
+        lib.shrike_head_rms.argtypes = [_P, _P, _P, _I, _I, _I, _I, _F, _P, _I, _LL, _I, _I, _I, _P]
         lib.shrike_head_prep_norms.argtypes = [_P, _I, _LL, _I, _P, _P, _P, _I, _P, _P, _F, _P, _P, _P, _P, _P] + [_I] * 10 + [_P]
         lib.shrike_route_top_scores.argtypes = [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P]
         lib.shrike_act_mul_blocks_at.argtypes = [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P]
-        lib.shrike_route_top_groups.argtypes = [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P, _I, _I, _P]
+        lib.shrike_route_top_groups.argtypes = [_P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I, _I, _P, _I, _I, _I, _P]
         lib.shrike_act_mul_blocks_limits.argtypes = [_P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _F, _P]
         lib.shrike_norm_join.argtypes = [_P, _P, _I, _LL, _P, _P, _F, _P, _P, _F, _P, _I, _I, _I, _P]
         lib.shrike_plain_act.argtypes = [_P, _I, _LL, _I, _P]
         lib.shrike_side_gate.argtypes = [_P, _I, _LL, _P, _I, _I, _I, _P, _P, _I, _I, _I, _I, _P, _I, _P]
         lib.shrike_short_conv_keep.argtypes = [_P, _I, _LL, _I, _P, _P, _P, _I, _I, _I, _I, _P]
         lib.shrike_delta_prep.argtypes = [_P, _I, _LL, _I, _P, _P, _P, _P, _P, _P, _P, _P] + [_I] * 12 + [_F, _F, _I, _P]
-        lib.shrike_delta_scan.argtypes = [_P, _P, _P, _I, _LL, _I, _P, _P, _P, _P, _P, _P] + [_I] * 9 + [_P, _I, _I, _I, _P]
-        lib.shrike_delta_scan_record.argtypes = [_I]
+        lib.shrike_delta_scan.argtypes = ([_P, _I, _LL, _I, _P, _P, _I, _LL, _I, _I, _I, _P, _P, _F, _F, _P, _P, _P, _P] + [_I] * 9
+                                          + [_P, _I, _I, _I, _P])
+        lib.shrike_delta_scan_record.argtypes = [_I, _I]
+        lib.shrike_low_rank.argtypes = [_P, _I, _LL, _I, _I, _P, _I, _I, _I, _P, _I, _I, _P]
+        lib.shrike_sum_norm.argtypes = [_P, _P, _P, _P, _P, _I, _P, _P, _I, _F, _P, _P, _F, _P, _I, _I, _I, _P]
+        lib.shrike_element_gate.argtypes = [_P, _P, _I, _LL, _I, _I, _I, _I, _I, _I, _I, _P]
+        lib.shrike_act_blocks.argtypes = [_P, _P, _I, _I, _I, _I, _I, _I, _P]
         lib.shrike_delta_scan_record.restype = _I
         lib.shrike_delta_scan_block.restype = _I
         for name in ("shrike_decay_scan", "shrike_norm_gate", "shrike_latent_rope_store", "shrike_concat_cast",
                      "shrike_stream_norm", "shrike_short_conv", "shrike_gated_scan", "shrike_head_rms",
                      "shrike_head_prep_norms", "shrike_route_top_scores", "shrike_act_mul_blocks_at",
                      "shrike_route_top_groups", "shrike_act_mul_blocks_limits", "shrike_norm_join", "shrike_plain_act",
-                     "shrike_side_gate", "shrike_short_conv_keep", "shrike_delta_prep", "shrike_delta_scan"):
+                     "shrike_side_gate", "shrike_short_conv_keep", "shrike_delta_prep", "shrike_delta_scan", "shrike_low_rank",
+                     "shrike_sum_norm", "shrike_element_gate", "shrike_act_blocks"):
             getattr(lib, name).restype = _I
         for name in ("shrike_embed_scaled", "shrike_act_mul_limit", "shrike_tanh_norm", "shrike_head_prep",
                      "shrike_matrix_memory_scan", "shrike_matrix_memory_out", "shrike_route_top", "shrike_act_mul_blocks"):
@@ -394,6 +404,49 @@ class CudaOps:
                                           _ptr(row_add), _ptr(weight), eps, _ptr(out), _DTYPE_CODE[out.dtype], count, width,
                                           self._stream()), "norm_join")
 
+    def sum_norm(self, resid, terms, weight, eps, out, rows=None, row_term=None):
+        """resid += sum over `terms` of scale * pending (each `(tensor, scale)`, at most four, the tensor float32 [N, W] or
+        a K-split stack [P, N, W]), then out = resid / rms(resid) * weight.  `row_term` (x, factors, scale), x [N, W] in the
+        type of `out` and factors float32 [N] (a column of an array will do): scale * factors[n] * x[n] is added too; x may be `out` itself
+        when no rows are gathered.  With `rows` (int32 [R]) only out[r] for row rows[r] is written, the residual stays."""
+        _dense(resid, torch.float32, "residual")
+        _dense(weight, torch.float32, "norm weight")
+        n, width = resid.shape
+        if len(terms) > 4:
+            raise KernelError("sum_norm takes at most four pending sums")
+        data, partials, strides, scales = self._terms(terms, n, width)
+        count = n
+        if rows is not None:
+            _dense(rows, torch.int32, "rows")
+            count = rows.shape[0]
+        if tuple(out.shape) != (count, width) or not out.is_contiguous():
+            raise KernelError(f"norm output {tuple(out.shape)} does not fit {count} rows of {width}")
+        x = factors = None
+        row_stride, row_scale = 0, 1.0
+        if row_term is not None:
+            x, factors, row_scale = row_term
+            _dense(x, out.dtype, "rows of the activation type")
+            if tuple(x.shape) != (n, width) or tuple(factors.shape) != (n,) or factors.dtype != torch.float32:
+                raise KernelError(f"row term {tuple(x.shape)} with factors {tuple(factors.shape)} beside a residual {tuple(resid.shape)}")
+            row_stride = factors.stride(0)
+        self.launches += 1
+        _check(self.core.shrike_sum_norm(_ptr(resid), data, partials, strides, scales, len(terms), _ptr(x), _ptr(factors), row_stride,
+                                         float(row_scale), _ptr(rows), _ptr(weight), eps, _ptr(out), _DTYPE_CODE[out.dtype], count,
+                                         width, self._stream()), "sum_norm")
+
+    def _terms(self, terms, n, width):
+        """Up to four pending sums as the C arrays a kernel's launcher takes: pointers, slices, strides, scales."""
+        data = (_P * 4)()
+        partials, strides, scales = (_I * 4)(), (_LL * 4)(), (_F * 4)()
+        for index, (tensor, scale) in enumerate(terms):
+            _dense(tensor, torch.float32, "pending sum")
+            if tuple(tensor.shape[-2:]) != (n, width):
+                raise KernelError(f"pending sum {tuple(tensor.shape)} does not fit the residual {(n, width)}")
+            data[index] = tensor.data_ptr()
+            partials[index], strides[index] = self._stack(tensor)
+            scales[index] = scale
+        return data, partials, strides, scales
+
     def gather_norm(self, resid, rows, weight, bias, eps, out, layer_norm=True):
         """out[r] = norm(resid[rows[r]]): the final norm on the wanted rows only."""
         _dense(resid, torch.float32, "residual")
@@ -451,6 +504,19 @@ class CudaOps:
         self.launches += 1
         _check(self.core.shrike_head_scale(_ptr(x), _ptr(gate), self.code, x.shape[0], heads, dim, self._stream()),
                "head_scale")
+
+    def element_gate(self, x, fused, gate_at, heads, vdim):
+        """x[n, h, i] *= sigmoid(fused[n, gate_at + h vdim + i]) for i < vdim, in place: x [N, heads * padded] in the engine's
+        type, `fused` float32 [N, total] or a K-split stack."""
+        _dense(x, self.dtype, "head outputs")
+        _dense(fused, torch.float32, "gate source")
+        partials, stride = self._stack(fused)
+        n, width = x.shape
+        if fused.shape[-2] != n or width % heads:
+            raise KernelError(f"element_gate: x{tuple(x.shape)} for {heads} heads, gates {tuple(fused.shape)}")
+        self.launches += 1
+        _check(self.core.shrike_element_gate(_ptr(x), _ptr(fused), partials, stride, fused.shape[-1], gate_at, self.code, n, heads,
+                                             vdim, width // heads, self._stream()), "element_gate")
 
     def linear(self, x, w, out, bias=None, allow_partials=False):
         """x[N, K] @ w[O, K]^T (+ bias) into `out` [N, O] (float32 or the activation type).
@@ -772,7 +838,7 @@ class CudaOps:
                "gemm_tcgen05")
         return True
 
-    PLAIN_ACTIVATIONS = {"relu2": 1}   # activations of an ungated feed-forward: the codes the kernels take
+    PLAIN_ACTIVATIONS = {"relu2": 1, "gelu": 2}   # activations of an ungated feed-forward: the codes the kernels take
 
     def linear_act(self, x, w, out, activation="relu2"):
         """act(x w^T) into `out` [N, O] in the engine's type; for few tokens in bfloat16 the activation is applied inside
@@ -822,15 +888,7 @@ class CudaOps:
         if len(terms) > 4 or len(norms) > 2:
             raise KernelError("tanh_norm takes at most four pending sums and two norms")
         count = rows.shape[0] if rows is not None else n
-        data = (_P * 4)()
-        partials, strides, scales = (_I * 4)(), (_LL * 4)(), (_F * 4)()
-        for index, (tensor, scale) in enumerate(terms):
-            _dense(tensor, torch.float32, "pending sum")
-            if tuple(tensor.shape[-2:]) != (n, width):
-                raise KernelError(f"pending sum {tuple(tensor.shape)} does not fit the residual {tuple(resid.shape)}")
-            data[index] = tensor.data_ptr()
-            partials[index], strides[index] = self._stack(tensor)
-            scales[index] = float(scale)
+        data, partials, strides, scales = self._terms(terms, n, width)
         alpha, weight, bias, out = (_F * 2)(), (_P * 2)(), (_P * 2)(), (_P * 2)()
         out_code = 0
         for index, (a, w, b, o) in enumerate(norms):
@@ -1023,13 +1081,15 @@ class CudaOps:
             torch.bmm(a, w.transpose(1, 2), out_dtype=torch.float32, out=target)
 
     def route_top(self, x, router, shared_gate, weights, top, renorm_eps, scoring="softmax", renormalise=True, correction=None,
-                  groups=None):
+                  groups=None, identity=0):
         """weights [N, E (+ 1)] float32: softmax(router x) over all E experts in 32-bit, the `top` largest
         divided by their sum (+ renorm_eps), 0 elsewhere; a last column, when there is one, holds
         sigmoid(shared_gate . x) (1 when `shared_gate` is None).  `scoring` "sigmoid": an expert's score is the
         sigmoid of its own logit; `renormalise` False: the chosen keep their scores as they are.  `correction` (float32
         [E]) is added to the scores for the choice alone; `groups` (count, keep): only experts of the `keep` best of `count`
-        equal groups of neighbours, by each group's largest choice score, can be chosen."""
+        equal groups of neighbours, by each group's largest choice score, can be chosen.  `identity`: the last so many of the E
+        are identity experts, which have no column of their own: the last column (behind a shared expert's) holds the sum of
+        what they are given."""
         if correction is not None:
             _dense(correction, torch.float32, "choice correction")
             if correction.numel() != router.shape[0]:
@@ -1042,7 +1102,19 @@ class CudaOps:
         _check(self.core.shrike_route_top_groups(_ptr(x), self.code, _ptr(router), _ptr(shared_gate), _ptr(weights), x.shape[0],
                                                  x.shape[1], router.shape[0], top, weights.shape[1], renorm_eps,
                                                  int(scoring == "sigmoid"), int(bool(renormalise)), _ptr(correction), count, keep,
-                                                 self._stream()), "route_top")
+                                                 identity, self._stream()), "route_top")
+
+    def act_blocks(self, x, weights, experts, each, activation):
+        """x [N, experts * each] in place, in the engine's type: x[n, c] = act(x[n, c]) * weights[n, c // each], an ungated
+        expert's activation times its weight; a column whose weight is 0 becomes exactly 0."""
+        _dense(x, self.dtype, "experts' columns")
+        _dense(weights, torch.float32, "expert weights")
+        n, inter = x.shape
+        if inter != experts * each or weights.shape[0] != n:
+            raise KernelError(f"act_blocks: x{tuple(x.shape)} weights{tuple(weights.shape)} for {experts} experts of {each}")
+        self.launches += 1
+        _check(self.core.shrike_act_blocks(_ptr(x), _ptr(weights), self.code, n, experts, each, weights.shape[1],
+                                           self.PLAIN_ACTIVATIONS[activation], self._stream()), "act_blocks")
 
     def act_mul_blocks(self, gate_up, weights, out, experts, each, activation="silu", limit=None, weight_on="output",
                        shared_limit=None):
@@ -1147,9 +1219,10 @@ class CudaOps:
             _ptr(out), num_seqs, num_heads, dim, vdim, state.shape[-1], state.shape[0], run, _ptr(run_state), _ptr(run_decay),
             _ptr(run_first), runs, int(self.dtype == torch.bfloat16), self._stream()), "gated_scan")
 
-    def head_rms(self, x, weight, eps, out, heads, gate_source=None, gate_at=0):
+    def head_rms(self, x, weight, eps, out, heads, gate_source=None, gate_at=0, gate="sigmoid"):
         """out[n, h, :] = x[n, h, :] / sqrt(mean(x[n, h, :]^2) + eps) * weight for x float32 [N, heads * size]; with
-        `gate_source` (float32 [N, total] or a K-split stack) times the sigmoid of its columns from `gate_at` on."""
+        `gate_source` (float32 [N, total] or a K-split stack) times the sigmoid (`gate` "silu": the SiLU) of its columns from
+        `gate_at` on."""
         _dense(x, torch.float32, "head outputs")
         n, width = x.shape
         partials, stride, gate_width = 1, 0, 0
@@ -1159,23 +1232,25 @@ class CudaOps:
             gate_width = gate_source.shape[-1]
         self.launches += 1
         _check(self.core.shrike_head_rms(_ptr(x), _ptr(weight), _ptr(out), _DTYPE_CODE[out.dtype], n, heads, width // heads, eps,
-                                         _ptr(gate_source), partials, stride, gate_width, gate_at, self._stream()), "head_rms")
+                                         _ptr(gate_source), partials, stride, gate_width, gate_at, int(gate == "silu"),
+                                         self._stream()), "head_rms")
 
-    # ---- a delta rule with a decay per key channel -------------------------------------------------------
+    # ---- recurrences whose matrix state decays per key channel or per head -------------------------------
     def delta_prep(self, fused, taps, conv_state, q_start, state_slot, seq_of_token, mixed, beta, low, num_seqs, num_heads,
                    num_kv_heads, dim, vdim, beta_at, low_at, unit_eps, longest=0):
         """A fused projection ([N, total] float32 or a K-split stack) whose first columns are q (G dim) | k (G dim) | v (H
         vdim): a causal convolution over time per channel (`taps` [channels, T]; the T - 1 values before a portion's first
         token from `conv_state` [slots, T - 1, channels], which is left holding the portion's last ones), a SiLU, q and k
         per head over sqrt(sum of squares + unit_eps), q times dim^(-1/2), into `mixed` [N, channels]; the sigmoid of the H
-        columns from `beta_at` into `beta`; the columns from `low_at` cast into `low`.  `longest`: the most new tokens a
+        columns from `beta_at` into `beta`; the columns from `low_at` cast into `low` (None: no such columns).  `longest`: the most new tokens a
         sequence of the batch brings (the batch's shape; 0: not known)."""
         _dense(fused, torch.float32, "fused projection")
         _dense(taps, torch.float32, "convolution taps")
         _dense(conv_state, torch.float32, "convolution state")
         _dense(mixed, torch.float32, "q, k and v")
         _dense(beta, torch.float32, "beta")
-        _dense(low, self.dtype, "low-rank rows")
+        if low is not None:
+            _dense(low, self.dtype, "low-rank rows")
         partials, stride = self._stack(fused)
         n, total = fused.shape[-2], fused.shape[-1]
         channels, count = taps.shape
@@ -1187,31 +1262,39 @@ class CudaOps:
         _check(self.core.shrike_delta_prep(
             _ptr(fused), partials, stride, total, _ptr(taps), _ptr(conv_state), _ptr(q_start), _ptr(state_slot),
             _ptr(seq_of_token), _ptr(mixed), _ptr(beta), _ptr(low), self.code, n, num_heads, num_kv_heads, dim, vdim, count,
-            beta_at, low_at, low.shape[1], num_seqs, conv_state.shape[0], unit_eps, float(dim) ** -0.5, int(longest),
+            beta_at, low_at, 0 if low is None else low.shape[1], num_seqs, conv_state.shape[0], unit_eps, float(dim) ** -0.5, int(longest),
             self._stream()), "delta_prep")
 
     DELTA_BLOCKS_FROM = 16            # a sequence that brings at least this many tokens goes eight tokens at a time
     DELTA_SCRATCH_FLOATS = 128 << 20   # at most 512 MiB of what the blocks hand to the walk: heads take turns beyond
 
     def delta_scan(self, mixed, beta, gates, rate, bias, state, q_start, state_slot, out, num_seqs, num_heads, num_kv_heads,
-                   dim, vdim, q_lens=None, early_state=False):
-        """The delta rule over the batch's new tokens, per value head h with q/k head h // (H / G) of `mixed` (as
-        `delta_prep` leaves it): S <- diag(g) S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q, with g =
-        exp(-rate[h] softplus(z + bias)), z column h dim + d of `gates` ([N, at least H dim] float32 or a K-split stack).
-        `state` float32 [slots, H, at least dim * vdim, a multiple of four] is read and left updated for the slots
+                   dim, vdim, q_lens=None, early_state=False, gate_at=0, per_head=False, sign=1.0, q_scale=1.0):
+        """The delta rule over the batch's new tokens, per value head h with q/k head h // (H / G) of `mixed` (its first columns
+        as `delta_prep` leaves them; q times `q_scale`): S <- diag(g) S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q, with g =
+        exp(-rate[h] softplus(sign (z + bias))), z column gate_at + h dim + d of `gates` (float32 [N, width] or a K-split
+        stack), or column gate_at + h with `per_head` (one decay a head).  `beta` None: no delta rule, u = v.  `bias` may be
+        None.  `state` float32 [slots, H, at least dim * vdim, a multiple of four] is read and left updated for the slots
         `state_slot` names (-1: zeros out, nothing kept); `out` float32 [N, H * vdim].  `q_lens` (the batch's lengths, host):
         longer portions go eight tokens at a time, with the same result up to the order of the sums; without it every
-        sequence walks token by token.  `early_state`: the states were last written by an earlier step (whose kernels have
-        finished), not merely by an earlier launch; single tokens then read them while the kernel before this one runs."""
+        sequence walks token by token, and `mixed` may be a K-split stack (see `delta_walks`).  `early_state`: the states were
+        last written by an earlier step (whose kernels have finished), not merely by an earlier launch; single tokens then
+        read them while the kernel before this one runs."""
         for name, tensor in (("q, k and v", mixed), ("beta", beta), ("gates", gates), ("rate", rate), ("bias", bias),
                              ("state", state), ("scan output", out)):
-            _dense(tensor, torch.float32, name)
+            if tensor is not None:
+                _dense(tensor, torch.float32, name)
         partials, stride = self._stack(gates)
-        if state.dim() != 3 or state.shape[1] != num_heads or state.shape[2] < dim * vdim or bias.numel() != num_heads * dim:
+        mixed_partials, mixed_stride = self._stack(mixed)
+        each = 1 if per_head else dim
+        if (state.dim() != 3 or state.shape[1] != num_heads or state.shape[2] < dim * vdim
+                or (bias is not None and bias.numel() != num_heads * each)):
             raise KernelError(f"state {tuple(state.shape)} does not fit {num_heads} heads of {dim} x {vdim}")
         blocks, records, head_count, shorter = 0, None, 0, True
-        record = self.core.shrike_delta_scan_record(dim) if q_lens is not None and max(q_lens) >= self.DELTA_BLOCKS_FROM else 0
+        record = 0 if self.delta_walks(dim, q_lens) else self.core.shrike_delta_scan_record(dim, int(beta is not None))
         if record:
+            if mixed_partials > 1:
+                raise KernelError("delta_scan: longer portions take q, k and v as one array, not as a stack")
             size = self.core.shrike_delta_scan_block()
             blocks = sum(-(-length // size) for length in q_lens if length >= self.DELTA_BLOCKS_FROM)
             shorter = min(q_lens) < self.DELTA_BLOCKS_FROM
@@ -1224,10 +1307,28 @@ class CudaOps:
             records = self._delta_scratch
         self.launches += int(shorter) + (2 * -(-num_heads // head_count) if blocks else 0)
         _check(self.core.shrike_delta_scan(
-            _ptr(mixed), _ptr(beta), _ptr(gates), partials, stride, gates.shape[-1], _ptr(rate), _ptr(bias), _ptr(state),
-            _ptr(q_start), _ptr(state_slot), _ptr(out), num_seqs, num_heads, num_kv_heads, dim, vdim, state.shape[2],
-            state.shape[0], self.DELTA_BLOCKS_FROM if blocks else 0, int(shorter), _ptr(records), blocks, head_count,
-            int(bool(early_state)), self._stream()), "delta_scan")
+            _ptr(mixed), mixed_partials, mixed_stride, mixed.shape[-1], _ptr(beta), _ptr(gates), partials, stride, gates.shape[-1],
+            gate_at, each, _ptr(rate), _ptr(bias), float(sign), float(q_scale), _ptr(state), _ptr(q_start), _ptr(state_slot), _ptr(out),
+            num_seqs, num_heads, num_kv_heads, dim, vdim, state.shape[2], state.shape[0], self.DELTA_BLOCKS_FROM if blocks else 0,
+            int(shorter), _ptr(records), blocks, head_count, int(bool(early_state)), self._stream()), "delta_scan")
+
+    def delta_walks(self, dim, q_lens) -> bool:
+        """Whether `delta_scan` walks every sequence of such a batch token by token, so that its input may be a stack."""
+        return q_lens is None or max(q_lens) < self.DELTA_BLOCKS_FROM or not self.core.shrike_delta_scan_record(dim, 1)
+
+    def low_rank(self, fused, at, rank, matrix, out):
+        """out [N, C] = matrix (fused's `rank` columns from `at` on), in float32: the second half of a low-rank product.
+        `fused` float32 [N, total] or a K-split stack, `matrix` [C, padded] in the engine's type, zeros behind its rank."""
+        _dense(fused, torch.float32, "fused projection")
+        _dense(matrix, self.dtype, "low-rank matrix")
+        _dense(out, torch.float32, "low-rank product")
+        partials, stride = self._stack(fused)
+        n, columns = out.shape
+        if fused.shape[-2] != n or matrix.shape[0] != columns:
+            raise KernelError(f"low_rank: fused {tuple(fused.shape)} matrix {tuple(matrix.shape)} out {tuple(out.shape)}")
+        self.launches += 1
+        _check(self.core.shrike_low_rank(_ptr(fused), partials, stride, fused.shape[-1], at, _ptr(matrix), self.code, matrix.shape[1],
+                                         rank, _ptr(out), n, columns, self._stream()), "low_rank")
 
     def sample(self, logits, temperature, top_p, seeds, out):
         _dense(logits, torch.float32, "logits")

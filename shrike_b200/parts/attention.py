@@ -194,7 +194,7 @@ class SharedKeyValueAttention:
 class GatedHeadAttention:
     """Grouped-query attention with the options of `GatedHeadAttentionSpec`: biases, a root-mean-square
     norm of q and k per head with one weight for all heads, a rotation of each head's first
-    dimensions, a window or chunks of positions, an output gate per head.  q, k, v and the gate are
+    dimensions, a window or chunks of positions, an output gate per head or per element.  q, k, v and the gate are
     one matrix product; one kernel turns its 32-bit result into queries and cache rows; the paged
     attention kernels run as they are (a chunk is handed to them as a negative window).  Keys and
     values share the pages' head size, the next multiple of 16 above the larger of the two; the
@@ -233,6 +233,8 @@ class GatedHeadAttention:
             params["v_conv.weight"] = ParamSpec((v_out, spec.conv), "conv")
         if spec.head_gate:
             params["gate.weight"] = ParamSpec((spec.num_heads, spec.width), "matrix")
+        if getattr(spec, "element_gate", False):
+            params["gate.weight"] = ParamSpec((spec.num_heads * spec.value_dim, spec.width), "matrix")
         if getattr(spec, "sink", False):
             params["sink"] = ParamSpec((spec.num_heads,), "sink")
         return params
@@ -270,7 +272,9 @@ class GatedHeadAttention:
         if self.own_kv:
             rows += [tensors.pop("k_proj.weight"), tensors.pop("v_proj.weight")]
         self.channels = sum(r.shape[0] for r in rows)   # what a convolution runs over: q, k and v
-        if spec.head_gate:
+        self.element_gate = getattr(spec, "element_gate", False)
+        self.gate_at = self.channels   # the gates' first column of the fused product
+        if spec.head_gate or self.element_gate:
             rows.append(tensors.pop("gate.weight").to(rows[0].dtype))
         extra = -sum(r.shape[0] for r in rows) % 16   # rows of zeros: output rows of a whole number of 64 bytes
         if extra:
@@ -357,6 +361,8 @@ class GatedHeadAttention:
         )
         if gate is not None:
             ops.head_scale(attn, gate, spec.num_heads, self.padded)
+        if self.element_gate:
+            ops.element_gate(attn, fused, self.gate_at, spec.num_heads, spec.value_dim)
         delta = rt.buffer("mixer_delta", (n, spec.width), torch.float32)
         return ops.linear(attn, self.w_o, delta, bias=self.b_o, allow_partials=True)
 

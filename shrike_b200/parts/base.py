@@ -75,7 +75,8 @@ class ParamSpec:
     init: "matrix" | "table" (N(0, 0.02)), "bias" (N(0, 0.02)), "norm" (1 + N(0, 0.1)),
     "around_zero" (N(0, 0.1)), "sink" (N(0, 1)), "mix" ([W, 2 W]: identity | 0, plus N(0, 0.02)),
     "conv" (N(0, 0.4)), "unit_interval" (sigmoid of N(0, 1)), "stream_mix" ([S, S]: identity plus N(0, 0.15)),
-    "decay_rate" (N(0, 0.5)), "decay_bias" (N(-3, 1): softplus of it spans slow and quick decays), "choice" (N(0, 0.01)),
+    "decay_rate" (N(0, 0.5)), "decay_bias" (N(-3, 1): softplus of it spans slow and quick decays), "gate_bias" (N(2, 2): a
+    sigmoid of it from half open to nearly one), "choice" (N(0, 0.01)),
     "side_table" (N(0, 1)).
 
     `free`: axes whose extent the model's tensor gives (the rank of a low-rank product, which no configuration key
@@ -121,7 +122,7 @@ class StateNeed:
 
 class PendingSum:
     """Branch outputs that are not yet added to the residual: `terms`, a list of (tensor, scale), each
-    tensor float32 [N, W] or a K-split stack [P, N, W].  A block whose branches run side by side hands
+    tensor float32 [N, W] or a K-split stack [P, N, W] (or a `RowScaled`).  A block whose branches run side by side hands
     one on as its `delta`; a norm that takes it adds every term in the kernel that norms the sum."""
 
     __slots__ = ("terms",)
@@ -137,6 +138,17 @@ class PendingSum:
         if isinstance(delta, PendingSum):
             return [(tensor, s * scale) for tensor, s in delta.terms]
         return [(delta, scale)]
+
+
+class RowScaled:
+    """A pending term that is not an array of its own: rows `x` [N, W] in the activation type, each times its own factor
+    (`factors`, float32 [N], a column of an array will do; most may be zero).  It stands in a `PendingSum` as the tensor of a
+    term; the RMS norm's kernel forms the product as it adds it."""
+
+    __slots__ = ("x", "factors")
+
+    def __init__(self, x, factors):
+        self.x, self.factors = x, factors
 
 
 class PendingNorm:

@@ -1,8 +1,8 @@
 """Residual blocks.
 
-`ParallelBlock`: both branches read the same residual, x += mixer(norm1(x)) + ff(norm2(x)).  The two
-norms come from one pass over the row where the norm part offers that (`add_norm_pair`), and the
-branch outputs stay pending (a `PendingSum`): the next norm kernel adds them, so the sum costs no pass.
+`ParallelBlock`: both branches read the same residual, x += scale * (mixer(norm1(x)) + ff(norm2(x))).  The two
+norms come from one pass over the row where the norm part offers that (`add_norm_pair`); a feed-forward without a norm of
+its own reads what the mixer reads.  The branch outputs stay pending (a `PendingSum`): the next norm kernel adds them, so the sum costs no pass.
 
 `BranchNormBlock`: the norm sits on a branch's OUTPUT, x += norm(mixer(x)); x += norm(ffn(x)), and both
 branches read x itself; the feed-forward may be absent.  The residual sum is 32-bit; a 16-bit engine
@@ -94,18 +94,23 @@ class BranchNormBlock:
 class ParallelBlock:
     capture_safe = True
 
-    def __init__(self, mixer, mixer_norm, feed_forward=None, feed_forward_norm=None):
-        if (feed_forward is None) != (feed_forward_norm is None):
-            raise ValueError("a feed-forward and its norm come together")
+    def __init__(self, mixer, mixer_norm, feed_forward=None, feed_forward_norm=None, scale=1.0):
+        if feed_forward is None and feed_forward_norm is not None:
+            raise ValueError("a feed-forward's norm without a feed-forward")
         self.mixer = mixer
         self.mixer_norm = mixer_norm
         self.feed_forward = feed_forward
         self.feed_forward_norm = feed_forward_norm
+        self.scale = float(scale)   # what both branches are multiplied by as they join the residual
 
     def forward(self, resid, delta, ctx, run):
-        if self.feed_forward is None:
+        scale = self.scale
+        if self.feed_forward_norm is None:   # one norm; both branches (or the mixer alone) read it
             hidden = self.mixer_norm.add_norm(resid, delta)
-            return resid, PendingSum(PendingSum.of(self.mixer.forward(hidden, ctx, run)))
+            terms = PendingSum.of(self.mixer.forward(hidden, ctx, run), scale)
+            if self.feed_forward is not None:
+                terms += PendingSum.of(self.feed_forward.forward(hidden, ctx), scale)
+            return resid, PendingSum(terms)
         pair = getattr(self.mixer_norm, "add_norm_pair", None)
         if pair is not None:
             for_mixer, for_ffn = pair(resid, delta, self.feed_forward_norm)
@@ -114,7 +119,7 @@ class ParallelBlock:
             for_ffn = self.feed_forward_norm.add_norm(resid, None, "normed_b")
         mixed = self.mixer.forward(for_mixer, ctx, run)
         fed = self.feed_forward.forward(for_ffn, ctx)
-        return resid, PendingSum(PendingSum.of(mixed) + PendingSum.of(fed))
+        return resid, PendingSum(PendingSum.of(mixed, scale) + PendingSum.of(fed, scale))
 
 
 class SandwichBlock:

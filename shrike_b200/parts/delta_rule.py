@@ -1,4 +1,6 @@
-"""A delta rule whose state decays per key channel (gated delta rule with a vector of decays).
+"""Delta rules whose state decays: per key channel (`ChannelDelta`) or by one number a head (`HeadDelta`).
+
+`ChannelDelta`, a gated delta rule with a vector of decays.
 
 q and k (heads of `head_dim`) and v (heads of `value_dim`) are projections of x, each behind a causal convolution over
 time per channel and a SiLU; q and k are unit vectors per head, q also times head_dim^(-1/2).  Per value head, with
@@ -16,6 +18,10 @@ request's state, named "conv"); a second product gives decays and output gates f
 matrix over both); `delta_scan` runs the recurrence on the request's float32 state slot
 `[heads, head_dim * value_dim (rounded up to four)]`; `head_rms` norms, gates and casts.  Both states are zeroed by the
 step function when the request is opened.  The ranks of the low-rank products come from the model's tensors.
+
+`HeadDelta`, the same rule with one decay a head, g = exp(-exp(A_log) softplus(Wa x + dt_bias)), and an output gate
+silu(Wg x): decay and gate columns are part of the one product, whose 32-bit result the scan and the head norm read, so
+there is no second product.
 """
 
 from __future__ import annotations
@@ -134,3 +140,72 @@ class ChannelDelta:
 
 
 register_part("mixer", "channel_delta", ChannelDelta)
+
+
+class HeadDelta:
+    capture_safe = True   # it reads the batch's metadata on the device only and leaves rows alone whose state slot is -1
+
+    @staticmethod
+    def parameters(spec) -> dict[str, ParamSpec]:
+        qk, v = spec.num_kv_heads * spec.head_dim, spec.num_heads * spec.value_dim
+        return {
+            "q_proj.weight": ParamSpec((qk, spec.width), "matrix"),
+            "k_proj.weight": ParamSpec((qk, spec.width), "matrix"),
+            "v_proj.weight": ParamSpec((v, spec.width), "matrix"),
+            "q_conv.weight": ParamSpec((qk, spec.conv), "conv"),
+            "k_conv.weight": ParamSpec((qk, spec.conv), "conv"),
+            "v_conv.weight": ParamSpec((v, spec.conv), "conv"),
+            "beta.weight": ParamSpec((spec.num_heads, spec.width), "matrix"),
+            "decay.weight": ParamSpec((spec.num_heads, spec.width), "matrix"),
+            "decay_log": ParamSpec((spec.num_heads,), "decay_rate"),
+            "decay_bias": ParamSpec((spec.num_heads,), "decay_bias"),
+            "gate.weight": ParamSpec((v, spec.width), "matrix"),
+            "norm.weight": ParamSpec((spec.value_dim,), "norm"),
+            "o_proj.weight": ParamSpec((spec.width, v), "matrix"),
+        }
+
+    cache_needs = staticmethod(ChannelDelta.cache_needs)   # the same two states: S, and the convolution's last inputs
+
+    def __init__(self, spec, tensors, ops, runtime):
+        self.spec, self.ops, self.runtime = spec, ops, runtime
+        self.channels = ChannelDelta.channels(spec)
+        self.out_width = spec.num_heads * spec.value_dim
+        # rows: q | k | v | gate | beta | decay
+        rows = [tensors.pop(f"{name}.weight") for name in ("q_proj", "k_proj", "v_proj", "gate")]
+        rows += [tensors.pop(f"{name}.weight").to(rows[0].dtype) for name in ("beta", "decay")]
+        self.gate_at = self.channels
+        self.beta_at = self.gate_at + self.out_width
+        self.decay_at = self.beta_at + spec.num_heads
+        self.w_fused = padded_rows(torch.cat(rows))
+        self.total = self.w_fused.shape[0]
+        self.taps = torch.cat([tensors.pop(f"{name}_conv.weight") for name in ("q", "k", "v")]).to(torch.float32).contiguous()
+        self.no_state = torch.zeros(1, 0, self.channels, dtype=torch.float32, device=runtime.device)
+        self.rate = tensors.pop("decay_log").to(torch.float32).exp().contiguous()   # what softplus(.) is multiplied by
+        self.bias = tensors.pop("decay_bias").to(torch.float32).contiguous()
+        self.norm_weight = tensors.pop("norm.weight").to(torch.float32).contiguous()
+        self.w_o = tensors.pop("o_proj.weight").contiguous()
+
+    def forward(self, x, ctx, run):
+        spec, rt, ops = self.spec, self.runtime, self.ops
+        if not run.writes_cache:
+            raise NotImplementedError("a delta rule owns its state: no run can read another run's")
+        n = x.shape[0]
+        fused = rt.buffer("memory_in", (n, self.total), torch.float32)
+        fused = ops.linear(x, self.w_fused, fused, allow_partials=True)
+        mixed = rt.buffer("delta_mixed", (n, self.channels), torch.float32)
+        beta = rt.buffer("delta_beta", (n, spec.num_heads), torch.float32)
+        conv_state = ctx.storage.state[(run.cache, "conv")] if spec.conv > 1 else self.no_state
+        ops.delta_prep(fused, self.taps, conv_state, ctx.q_start, ctx.state_slot, ctx.seq_of_token, mixed, beta, None,
+                       ctx.num_seqs, spec.num_heads, spec.num_kv_heads, spec.head_dim, spec.value_dim, self.beta_at,
+                       0, spec.unit_eps, longest=ctx.max_q_len)
+        scanned = rt.buffer("memory_num", (n, self.out_width), torch.float32)
+        ops.delta_scan(mixed, beta, fused, self.rate, self.bias, ctx.storage.state[run.cache], ctx.q_start, ctx.state_slot,
+                       scanned, ctx.num_seqs, spec.num_heads, spec.num_kv_heads, spec.head_dim, spec.value_dim, q_lens=ctx.q_lens,
+                       early_state=True, gate_at=self.decay_at, per_head=True)   # only earlier steps wrote a run's own state
+        out = rt.buffer("memory_out", (n, self.out_width), rt.act_dtype)
+        ops.head_rms(scanned, self.norm_weight, spec.eps, out, spec.num_heads, gate_source=fused, gate_at=self.gate_at, gate="silu")
+        delta = rt.buffer("memory_delta", (n, spec.width), torch.float32)
+        return ops.linear(out, self.w_o, delta, allow_partials=True)
+
+
+register_part("mixer", "head_delta", HeadDelta)

@@ -18,7 +18,8 @@ from .base import ParamSpec, register_part
 # gelu_tanh(z) = 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)));
 # clamped_swish with limit L: g <- min(g, L), u <- clamp(u, -L, L), then g sigmoid(1.702 g) (u + 1) in place of act(g) u
 ACTIVATIONS = ("silu", "gelu_tanh", "clamped_swish")
-PLAIN_ACTIVATIONS = ("relu2",)   # act(z) of an ungated feed-forward: relu2 is max(z, 0)^2
+# act(z) of an ungated feed-forward: relu2 is max(z, 0)^2, gelu z (1 + erf(z / sqrt(2))) / 2
+PLAIN_ACTIVATIONS = ("relu2", "gelu")
 
 
 class GatedMLP:

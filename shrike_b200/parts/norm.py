@@ -4,7 +4,8 @@ y = x * rsqrt(mean(x^2) + eps) * w with a plain weight, all in 32-bit, one
 rounding at the end (shrike/models/qwen.py:64-74).  The residual stream is kept in
 float32; `add_norm` first adds the pending branch output to it, so the sum that
 Azimml/shrike does in the model dtype (qwen.py:148-149) is a 32-bit sum here and
-costs no pass of its own.
+costs no pass of its own.  A `PendingSum` (several branch outputs, a scale each, rows with a factor each) is added
+the same way by the kernel that norms the sum.
 
 Two ways of sitting in a layer.  Before a branch (`add_norm`): the pending branch output is added to
 the residual and the sum is normed.  On a branch's output (`norm_add`): the branch output is normed
@@ -18,11 +19,12 @@ from __future__ import annotations
 
 import torch
 
-from .base import ParamSpec, PendingNorm, PendingSum, register_part
+from .base import ParamSpec, PendingNorm, PendingSum, RowScaled, register_part
 
 
 class RMSNorm:
     capture_safe = True   # forward() launches the same kernels for the same batch shape, whatever the positions
+    MAX_TERMS = 4   # pending sums one launch of the kernel adds
 
     @staticmethod
     def parameters(spec) -> dict[str, ParamSpec]:
@@ -42,6 +44,9 @@ class RMSNorm:
         if isinstance(delta, PendingNorm):
             self.ops.norm_join(resid, delta.branch, delta.norm.weight, delta.norm.spec.eps, delta.row_add, self.weight,
                                self.spec.eps, out)
+        elif isinstance(delta, PendingSum):
+            terms, row_term = self._flush(resid, delta, out)
+            self.ops.sum_norm(resid, terms, self.weight, self.spec.eps, out, row_term=row_term)
         else:
             self.ops.add_rmsnorm(resid, delta, self.weight, self.spec.eps, out)
         return out
@@ -52,9 +57,30 @@ class RMSNorm:
             self.ops.norm_join(resid, delta.branch, delta.norm.weight, delta.norm.spec.eps, delta.row_add, self.weight,
                                self.spec.eps, out, rows=rows)
             return out
+        if isinstance(delta, PendingSum):
+            scratch = self.runtime.buffer("normed_flush", tuple(resid.shape), self.runtime.act_dtype) if self._over(delta) else None
+            terms, row_term = self._flush(resid, delta, scratch)
+            self.ops.sum_norm(resid, terms, self.weight, self.spec.eps, out, rows=rows, row_term=row_term)
+            return out
         self.ops.gather_add_rmsnorm(resid, delta, rows, self.weight, self.spec.eps, out)
         return out
 
+    @classmethod
+    def _over(cls, delta) -> bool:
+        row_terms = sum(isinstance(tensor, RowScaled) for tensor, _ in delta.terms)
+        return len(delta.terms) - row_terms > cls.MAX_TERMS or row_terms > 1
+
+    def _flush(self, resid, delta, scratch):
+        """The pending terms one launch can take, (sums, the row term or None); what is over is added to the residual first."""
+        terms = [(tensor, scale) for tensor, scale in delta.terms if not isinstance(tensor, RowScaled)]
+        row_terms = [(tensor.x, tensor.factors, scale) for tensor, scale in delta.terms if isinstance(tensor, RowScaled)]
+        if self._over(delta) and any(x.data_ptr() == scratch.data_ptr() for x, _, _ in row_terms):
+            raise NotImplementedError("rows that are still to be added lie where the norm's output goes")
+        while len(terms) > self.MAX_TERMS or len(row_terms) > 1:
+            self.ops.sum_norm(resid, terms[: self.MAX_TERMS], self.weight, self.spec.eps, scratch,
+                              row_term=row_terms.pop() if row_terms else None)
+            terms = terms[self.MAX_TERMS:]
+        return terms, (row_terms[0] if row_terms else None)
 
     def norm_add(self, resid, branch, out_name="hidden"):
         """resid += norm(branch) in 32-bit; returns the new residual in the activation type."""

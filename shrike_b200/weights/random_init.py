@@ -45,6 +45,8 @@ def random_tensor(name: str, spec, seed: int, device="cpu", dtype=torch.float32)
         values = 0.5 * values
     elif spec.init == "decay_bias":      # softplus of it: steps from about 0.01 to 1, slow and quick decays side by side
         values = values - 3.0
+    elif spec.init == "gate_bias":       # what a sigmoid gate is shifted by: half open to nearly one
+        values = 2.0 + 2.0 * values
     elif spec.init == "choice":          # what a router's choice is corrected by, of the order of the scores' differences
         values = 0.01 * values
     elif spec.init == "unit_interval":   # a bound inside (0, 1)

@@ -129,7 +129,7 @@ class EmulatedOps:
             held[:, D * Dv + D] = m
 
     def route_top(self, x, router, shared_gate, weights, top, renorm_eps, scoring="softmax", renormalise=True,
-                  correction=None, groups=None):
+                  correction=None, groups=None, identity=0):
         logits = x.float() @ router.T
         scores = torch.sigmoid(logits) if scoring == "sigmoid" else torch.softmax(logits, -1)
         choice = logits if correction is None and groups is None else scores   # the logits order the experts as either score does
@@ -142,10 +142,13 @@ class EmulatedOps:
             choice = choice.masked_fill(shut.repeat_interleave(router.shape[0] // count, 1), float("-inf"))
         _, chosen = torch.topk(choice, top, -1)
         best = scores.gather(1, chosen)
-        weights.zero_()
-        weights[:, : router.shape[0]].scatter_(1, chosen, best / (best.sum(-1, keepdim=True) + renorm_eps) if renormalise else best)
-        if weights.shape[1] > router.shape[0]:
-            weights[:, -1] = 1.0 if shared_gate is None else torch.sigmoid(x.float() @ shared_gate)
+        given = torch.zeros_like(logits).scatter_(1, chosen, best / (best.sum(-1, keepdim=True) + renorm_eps) if renormalise else best)
+        real = router.shape[0] - identity
+        weights[:, :real] = given[:, :real]
+        if weights.shape[1] > real + (identity > 0):
+            weights[:, real] = 1.0 if shared_gate is None else torch.sigmoid(x.float() @ shared_gate)
+        if identity:
+            weights[:, -1] = given[:, real:].sum(-1)
 
     def act_mul_blocks(self, gate_up, weights, out, experts, each, activation="silu", limit=None, weight_on="output",
                        shared_limit=None):
@@ -449,7 +452,7 @@ class EmulatedOps:
                 out[t] = torch.einsum("hdv,hd->hv", S, q).reshape(-1)
             state[slot][:, : D * Dv] = S.reshape(H, -1)
 
-    def head_rms(self, x, weight, eps, out, heads, gate_source=None, gate_at=0):
+    def head_rms(self, x, weight, eps, out, heads, gate_source=None, gate_at=0, gate="sigmoid"):
         shaped = x.float().view(x.shape[0], heads, -1)
         normed = shaped / torch.sqrt(shaped.pow(2).mean(-1, keepdim=True) + eps)
         if weight is not None:
@@ -457,7 +460,8 @@ class EmulatedOps:
         normed = normed.reshape(x.shape)
         if gate_source is not None:
             gates = gate_source.sum(0) if gate_source.dim() == 3 else gate_source
-            normed = normed * torch.sigmoid(gates[:, gate_at: gate_at + x.shape[1]])
+            z = gates[:, gate_at: gate_at + x.shape[1]]
+            normed = normed * (z * torch.sigmoid(z) if gate == "silu" else torch.sigmoid(z))
         out.copy_(normed.to(out.dtype))
 
     def norm_join(self, resid, branch, branch_weight, branch_eps, row_add, weight, eps, out, rows=None):
@@ -481,11 +485,48 @@ class EmulatedOps:
         out.zero_()
         out[:, :dim] = (act * table[ids, first: first + dim].float()).to(out.dtype)
 
-    def linear_act(self, x, w, out, activation="relu2"):
+    @staticmethod
+    def _plain_act(z, activation):
+        if activation == "gelu":
+            return 0.5 * z * (1.0 + torch.erf(z / math.sqrt(2.0)))
         assert activation == "relu2"
+        return torch.relu(z).pow(2)
+
+    def linear_act(self, x, w, out, activation="relu2"):
         z = torch.empty(out.shape, dtype=out.dtype)
         self.linear(x, w, z)
-        out.copy_(torch.relu(z.float()).pow(2).to(out.dtype))
+        out.copy_(self._plain_act(z.float(), activation).to(out.dtype))
+
+    def act_blocks(self, x, weights, experts, each, activation):
+        share = weights[:, :experts].repeat_interleave(each, 1)
+        x.copy_((self._plain_act(x.float(), activation) * share).to(x.dtype))
+
+    def sum_norm(self, resid, terms, weight, eps, out, rows=None, row_term=None):
+        x = resid.clone()
+        for tensor, scale in terms:
+            x += scale * (tensor.sum(0) if tensor.dim() == 3 else tensor)
+        if row_term is not None:
+            own, factors, scale = row_term
+            x += scale * factors[:, None] * own.float()
+        if rows is None:
+            resid.copy_(x)
+        else:
+            x = x[rows.long()]
+        out.copy_(self._norm(x, weight, None, eps, False).to(out.dtype))
+
+    def element_gate(self, x, fused, gate_at, heads, vdim):
+        fused = fused.sum(0) if fused.dim() == 3 else fused
+        n = x.shape[0]
+        view = x.view(n, heads, -1)
+        gates = torch.sigmoid(fused[:, gate_at: gate_at + heads * vdim]).view(n, heads, vdim)
+        view[..., :vdim] = (view[..., :vdim].float() * gates).to(x.dtype)
+
+    def low_rank(self, fused, at, rank, matrix, out):
+        fused = fused.sum(0) if fused.dim() == 3 else fused
+        out.copy_(fused[:, at: at + rank] @ matrix[:, :rank].float().T)
+
+    def delta_walks(self, dim, q_lens):
+        return q_lens is None or max(q_lens) < 16 or dim > 256
 
     def delta_prep(self, fused, taps, conv_state, q_start, state_slot, seq_of_token, mixed, beta, low, num_seqs, num_heads,
                    num_kv_heads, dim, vdim, beta_at, low_at, unit_eps, longest=0):
@@ -501,18 +542,24 @@ class EmulatedOps:
         mixed[:, qk: 2 * qk] = unit(conv[:, qk: 2 * qk].view(n, num_kv_heads, dim)).view(n, qk)
         mixed[:, 2 * qk:] = conv[:, 2 * qk:]
         beta.copy_(torch.sigmoid(fused[:, beta_at: beta_at + num_heads]))
+        if low is None:
+            return
         low.copy_(fused[:, low_at: low_at + low.shape[1]].to(low.dtype))
 
     def delta_scan(self, mixed, beta, gates, rate, bias, state, q_start, state_slot, out, num_seqs, num_heads, num_kv_heads,
-                   dim, vdim, q_lens=None, early_state=False):
-        if gates.dim() == 3:
-            gates = gates.sum(0)
+                   dim, vdim, q_lens=None, early_state=False, gate_at=0, per_head=False, sign=1.0, q_scale=1.0):
+        gates = gates.sum(0) if gates.dim() == 3 else gates
+        if mixed.dim() == 3:
+            assert self.delta_walks(dim, q_lens), "longer portions take q, k and v as one array"
+            mixed = mixed.sum(0)
         n, qk, share = mixed.shape[0], num_kv_heads * dim, num_heads // num_kv_heads
-        step = torch.nn.functional.softplus(gates[:, : num_heads * dim] + bias, threshold=60.0).view(n, num_heads, dim)
-        g = torch.exp(-rate[None, :, None] * step)
-        q = mixed[:, :qk].view(n, num_kv_heads, dim).repeat_interleave(share, 1)
+        each = 1 if per_head else dim
+        z = gates[:, gate_at: gate_at + num_heads * each]
+        step = torch.nn.functional.softplus(sign * (z if bias is None else z + bias), threshold=60.0).view(n, num_heads, each)
+        g = torch.exp(-rate[None, :, None] * step).expand(n, num_heads, dim)
+        q = q_scale * mixed[:, :qk].view(n, num_kv_heads, dim).repeat_interleave(share, 1)
         k = mixed[:, qk: 2 * qk].view(n, num_kv_heads, dim).repeat_interleave(share, 1)
-        v = mixed[:, 2 * qk:].view(n, num_heads, vdim)
+        v = mixed[:, 2 * qk: 2 * qk + num_heads * vdim].view(n, num_heads, vdim)
         out.zero_()
         for s in range(num_seqs):
             slot = int(state_slot[s])
@@ -521,7 +568,7 @@ class EmulatedOps:
             held = state[slot][:, : dim * vdim].reshape(num_heads, dim, vdim).clone()
             for t in range(int(q_start[s]), int(q_start[s + 1])):
                 held = g[t, :, :, None] * held
-                u = beta[t, :, None] * (v[t] - torch.einsum("hdv,hd->hv", held, k[t]))
+                u = v[t] if beta is None else beta[t, :, None] * (v[t] - torch.einsum("hdv,hd->hv", held, k[t]))
                 held = held + k[t, :, :, None] * u[:, None, :]
                 out[t] = torch.einsum("hdv,hd->hv", held, q[t]).reshape(-1)
             state[slot][:, : dim * vdim] = held.reshape(num_heads, -1)
