@@ -236,7 +236,7 @@ def test_delta_scan_takes_heads_in_turns_when_the_scratch_is_bounded():
     q, k, v, beta, z, a_log, bias = delta_inputs(n, heads, heads, dim, vdim, 8)
     mixed = torch.cat([q.reshape(n, -1), k.reshape(n, -1), v.reshape(n, -1)], -1).cuda().contiguous()
     results = []
-    for bound in (ops.DELTA_SCRATCH_FLOATS, 2 * 13 * ops.core.shrike_delta_scan_record(dim)):
+    for bound in (ops.DELTA_SCRATCH_FLOATS, 2 * 13 * ops.core.shrike_delta_scan_record(dim, 1)):
         ops.DELTA_SCRATCH_FLOATS = bound
         state, out = torch.zeros(1, heads, dim * vdim, device="cuda"), torch.empty(n, heads * vdim, device="cuda")
         ops.delta_scan(mixed, beta.cuda(), z.reshape(n, -1).cuda(), a_log.exp().cuda(), bias.cuda(), state,
