@@ -477,7 +477,7 @@ def run_mixed(args) -> dict:
 
     torch.cuda.set_device(0)
     design = getattr(args, "arch", "qwen2")   # the same workload on another decoder at the same widths
-    sadodra = design in ("sadodra", "vupitar", "kavedra", "setotar", "nulazen")
+    sadodra = design in ("sadodra", "vupitar", "kavedra", "setotar", "nulazen", "radilix")
     if sadodra:
         from shrike_b200.shapes import shape_config
 
@@ -752,6 +752,89 @@ def run_case(args) -> dict:
             times.append(start.elapsed_time(stop) * 1e3)
         # a token and head: dim x vdim each of the decay (1 flop), S^T k, k u^T and S^T q (2 flops a multiply-add)
         work = {"bytes": seqs * heads * d * d * 4 * 2 + n * heads * (5 * d + 1) * 4} if single else {"flops": 7.0 * n * heads * d * d}
+    elif args.case in ("head_delta_scan", "head_delta_scan_single", "gla_scan", "gla_scan_single"):
+        # the delta rule with one decay a head (--heads value heads on half as many key heads, default 8) and linear attention
+        # with decays per key channel (default 28 heads), heads of 128 x 128: one prompt of --prefill-tokens tokens, or
+        # --batch sequences one token each
+        single, delta = args.case.endswith("_single"), args.case.startswith("head_delta")
+        count = args.heads or (8 if delta else 28)
+        groups = count // 2 if delta and count % 2 == 0 else count
+        seqs, q_len = (tokens, 1) if single else (1, args.prefill_tokens)
+        n = seqs * q_len
+        width = (2 * groups + count) * d
+        mixed = torch.randn(n, width, device=dev)
+        mixed[:, : 2 * groups * d] = torch.nn.functional.normalize(mixed[:, : 2 * groups * d].view(n, 2 * groups, d), dim=-1).view(n, -1)
+        beta = torch.rand(n, count, device=dev) if delta else None
+        gates = torch.randn(n, count if delta else count * d, device=dev) - (3.0 if delta else -3.0)
+        rate, bias = torch.full((count,), 1.0 if delta else 1 / 16.0, device=dev), torch.zeros(gates.shape[1], device=dev)
+        state = torch.zeros(seqs, count, d * d, device=dev)
+        q_start = torch.arange(seqs + 1, dtype=torch.int32, device=dev) * q_len
+        slots = torch.arange(seqs, dtype=torch.int32, device=dev)
+        out = torch.empty(n, count * d, device=dev)
+        for _ in range(6):
+            keep_busy()
+            start.record()
+            ops.delta_scan(mixed, beta, gates, rate, bias, state, q_start, slots, out, seqs, count, groups, d, d, q_lens=[q_len] * seqs,
+                           per_head=delta, sign=1.0 if delta else -1.0)
+            stop.record()
+            torch.cuda.synchronize()
+            times.append(start.elapsed_time(stop) * 1e3)
+        # a token and head: dim x vdim of the decay (1 flop), k u^T and S^T q, with the delta rule also S^T k (2 flops each)
+        work = {"bytes": seqs * count * d * d * 4 * 2 + n * (width + gates.shape[1] + count * d) * 4} if single else \
+               {"flops": (7.0 if delta else 5.0) * n * count * d * d}
+    elif args.case == "sum_norm":
+        # --batch rows of the 7B width: two pending sums, and rows with a factor each of which a fifth is not zero
+        resid, weight = torch.randn(tokens, h, device=dev), torch.ones(h, device=dev)
+        terms = [(torch.randn(tokens, h, device=dev), 0.6), (torch.randn(tokens, h, device=dev), 0.4)]
+        out = torch.randn(tokens, h, device=dev).to(torch.bfloat16)
+        factors = torch.rand(tokens, device=dev)
+        factors[torch.arange(tokens, device=dev) % 5 > 0] = 0.0
+        for _ in range(6):
+            keep_busy()
+            start.record()
+            ops.sum_norm(resid, terms, weight, 1e-6, out, row_term=(out, factors, 0.6))
+            stop.record()
+            torch.cuda.synchronize()
+            times.append(start.elapsed_time(stop) * 1e3)
+        work = {"bytes": tokens * h * (4 + 2 * 4 + 4 + 2 + 2 / 5)}
+    elif args.case == "element_gate":
+        # --batch rows of 28 heads of 128, gates from a fused q | k | v | gate product
+        x = torch.randn(tokens, heads * d, device=dev).to(torch.bfloat16)
+        fused = torch.randn(tokens, (2 * heads + 2 * kv) * d, device=dev)
+        for _ in range(6):
+            keep_busy()
+            start.record()
+            ops.element_gate(x, fused, (heads + 2 * kv) * d, heads, d)
+            stop.record()
+            torch.cuda.synchronize()
+            times.append(start.elapsed_time(stop) * 1e3)
+        work = {"bytes": tokens * heads * d * (4 + 2 + 2)}
+    elif args.case == "act_blocks":
+        # --batch rows of 8 experts of 7,104 columns, two chosen a row: those are read, all are written
+        x = torch.randn(tokens, 8 * 7104, device=dev).to(torch.bfloat16)
+        share = torch.zeros(tokens, 9, device=dev)
+        share[:, :2] = 0.4
+        for _ in range(6):
+            keep_busy()
+            start.record()
+            ops.act_blocks(x, share, 8, 7104, "gelu")
+            stop.record()
+            torch.cuda.synchronize()
+            times.append(start.elapsed_time(stop) * 1e3)
+        work = {"bytes": tokens * 7104 * 2 * (8 + 2)}
+    elif args.case == "low_rank":
+        # --batch rows: 3,584 decays from a rank of 16
+        fused = torch.randn(tokens, 4 * heads * d + 16, device=dev)
+        matrix = torch.randn(heads * d, 16, device=dev).to(torch.bfloat16)
+        out = torch.empty(tokens, heads * d, device=dev)
+        for _ in range(6):
+            keep_busy()
+            start.record()
+            ops.low_rank(fused, 4 * heads * d, 16, matrix, out)
+            stop.record()
+            torch.cuda.synchronize()
+            times.append(start.elapsed_time(stop) * 1e3)
+        work = {"bytes": tokens * (heads * d * 4 + 64)}
     elif args.case == "delta_prep":
         # --batch tokens of one sequence, q, k and v of 28 heads of 128 behind four taps, beta and two low-rank rows of 128
         channels = 3 * heads * d
@@ -983,7 +1066,7 @@ def run_timeline(args) -> dict:
 
 
 def run_design(args) -> dict:
-    """A design (--arch sadodra, the default here, vupitar, kavedra, setotar or nulazen; the last two also beside the designs they are closest to) beside the Qwen2 decoder of the same widths, layer count and vocabulary (the
+    """A design (--arch sadodra, the default here, vupitar, kavedra, setotar, nulazen or radilix; the last three also beside the designs they are closest to) beside the Qwen2 decoder of the same widths, layer count and vocabulary (the
     closest model this engine serves), random weights: one 2,048-token prompt in one step, and decoding
     at --batch sequences of --context tokens, device-timed through the step function and the sampling
     kernel; for each, the kernels of one step by the time they take (CUPTI activity records).
@@ -1119,8 +1202,9 @@ def run_design(args) -> dict:
     t0 = time.perf_counter()
     results = [measure(f"{design.capitalize()} at Qwen2.5-{args.design.upper()} widths", ours)]
     # the designs it is closest to among those served: Setotar to Vupitar (attention beside a recurrent memory in one layer,
-    # routed experts); Nulazen to Kavedra (latent attention, a linear recurrence) and for its experts to Vupitar
-    for like in {"setotar": ("vupitar",), "nulazen": ("kavedra", "vupitar")}.get(design, ()):
+    # routed experts); Nulazen to Kavedra (latent attention, a linear recurrence) and for its experts to Vupitar; Radilix to
+    # Setotar (attention beside a recurrence, experts in every layer) and for its recurrences to Nulazen
+    for like in {"setotar": ("vupitar",), "nulazen": ("kavedra", "vupitar"), "radilix": ("setotar", "nulazen")}.get(design, ()):
         likeness = dict(shape_config(f"{like}-{args.design}"))
         if args.layers:
             loop = likeness.get("loop")
@@ -1157,13 +1241,14 @@ def main():
     parser.add_argument("--context", type=int, default=1024, help="tokens each sequence holds when decoding is timed")
     parser.add_argument("--workload", default="decode", choices=["decode", "mixed"],
                         help="decode: the headline line; mixed: 64 requests through the scheduler at 1.5B shape")
-    parser.add_argument("--arch", default="qwen2", choices=["qwen2", "sadodra", "vupitar", "kavedra", "setotar", "nulazen"],
+    parser.add_argument("--arch", default="qwen2", choices=["qwen2", "sadodra", "vupitar", "kavedra", "setotar", "nulazen", "radilix"],
                         help="--workload mixed: the decoder the 64 requests run on (all at Qwen2.5-1.5B widths); "
                              "--case design: the design that is set beside the Qwen2 decoder (default there: sadodra)")
     parser.add_argument("--num-blocks", type=int, default=0, help="cache pages for --workload mixed (few pages force preemption)")
     parser.add_argument("--skip-mixed", action="store_true", help="leave the mixed workload out of the default line")
     parser.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS,
                         help="prompt length of --case attention_portions")
+    parser.add_argument("--heads", type=int, default=0, help="--case head_delta_scan / gla_scan: heads (0: those of the 7B-width shape)")
     parser.add_argument("--design", default="1.5b", choices=["1.5b", "7b"],
                         help="--case design: the widths at which the Sadodra decoder and the Qwen2 decoder are compared")
     parser.add_argument("--case", default=None,
@@ -1172,6 +1257,7 @@ def main():
                              "one key/value head of 256 whose keys are its values; with _sink: a sink in every softmax), "
                              "branch_norm, tanh_norm, head_prep, matrix_memory (a prompt of --prefill-tokens), matrix_memory_single, "
                              "decay_scan (a prompt of --prefill-tokens), decay_scan_single, latent_rope_store, gated_scan, gated_scan_single, "
+                             "head_delta_scan, gla_scan (a prompt of --prefill-tokens; --heads), the same with _single, sum_norm, element_gate, act_blocks, low_rank, "
                              "stream_norm, short_conv, delta_scan (a prompt of --prefill-tokens), delta_scan_single, delta_prep, norm_join, head_rms, "
                              "attention_single_kept, attention_portions_kept; "
                              "--batch gives tokens / sequences / rows.  timeline: per-kernel "

@@ -445,6 +445,14 @@ struct BlockArgs {
   int num_seqs, from;       // sequences that bring at least `from` tokens run here
   int blocks;               // of the whole batch
   int head0, head_count;    // the heads this launch serves
+  // Where the walks are few, a sequence is cut into runs of `run_blocks` blocks that walk side by side (0: it is not): first
+  // every run but the last by itself, for what it makes of a zero state (A) and of any state (the delta rule: a matrix F,
+  // S -> F S + A; without it a decay per row), then the states are carried from run to run, then every run walks again
+  // from the state it starts from and gives its outputs.
+  int run_blocks, value_slices;
+  float* run_states;        // [runs][head_count][D][run_ld]: A, later the state a run starts from (vdim rounded up to four) | F [Dp]
+  float* run_decays;        // [runs][head_count][Dp], without the delta rule
+  int run_ld, run_values;   // run_values: the column where F begins
 };
 
 __host__ __device__ constexpr int record_floats(int padded_dim, bool delta) { return ((delta ? 3 : 2) * BLOCK + 1) * padded_dim + BLOCK * BLOCK; }
@@ -453,6 +461,34 @@ __host__ __device__ constexpr int record_floats(int padded_dim, bool delta) { re
 __device__ __forceinline__ int blocks_of(const BlockArgs& a, int seq) {
   const int length = a.s.q_start[seq + 1] - a.s.q_start[seq];
   return length >= a.from ? (length + BLOCK - 1) / BLOCK : 0;
+}
+
+__device__ __forceinline__ int runs_of(const BlockArgs& a, int seq) { return (blocks_of(a, seq) + a.run_blocks - 1) / a.run_blocks; }
+
+struct RunPlace { int seq, run, base; };   // base: the first block of the sequence among the batch's
+
+// The sequence and the run within it of run `index` of the batch; lanes count 32 sequences at a time.
+__device__ __forceinline__ RunPlace place_of_run(const BlockArgs& a, int index, int lane) {
+  int runs_before = 0, blocks_before = 0;
+  for (int base = 0; base < a.num_seqs; base += 32) {
+    const int blocks = base + lane < a.num_seqs ? blocks_of(a, base + lane) : 0;
+    const int runs = (blocks + a.run_blocks - 1) / a.run_blocks;
+    int runs_sum = runs, blocks_sum = blocks;
+#pragma unroll
+    for (int offset = 1; offset < 32; offset <<= 1) {
+      const int other_runs = __shfl_up_sync(0xffffffffu, runs_sum, offset), other_blocks = __shfl_up_sync(0xffffffffu, blocks_sum, offset);
+      if (lane >= offset) { runs_sum += other_runs; blocks_sum += other_blocks; }
+    }
+    const unsigned hit = __ballot_sync(0xffffffffu, runs > 0 && index < runs_before + runs_sum);
+    if (hit) {
+      const int owner = __ffs(hit) - 1;
+      return {base + owner, index - runs_before - __shfl_sync(0xffffffffu, runs_sum - runs, owner),
+              blocks_before + __shfl_sync(0xffffffffu, blocks_sum - blocks, owner)};
+    }
+    runs_before += __shfl_sync(0xffffffffu, runs_sum, 31);
+    blocks_before += __shfl_sync(0xffffffffu, blocks_sum, 31);
+  }
+  return {-1, 0, 0};
 }
 
 // The sums of COUNT values over 2 * OFFSET lanes, transposed: every step halves the values a lane holds, so that lane g of
@@ -526,16 +562,17 @@ __global__ void __launch_bounds__(128) delta_local_kernel(const BlockArgs a) {
     const float z = sum_partials(s.gates + static_cast<size_t>(first + lane) * s.gate_width + s.gate_at + head, s.stride, s.partials);
     head_decay = decay_of(s, rate, z, s.bias != nullptr ? s.bias[head] : 0.f);
   }
-  for (int d = lane; d - lane < Dp; d += 32) {   // every lane takes part in the shuffles; rows past Dp are not stored
+  const float q_scale = s.q_scale;
+  for (int d = lane; (HEAD ? d - lane : d) < Dp; d += 32) {   // (one decay a head: every lane takes part in the shuffles)
     float g[BLOCK], k[BLOCK], q[BLOCK];
-    const bool row = d < D, kept = d < Dp;
+    const bool row = d < D, kept = !HEAD || d < Dp;
     const float shift = !HEAD && row && s.bias != nullptr ? s.bias[head * D + d] : 0.f;
 #pragma unroll
     for (int t = 0; t < BLOCK; ++t) {
       const bool real = row && t < here;
       const float* at = s.mixed + static_cast<size_t>(first + (t < here ? t : 0)) * s.pitch;
       k[t] = real ? at[k_col + d] : 0.f;
-      q[t] = real ? s.q_scale * at[q_col + d] : 0.f;
+      q[t] = real ? q_scale * at[q_col + d] : 0.f;
       if (!HEAD) g[t] = real ? s.gates[static_cast<size_t>(first + t) * s.gate_width + s.gate_at + head * D + d] : 0.f;
     }
     if (!HEAD && s.partials > 1) {
@@ -544,10 +581,7 @@ __global__ void __launch_bounds__(128) delta_local_kernel(const BlockArgs a) {
         if (row && t < here) g[t] = sum_partials(s.gates + static_cast<size_t>(first + t) * s.gate_width + s.gate_at + head * D + d, s.stride, s.partials);
     }
 #pragma unroll
-    for (int t = 0; t < BLOCK; ++t) {
-      if (HEAD) g[t] = __shfl_sync(0xffffffffu, head_decay, t);
-      else g[t] = row && t < here ? decay_of(s, rate, g[t], shift) : (row ? 1.f : 0.f);
-    }
+    for (int t = 0; t < BLOCK; ++t) g[t] = HEAD ? __shfl_sync(0xffffffffu, head_decay, t) : (row && t < here ? decay_of(s, rate, g[t], shift) : (row ? 1.f : 0.f));
 #pragma unroll
     for (int from = 0; from < BLOCK; ++from) {
       float w = k[from];
@@ -656,9 +690,13 @@ constexpr int STAGES = 3;
 // rows 4 g .. 4 g + 3 (with CHUNKS 2 also the same LANES * 4 further on) of four neighbouring columns; LANES lanes, a
 // team, cover the head's rows.  Register c of a lane is column c ^ turn of the team's four, `turn` the lane's top two bits:
 // adding up over those lanes then needs no selection, every step keeps the first half of the columns and sends the other.
-template <int LANES, int CHUNKS, bool DELTA>
+// Whole: blockIdx.z is a sequence.  In runs it is a run of the batch: Gather walks a run for its A and, in the CTAs behind the
+// value columns', its F (from the identity with values of zero) and reads nothing out; FromStart walks it from its own state.
+enum class Walk { Whole, Gather, FromStart };
+template <int LANES, int CHUNKS, bool DELTA, Walk WALK>
 __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(const BlockArgs a) {
   extern __shared__ __align__(16) float blocks_shared[];
+  constexpr bool OUT = WALK != Walk::Gather, RUNS = WALK != Walk::Whole;
   constexpr int C = 4, PAIRS = 2 * CHUNKS, N = BLOCK * C;
   constexpr int COLUMN_LANES = LANES >= C ? C : LANES;   // lanes the columns are shared out over, then the tokens
   constexpr int TOKEN_LANES = LANES / COLUMN_LANES;
@@ -668,25 +706,47 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
   const ScanArgs& s = a.s;
   let_dependents_start();
   wait_for_previous();
-  const int local_head = blockIdx.y, head = a.head0 + local_head, seq = blockIdx.z, cols = s.cols, col0 = blockIdx.x * cols;
-  const int first = s.q_start[seq], length = s.q_start[seq + 1] - first;
-  if (length < a.from) return;   // the token-by-token walk serves it
+  const int local_head = blockIdx.y, head = a.head0 + local_head, cols = s.cols;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane % LANES, team = lane / LANES;
+  int seq = blockIdx.z, base = 0;   // base: the first block of this walk
+  bool last = true;
+  int first, length;
+  if constexpr (RUNS) {
+    const RunPlace place = place_of_run(a, blockIdx.z, lane);
+    if (place.seq < 0) return;
+    seq = place.seq;
+    const int begin = place.run * a.run_blocks;
+    base = place.base + begin;
+    first = s.q_start[seq] + begin * BLOCK;
+    const int left = s.q_start[seq + 1] - first;
+    last = left <= a.run_blocks * BLOCK;
+    length = last ? left : a.run_blocks * BLOCK;
+    if (!OUT && last) return;   // no run starts from what the last one makes
+  } else {
+    first = s.q_start[seq];
+    length = s.q_start[seq + 1] - first;
+    if (length < a.from) return;   // the token-by-token walk serves it
+  }
+  const bool whole_map = !OUT && static_cast<int>(blockIdx.x) >= a.value_slices;   // this CTA's columns are F's
+  const int col0 = (whole_map ? blockIdx.x - a.value_slices : blockIdx.x) * cols;
   const int j = (warp * (32 / LANES) + team) * C;   // the first of the team's columns among the CTA's
   const int turn = COLUMN_LANES == 4 ? g / TOKEN_LANES : (COLUMN_LANES == 2 ? 2 * g : 0);
-  const int cols_here = min(cols, s.vdim - col0);
+  const int cols_here = min(cols, (whole_map ? Dp : s.vdim) - col0);
+  const int values_here = whole_map ? 0 : cols_here;   // columns whose values are read; the others' are zero
   const int slot = s.state_slot[seq];
   const size_t out_width = static_cast<size_t>(s.heads) * s.vdim;
   float* out = s.out + static_cast<size_t>(first) * out_width + head * s.vdim + col0;
   if (slot < 0 || slot >= s.num_slots) {
-    for (int t = 0; t < length; ++t)
-      for (int c = threadIdx.x; c < cols_here; c += blockDim.x) out[t * out_width + c] = 0.f;
+    if (OUT)
+      for (int t = 0; t < length; ++t)
+        for (int c = threadIdx.x; c < cols_here; c += blockDim.x) out[t * out_width + c] = 0.f;
     return;
   }
-  int base = 0;   // the sequence's first block
-  for (int other = lane; other < seq; other += 32) base += blocks_of(a, other);
+  if constexpr (!RUNS) {
+    for (int other = lane; other < seq; other += 32) base += blocks_of(a, other);
 #pragma unroll
-  for (int offset = 16; offset > 0; offset >>= 1) base += __shfl_xor_sync(0xffffffffu, base, offset);
+    for (int offset = 16; offset > 0; offset >>= 1) base += __shfl_xor_sync(0xffffffffu, base, offset);
+  }
   const int blocks = (length + BLOCK - 1) / BLOCK;
   const int stage_floats = RECORD + BLOCK * cols;
   float* team_values = blocks_shared + STAGES * stage_floats + (warp * (32 / LANES) + team) * 2 * N;   // d, then c, of this team's columns
@@ -709,13 +769,13 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
       const float* from = s.mixed + static_cast<size_t>(first + block * BLOCK) * s.pitch + v_col;
       if (one_piece) {
         if (static_cast<int>(threadIdx.x) < pieces) {
-          if (piece_t < here && piece_c < cols_here) copy16(v + piece_t * cols + piece_c, from + static_cast<size_t>(piece_t) * s.pitch + piece_c);
+          if (piece_t < here && piece_c < values_here) copy16(v + piece_t * cols + piece_c, from + static_cast<size_t>(piece_t) * s.pitch + piece_c);
           else *reinterpret_cast<float4*>(v + piece_t * cols + piece_c) = make_float4(0.f, 0.f, 0.f, 0.f);
         }
       } else {
         for (int i = threadIdx.x; i < BLOCK * cols; i += blockDim.x) {
           const int t = i / cols, c = i - t * cols;
-          if (t < here && c < cols_here) copy4(v + i, from + static_cast<size_t>(t) * s.pitch + c);
+          if (t < here && c < values_here) copy4(v + i, from + static_cast<size_t>(t) * s.pitch + c);
           else v[i] = 0.f;
         }
       }
@@ -726,16 +786,26 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
 #pragma unroll
   for (int i = 0; i < STAGES - 1; ++i) stage(i);
   float* state = s.state + (static_cast<size_t>(slot) * s.heads + head) * s.head_stride;
+  const size_t run_at = (static_cast<size_t>(blockIdx.z) * a.head_count + local_head) * s.dim * a.run_ld + (whole_map ? a.run_values : 0) + col0;
   unsigned long long S[C][PAIRS];
 #pragma unroll
   for (int p = 0; p < PAIRS; ++p)
 #pragma unroll
     for (int c = 0; c < C; ++c) {
       const int d = (p / 2) * 4 * LANES + 4 * g + (p & 1) * 2, column = j + (c ^ turn);
-      const float* at = state + static_cast<size_t>(d) * s.vdim + col0 + column;
       const bool mine = column < cols_here;
-      S[c][p] = pack2(mine && d < s.dim ? at[0] : 0.f, mine && d + 1 < s.dim ? at[s.vdim] : 0.f);
+      if constexpr (OUT) {
+        const float* at = RUNS ? a.run_states + run_at + static_cast<size_t>(d) * a.run_ld + column
+                               : state + static_cast<size_t>(d) * s.vdim + col0 + column;
+        S[c][p] = pack2(mine && d < s.dim ? at[0] : 0.f, mine && d + 1 < s.dim ? at[RUNS ? a.run_ld : s.vdim] : 0.f);
+      } else {
+        S[c][p] = pack2(whole_map && d < s.dim && d == col0 + column ? 1.f : 0.f, whole_map && d + 1 < s.dim && d + 1 == col0 + column ? 1.f : 0.f);
+      }
     }
+  constexpr int DECAYS = !OUT && !DELTA ? (Dp + 31) / 32 : 1;   // a thread's share of the rows' decays, at one warp a CTA
+  float run_decay[DECAYS];
+#pragma unroll
+  for (int k = 0; k < DECAYS; ++k) run_decay[k] = 1.f;
   int taken = 0;   // the stage of the block at hand
   for (int block = 0; block < blocks; ++block) {
     asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
@@ -747,7 +817,7 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
     const float* v = at + RECORD;
     float sum[2][N];   // a_t, then c_t, of this thread's rows: [column][token]
 #pragma unroll
-    for (int which = DELTA ? 0 : 1; which < 2; ++which) {
+    for (int which = DELTA ? 0 : 1; which < (OUT ? 2 : 1); ++which) {
 #pragma unroll
       for (int t = 0; t < BLOCK; ++t) {
         unsigned long long acc[C];
@@ -772,22 +842,27 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
 #pragma unroll
       for (int i = 0; i < half; ++i)
 #pragma unroll
-        for (int which = DELTA ? 0 : 1; which < 2; ++which) sum[which][i] += __shfl_xor_sync(0xffffffffu, sum[which][i + half], offset);
+        for (int which = DELTA ? 0 : 1; which < (OUT ? 2 : 1); ++which) sum[which][i] += __shfl_xor_sync(0xffffffffu, sum[which][i + half], offset);
     // this lane holds its columns' sums, shared with TOKEN_LANES - 1 others: d_t = v_t - a_t of its own tokens
 #pragma unroll
     for (int i = 0; i < OWN_COLUMNS; ++i) {
       if constexpr (DELTA) FoldLanes<BLOCK, TOKEN_LANES / 2>::run(sum[0] + i * BLOCK, lane);
-      FoldLanes<BLOCK, TOKEN_LANES / 2>::run(sum[1] + i * BLOCK, lane);
+      if constexpr (OUT) FoldLanes<BLOCK, TOKEN_LANES / 2>::run(sum[1] + i * BLOCK, lane);
       const int c = turn + i;
 #pragma unroll
       for (int k = 0; k < OWN_TOKENS; ++k) {
         const int t = g % TOKEN_LANES * OWN_TOKENS + k;
         team_values[c * BLOCK + t] = v[t * cols + j + c] - (DELTA ? sum[0][i * BLOCK + k] : 0.f);
-        team_values[N + c * BLOCK + t] = sum[1][i * BLOCK + k];
+        if (OUT) team_values[N + c * BLOCK + t] = sum[1][i * BLOCK + k];
       }
     }
     __syncwarp();
     const float* decay = at + (K_ROW + BLOCK) * Dp;
+    if (!OUT && !DELTA && blockIdx.x == 0) {
+#pragma unroll
+      for (int k = 0; k < DECAYS; ++k)
+        if (static_cast<int>(threadIdx.x + k * blockDim.x) < Dp) run_decay[k] *= decay[threadIdx.x + k * blockDim.x];
+    }
 #pragma unroll
     for (int chunk = 0; chunk < CHUNKS; ++chunk) {
       const ulonglong2 x = *(reinterpret_cast<const ulonglong2*>(decay) + g + chunk * LANES);
@@ -823,7 +898,7 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
     const float* m = decay + Dp;
     const int here = min(BLOCK, length - block * BLOCK);
 #pragma unroll
-    for (int i = 0; i < (N + LANES - 1) / LANES; ++i) {
+    for (int i = 0; i < (OUT ? (N + LANES - 1) / LANES : 0); ++i) {
       const int at_value = g + i * LANES, t = at_value / C, c = at_value % C;
       if (at_value < N && t < here && j + c < cols_here) {
         float o = team_values[N + c * BLOCK + t];
@@ -842,18 +917,179 @@ __global__ void __launch_bounds__(CHUNKS == 2 ? 128 : 256) delta_blocks_kernel(c
     __syncwarp();   // the team's values are used up before the next block overwrites them
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
+  if (RUNS && OUT && !last) return;   // the run behind this one starts from what the carry made
 #pragma unroll
   for (int p = 0; p < PAIRS; ++p)
 #pragma unroll
     for (int c = 0; c < C; ++c) {
       const int d = (p / 2) * 4 * LANES + 4 * g + (p & 1) * 2, column = j + (c ^ turn);
-      float* at = state + static_cast<size_t>(d) * s.vdim + col0 + column;
+      float* at = OUT ? state + static_cast<size_t>(d) * s.vdim + col0 + column
+                      : a.run_states + run_at + static_cast<size_t>(d) * a.run_ld + column;
       const float2 two = unpack2(S[c][p]);
       if (column < cols_here) {
         if (d < s.dim) at[0] = two.x;
-        if (d + 1 < s.dim) at[s.vdim] = two.y;
+        if (d + 1 < s.dim) at[OUT ? s.vdim : a.run_ld] = two.y;
       }
     }
+  if (!OUT && !DELTA && blockIdx.x == 0) {
+#pragma unroll
+    for (int k = 0; k < DECAYS; ++k)
+      if (static_cast<int>(threadIdx.x + k * blockDim.x) < Dp)
+        a.run_decays[(static_cast<size_t>(blockIdx.z) * a.head_count + local_head) * Dp + threadIdx.x + k * blockDim.x] = run_decay[k];
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ states from run to run
+// grid (columns / CARRY_COLS, heads, sequences): S <- F S + A over a sequence's runs, each left the state it starts from
+// where its A was.  A warp takes every eighth row of F, whose columns its lanes hold the state's rows for (EC groups of 128);
+// the products meet by shuffles, the new state in shared memory.  STAGED: the next run's F and A are brought into shared
+// memory (`padded_dim` columns and the CTA's own a row) while the present run's are multiplied; heads of more than 128 rows
+// read them where they lie.
+constexpr int CARRY_COLS = 8;
+__host__ __device__ constexpr int carry_pitch(int padded_dim) { return padded_dim + CARRY_COLS; }
+__host__ __device__ constexpr int carry_rows(int padded_dim) { return padded_dim + 4; }   // a state column's pitch: the columns fall into different banks
+
+template <int EC, bool STAGED>
+__global__ void __launch_bounds__(256) delta_carry_kernel(const BlockArgs a) {
+  extern __shared__ __align__(16) float carry_shared[];   // two states of [CARRY_COLS][rows], then (STAGED) two runs' [D][F | A]
+  const ScanArgs& s = a.s;
+  let_dependents_start();
+  wait_for_previous();
+  const int local_head = blockIdx.y, head = a.head0 + local_head, seq = blockIdx.z, col0 = blockIdx.x * CARRY_COLS;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, D = s.dim, slot = s.state_slot[seq];
+  const int runs = runs_of(a, seq), cols_here = min(CARRY_COLS, s.vdim - col0);
+  if (runs == 0 || slot < 0 || slot >= s.num_slots) return;
+  int first_run = 0;
+  for (int other = lane; other < seq; other += 32) first_run += runs_of(a, other);
+#pragma unroll
+  for (int offset = 16; offset > 0; offset >>= 1) first_run += __shfl_xor_sync(0xffffffffu, first_run, offset);
+  const float* state = s.state + (static_cast<size_t>(slot) * s.heads + head) * s.head_stride + col0;
+  const int rows = carry_rows(a.padded_dim);
+  float* now = carry_shared;
+  float* next = carry_shared + rows * CARRY_COLS;
+  for (int i = threadIdx.x; i < rows * CARRY_COLS; i += blockDim.x) {
+    const int d = i / CARRY_COLS, c = i % CARRY_COLS;
+    now[c * rows + d] = c < cols_here && d < D ? state[static_cast<size_t>(d) * s.vdim + c] : 0.f;
+    next[c * rows + d] = 0.f;
+  }
+  const int own_col = lane / 4;   // where a row's eight sums end: four lanes hold the same one
+  const bool keeper = lane % 4 == 0 && own_col < cols_here;
+  const int pitch = carry_pitch(a.padded_dim), stage_floats = D * pitch;
+  float* stages = carry_shared + 2 * rows * CARRY_COLS;
+  const bool wide_a = cols_here == CARRY_COLS;   // (columns of A beyond the head's own values are not there)
+  const auto stage = [&](int run) {   // asks for a run's F and this CTA's columns of A
+    if (run + 1 < runs) {
+      const float* held = a.run_states + (static_cast<size_t>(first_run + run) * a.head_count + local_head) * D * a.run_ld;
+      float* at = stages + (run & 1) * stage_floats;
+      const int pieces = a.padded_dim / 4;
+      for (int i = threadIdx.x; i < D * pieces; i += blockDim.x) {
+        const int d = i / pieces, p = (i - d * pieces) * 4;
+        copy16(at + d * pitch + p, held + static_cast<size_t>(d) * a.run_ld + a.run_values + p);
+      }
+      for (int i = threadIdx.x; i < D * 2; i += blockDim.x) {
+        const int d = i >> 1, p = (i & 1) * 4;
+        float* to = at + d * pitch + a.padded_dim + p;
+        const float* from = held + static_cast<size_t>(d) * a.run_ld + col0 + p;
+        if (wide_a) {
+          copy16(to, from);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            if (p + e < cols_here) copy4(to + e, from + e);
+            else to[e] = 0.f;
+          }
+        }
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  if (STAGED) stage(0);
+  for (int run = 0; run < runs; ++run) {
+    float* held = a.run_states + (static_cast<size_t>(first_run + run) * a.head_count + local_head) * D * a.run_ld;
+    if (STAGED) asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();   // `now` is complete, the run's F and A are there, and everyone is done with the stage filled next
+    if (STAGED) stage(run + 1);
+    if (run + 1 == runs) {
+      for (int i = threadIdx.x; i < D * CARRY_COLS; i += blockDim.x) {
+        const int d = i / CARRY_COLS, c = i % CARRY_COLS;
+        if (c < cols_here) held[static_cast<size_t>(d) * a.run_ld + col0 + c] = now[c * rows + d];
+      }
+      return;
+    }
+    float S[EC][4][CARRY_COLS];
+#pragma unroll
+    for (int ec = 0; ec < EC; ++ec)
+#pragma unroll
+      for (int c = 0; c < CARRY_COLS; ++c) {
+        float four[4] = {0.f, 0.f, 0.f, 0.f};
+        if (ec * 128 + lane * 4 < a.padded_dim) load4<float>(now + c * rows + ec * 128 + lane * 4, four);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) S[ec][i][c] = four[i];
+      }
+#pragma unroll 4
+    for (int d = warp; d < D; d += 8) {
+      const float* row = STAGED ? stages + (run & 1) * stage_floats + d * pitch : held + static_cast<size_t>(d) * a.run_ld + a.run_values;
+      float* mine = held + static_cast<size_t>(d) * a.run_ld + col0 + own_col;
+      const float added = keeper ? (STAGED ? row[a.padded_dim + own_col] : *mine) : 0.f;
+      float sum[CARRY_COLS];
+#pragma unroll
+      for (int c = 0; c < CARRY_COLS; ++c) sum[c] = 0.f;
+#pragma unroll
+      for (int ec = 0; ec < EC; ++ec) {
+        float f[4] = {0.f, 0.f, 0.f, 0.f};
+        if (ec * 128 + lane * 4 < D) load4<float>(row + ec * 128 + lane * 4, f);
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int c = 0; c < CARRY_COLS; ++c) sum[c] = __fmaf_rn(f[i], S[ec][i][c], sum[c]);
+      }
+      FoldLanes<CARRY_COLS, 16>::run(sum, lane);
+      if (keeper) {
+        next[own_col * rows + d] = sum[0] + added;
+        *mine = now[own_col * rows + d];
+      }
+    }
+    float* swap = now;
+    now = next;
+    next = swap;
+  }
+}
+
+// The same without the delta rule, where a run only multiplies every row of the state: a thread an element of it.
+__global__ void __launch_bounds__(256) gated_carry_kernel(const BlockArgs a, int padded_dim) {
+  const ScanArgs& s = a.s;
+  let_dependents_start();
+  wait_for_previous();
+  const int local_head = blockIdx.y, head = a.head0 + local_head, seq = blockIdx.z, lane = threadIdx.x & 31, slot = s.state_slot[seq];
+  const int runs = runs_of(a, seq);
+  if (runs == 0 || slot < 0 || slot >= s.num_slots) return;
+  int first_run = 0;
+  for (int other = lane; other < seq; other += 32) first_run += runs_of(a, other);
+#pragma unroll
+  for (int offset = 16; offset > 0; offset >>= 1) first_run += __shfl_xor_sync(0xffffffffu, first_run, offset);
+  const int index = blockIdx.x * blockDim.x + threadIdx.x;
+  if (index >= s.dim * s.vdim) return;
+  const int d = index / s.vdim, c = index - d * s.vdim;
+  float S = s.state[(static_cast<size_t>(slot) * s.heads + head) * s.head_stride + index];
+  const size_t step = static_cast<size_t>(a.head_count) * s.dim * a.run_ld, decay_step = static_cast<size_t>(a.head_count) * padded_dim;
+  float* held = a.run_states + (static_cast<size_t>(first_run) * a.head_count + local_head) * s.dim * a.run_ld + static_cast<size_t>(d) * a.run_ld + c;
+  const float* decay = a.run_decays + (static_cast<size_t>(first_run) * a.head_count + local_head) * padded_dim + d;
+  constexpr int AHEAD = 4;
+  for (int run = 0; run < runs; run += AHEAD) {
+    float added[AHEAD], keep[AHEAD];
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i)
+      if (run + i + 1 < runs) {
+        added[i] = held[(run + i) * step];
+        keep[i] = decay[(run + i) * decay_step];
+      }
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i)
+      if (run + i < runs) {
+        held[(run + i) * step] = S;
+        if (run + i + 1 < runs) S = __fmaf_rn(keep[i], S, added[i]);
+      }
+  }
 }
 
 // ------------------------------------------------------------------------------------------------ low_rank
@@ -998,6 +1234,27 @@ SHRIKE_API int shrike_delta_scan_record(int dim, int delta) {
 }
 SHRIKE_API int shrike_delta_scan_block() { return BLOCK; }
 
+// How many blocks a run has where a batch of `seqs` sequences in blocks (`blocks` in all, `longest` the most of one), `heads` heads at a
+// time, is to be cut into runs; 0: it is not.  A run is walked twice (the delta rule: dim / vdim times more), so runs pay where the
+// walks alone would leave most of the SMs idle.
+SHRIKE_API int shrike_delta_scan_run_blocks(int blocks, int longest, int seqs, int heads, int dim, int vdim, int delta) {
+  DeltaShape shape;
+  if (dim > 256 || seqs < 1 || longest < 48 || !delta_shape(dim, vdim, &shape)) return 0;
+  const long long sms = shrike_device().sm_count, each = static_cast<long long>((vdim + 31) / 32) * heads;   // each: CTAs of one run
+  const long long wanted = 2 * sms / each;   // runs that fill the device
+  if (wanted < 3 * static_cast<long long>(seqs) || (delta && sms / each < 4 * static_cast<long long>(seqs))) return 0;
+  const int run = static_cast<int>((blocks + wanted - 1) / wanted), least = delta ? 32 : 16;
+  return run < least ? least : run;
+}
+
+// Scratch floats of one head of one run.
+SHRIKE_API long long shrike_delta_scan_run_floats(int dim, int vdim, int delta) {
+  DeltaShape shape;
+  if (!delta_shape(dim, vdim, &shape)) return 0;
+  const long long padded = shape.lanes * shape.rows, values = (vdim + 3) / 4 * 4;
+  return static_cast<long long>(dim) * (values + (delta ? padded : 0)) + padded;
+}
+
 // `mixed` (`mixed_partials` slices `mixed_stride` apart, rows of `pitch`): q | k | v; only a walk takes more than one slice.
 // `beta` null: no delta rule.  `gate_each`: 1, one decay a head, or dim, one a key channel (`bias`, where there is one, has
 // heads * gate_each numbers); the decays' columns begin at `gate_at`.
@@ -1005,12 +1262,14 @@ SHRIKE_API int shrike_delta_scan_block() { return BLOCK; }
 // (blocks x head_count x shrike_delta_scan_record floats, `blocks` = the sum of ceil(length / BLOCK) over them); heads are
 // then served `head_count` at a time.  `early_state` 1: the caller knows that whatever kernel wrote the states has finished
 // (an earlier step, not merely an earlier launch), so that the walk may read them while the kernel before it runs.  `shorter`: whether the batch has sequences below `from`.
+// `run_blocks` > 0: sequences are cut into runs of so many blocks, `runs` in all (the sum of ceil(blocks / run_blocks)), for which the
+// caller holds `run_scratch` (runs x head_count x shrike_delta_scan_run_floats).
 SHRIKE_API int shrike_delta_scan(const float* mixed, int mixed_partials, long long mixed_stride, int pitch, const float* beta,
                                  const float* gates, int partials, long long stride, int gate_width, int gate_at, int gate_each,
                                  const float* rate, const float* bias, float sign, float q_scale, float* state, const int* q_start,
                                  const int* state_slot, float* out, int num_seqs, int heads, int kv_heads, int dim, int vdim,
                                  int head_stride, int num_slots, int from, int shorter, float* records, int blocks,
-                                 int head_count, int early_state, cudaStream_t stream) {
+                                 int head_count, int early_state, int run_blocks, int runs, float* run_scratch, cudaStream_t stream) {
   if (num_seqs <= 0) return SHRIKE_OK;
   if (heads < 1 || heads > 65535 || num_seqs > 65535 || kv_heads < 1 || heads % kv_heads || dim < 1 || vdim < 1 || partials < 1 ||
       mixed_partials < 1 || head_stride < dim * vdim || (gate_each != 1 && gate_each != dim) || gate_at < 0 ||
@@ -1045,21 +1304,28 @@ SHRIKE_API int shrike_delta_scan(const float* mixed, int mixed_partials, long lo
     // Four rows a thread where the walks are few (twice the warps hide each other's waits), eight where there are enough
     // of them (half the adding up over lanes); a head of more than 128 rows takes eight.
     const int sms = shrike_device().sm_count;
+    const bool in_runs = run_blocks > 0 && runs > 0 && run_scratch != nullptr;
+    if (in_runs && (runs > 65535 || vdim < 1)) return SHRIKE_BAD_ARGUMENT;
+    const long long walks = in_runs ? runs : num_seqs;
     const long long quarters = static_cast<long long>((vdim + 31) / 32) * min(head_count, heads) * num_seqs;   // CTAs of 32 columns
-    const int chunks = b.padded_dim > 128 || quarters > 2 * sms ? 2 : 1;
+    const int chunks = b.padded_dim > 128 || (quarters > 2 * sms && !in_runs) ? 2 : 1;
     const int lanes = b.padded_dim / (4 * chunks);
     const int per_warp = 32 / lanes * 4;
     int warps = max(1, min(chunks == 2 ? 4 : 8, (vdim + per_warp - 1) / per_warp));
     // few heads: narrower CTAs, as many as there are SMs for
-    while (warps > 2 && warps % 2 == 0 &&
+    while (warps > 2 && warps % 2 == 0 && !in_runs &&
            static_cast<long long>((vdim + per_warp * warps - 1) / (per_warp * warps)) * min(head_count, heads) * num_seqs * 2 <= sms)
       warps /= 2;
     b.s.cols = per_warp * warps;
     const unsigned block_slices = static_cast<unsigned>((vdim + b.s.cols - 1) / b.s.cols);
     void (*kernel)(BlockArgs) = nullptr;
+    void (*gather)(BlockArgs) = nullptr;   // the runs' first walk
+#define SHRIKE_DELTA_BLOCKS_OF(L, WALK)                                                                  \
+  (delta_rule ? (chunks == 2 ? delta_blocks_kernel<L, 2, true, WALK> : delta_blocks_kernel<L, 1, true, WALK>) \
+              : (chunks == 2 ? delta_blocks_kernel<L, 2, false, WALK> : delta_blocks_kernel<L, 1, false, WALK>))
 #define SHRIKE_DELTA_BLOCKS(L)                                                                                    \
-  kernel = delta_rule ? (chunks == 2 ? delta_blocks_kernel<L, 2, true> : delta_blocks_kernel<L, 1, true>) \
-                      : (chunks == 2 ? delta_blocks_kernel<L, 2, false> : delta_blocks_kernel<L, 1, false>)
+  kernel = in_runs ? SHRIKE_DELTA_BLOCKS_OF(L, Walk::FromStart) : SHRIKE_DELTA_BLOCKS_OF(L, Walk::Whole), \
+  gather = SHRIKE_DELTA_BLOCKS_OF(L, Walk::Gather)
     switch (lanes) {
       case 1: SHRIKE_DELTA_BLOCKS(1); break;
       case 2: SHRIKE_DELTA_BLOCKS(2); break;
@@ -1069,24 +1335,56 @@ SHRIKE_API int shrike_delta_scan(const float* mixed, int mixed_partials, long lo
       default: SHRIKE_DELTA_BLOCKS(32); break;
     }
 #undef SHRIKE_DELTA_BLOCKS
+#undef SHRIKE_DELTA_BLOCKS_OF
     const int teams = warps * 32 / lanes;
     size_t smem = (static_cast<size_t>(STAGES) * (b.record + BLOCK * b.s.cols) + static_cast<size_t>(teams) * 2 * BLOCK * 4) * sizeof(float);
     const size_t most = static_cast<size_t>(shrike_device().max_smem);
     if (smem > most) return SHRIKE_BAD_ARGUMENT;
     // The walk's CTAs are few and run long: each asks for so much shared memory that they spread evenly over the SMs
     // instead of being packed where there is room first.
-    const long long ctas = static_cast<long long>(block_slices) * min(head_count, heads) * num_seqs;
-    const long long per_sm = (ctas + sms - 1) / sms;
-    const size_t fair = most / static_cast<size_t>(per_sm) - 2048;
-    if (per_sm <= 8 && fair > smem) smem = fair;
-    if (smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    const auto spread = [&](long long ctas) {
+      const long long per_sm = (ctas + sms - 1) / sms;
+      const size_t fair = most / static_cast<size_t>(per_sm) - 2048;
+      return per_sm <= 8 && fair > smem ? fair : smem;
+    };
+    const size_t kernel_smem = spread(static_cast<long long>(block_slices) * min(head_count, heads) * walks);
+    if (kernel_smem > 48 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(kernel_smem));
+    unsigned gather_slices = block_slices;
+    size_t gather_smem = smem;
+    if (in_runs) {
+      b.run_blocks = run_blocks;
+      b.value_slices = static_cast<int>(block_slices);
+      b.run_values = (vdim + 3) / 4 * 4;
+      b.run_ld = b.run_values + (delta_rule ? b.padded_dim : 0);
+      b.run_states = run_scratch;
+      b.run_decays = run_scratch + static_cast<size_t>(runs) * min(head_count, heads) * dim * b.run_ld;
+      if (delta_rule) gather_slices += static_cast<unsigned>((b.padded_dim + b.s.cols - 1) / b.s.cols);
+      gather_smem = spread(static_cast<long long>(gather_slices) * min(head_count, heads) * runs);
+      if (gather_smem > 48 * 1024) cudaFuncSetAttribute(gather, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(gather_smem));
+    }
     for (int head0 = 0; head0 < heads; head0 += head_count) {
       b.head0 = head0;
       b.head_count = min(head_count, heads - head0);
       void (*local)(BlockArgs) = !delta_rule ? delta_local_kernel<false, false>
                                              : (per_head ? delta_local_kernel<true, true> : delta_local_kernel<true, false>);
       launch_dependent(local, dim3(static_cast<unsigned>(blocks), static_cast<unsigned>((b.head_count + 3) / 4)), 128, 0, stream, b);
-      launch_dependent(kernel, dim3(block_slices, b.head_count, num_seqs), static_cast<unsigned>(warps * 32), smem, stream, b);
+      if (in_runs) {
+        launch_dependent(gather, dim3(gather_slices, b.head_count, runs), static_cast<unsigned>(warps * 32), gather_smem, stream, b);
+        if (delta_rule) {
+          const dim3 grid(static_cast<unsigned>((vdim + CARRY_COLS - 1) / CARRY_COLS), b.head_count, num_seqs);
+          size_t held = static_cast<size_t>(2) * carry_rows(b.padded_dim) * CARRY_COLS * sizeof(float);
+          if (dim <= 128) {
+            held += static_cast<size_t>(2) * dim * carry_pitch(b.padded_dim) * sizeof(float);
+            if (held > 48 * 1024) cudaFuncSetAttribute(delta_carry_kernel<1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(held));
+            launch_dependent(delta_carry_kernel<1, true>, grid, 256, held, stream, b);
+          } else {
+            launch_dependent(delta_carry_kernel<2, false>, grid, 256, held, stream, b);
+          }
+        } else {
+          launch_dependent(gated_carry_kernel, dim3(static_cast<unsigned>((dim * vdim + 255) / 256), b.head_count, num_seqs), 256, 0, stream, b, b.padded_dim);
+        }
+      }
+      launch_dependent(kernel, dim3(block_slices, b.head_count, static_cast<unsigned>(walks)), static_cast<unsigned>(warps * 32), kernel_smem, stream, b);
     }
   }
   return shrike_launch_status();

@@ -900,37 +900,42 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) matrix_memory_out_kernel(cons
 }
 
 // ----------------------------------------------------------------------------------------------- route_top
-// One block a token.  The logits: the block's warps share a row's columns (warp w the w-th run of 128 columns, and
+// A block takes TOK tokens (one where tokens are few, ROUTE_TOKENS in a prompt, whose weight rows are then read once for
+// all of them).  The logits: the block's warps share a row's columns (warp w the w-th run of 128 columns, and
 // so on), experts eight at a time with the eight weight rows' loads in flight together; the warps' sums meet in shared
-// memory in a fixed order.  Then, by the first warp: softmax, `top` rounds of a warp-wide argmax, the sum of the
-// chosen, and the shared expert's gate (its vector is one more row of the product).
+// memory in a fixed order, the same for every TOK.  Then a warp a token: softmax, `top` rounds of a warp-wide argmax, the
+// sum of the chosen, and the shared expert's gate (its vector is one more row of the product).
 constexpr int ROUTE_WARPS = 8;
 constexpr int ROUTE_GROUP = 8;
+constexpr int ROUTE_TOKENS = 4;
 
-template <typename T>
+template <typename T, int TOK>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 route_top_kernel(const T* __restrict__ x, const float* __restrict__ router, const float* __restrict__ shared_gate,
                  float* __restrict__ weights, int n, int width, int experts, int top, int columns, float renorm_eps,
                  int sigmoid_scores, int renormalise, const float* __restrict__ correction, int group_count, int group_keep,
                  int identity) {
-  extern __shared__ float route_shared[];   // [ROUTE_WARPS][rows] sums of the warps, then [rows] scores in the first row
+  extern __shared__ float route_shared[];   // [TOK][ROUTE_WARPS][rows] sums of the warps, then [rows] scores in a token's first row
   let_dependents_start();
-  wait_for_previous();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int token = blockIdx.x;
-  const T* row = x + static_cast<size_t>(token) * width;
-  float* out = weights + static_cast<size_t>(token) * columns;
   // the last `identity` of the `experts` are identity experts: their weights leave as one sum in the last column
   const int real = experts - identity;
   const bool shared_column = columns > real + (identity > 0 ? 1 : 0);
   // rows of the product: the experts, then (when there is one) the shared expert's gate vector
   const int rows = experts + (shared_column && shared_gate != nullptr ? 1 : 0);
+  if (TOK == 1) {   // the router's weights are parameters: they may come nearer while the kernel before still runs
+    const char* first = reinterpret_cast<const char*>(router);
+    const size_t bytes = static_cast<size_t>(experts) * width * sizeof(float);
+    for (size_t at = static_cast<size_t>(threadIdx.x) * 128; at < bytes && at < (256u << 10); at += static_cast<size_t>(blockDim.x) * 128)
+      asm volatile("prefetch.global.L2 [%0];" ::"l"(first + at));
+  }
+  wait_for_previous();
+  const int token0 = blockIdx.x * TOK, here = min(TOK, n - token0);
   const bool wide = (width & 3) == 0 && (reinterpret_cast<uintptr_t>(router) & 15) == 0 &&
                     (shared_gate == nullptr || (reinterpret_cast<uintptr_t>(shared_gate) & 15) == 0) &&
                     (reinterpret_cast<uintptr_t>(x) & 15) == 0;
-  float* partial = route_shared + static_cast<size_t>(warp) * rows;
   for (int e0 = 0; e0 < rows; e0 += ROUTE_GROUP) {
-    float dot[ROUTE_GROUP] = {};
+    float dot[TOK][ROUTE_GROUP] = {};
     const float* from[ROUTE_GROUP];
 #pragma unroll
     for (int g = 0; g < ROUTE_GROUP; ++g) {
@@ -940,35 +945,46 @@ route_top_kernel(const T* __restrict__ x, const float* __restrict__ router, cons
     if (wide) {
 #pragma unroll 2
       for (int c = (warp * 32 + lane) * 4; c < width; c += ROUTE_WARPS * 128) {
-        float xv[4], w[ROUTE_GROUP][4];
-        load4<T>(row + c, xv);
+        float xv[TOK][4], w[ROUTE_GROUP][4];
+#pragma unroll
+        for (int t = 0; t < TOK; ++t) load4<T>(x + static_cast<size_t>(token0 + min(t, here - 1)) * width + c, xv[t]);
 #pragma unroll
         for (int g = 0; g < ROUTE_GROUP; ++g) load4<float>(from[g] + c, w[g]);
 #pragma unroll
-        for (int g = 0; g < ROUTE_GROUP; ++g)
+        for (int t = 0; t < TOK; ++t)
 #pragma unroll
-          for (int k = 0; k < 4; ++k) dot[g] = __fmaf_rn(xv[k], w[g][k], dot[g]);
+          for (int g = 0; g < ROUTE_GROUP; ++g)
+#pragma unroll
+            for (int k = 0; k < 4; ++k) dot[t][g] = __fmaf_rn(xv[t][k], w[g][k], dot[t][g]);
       }
     } else {
       for (int c = warp * 32 + lane; c < width; c += ROUTE_WARPS * 32) {
-        const float xv = to_float(row[c]);
 #pragma unroll
-        for (int g = 0; g < ROUTE_GROUP; ++g) dot[g] = __fmaf_rn(xv, from[g][c], dot[g]);
+        for (int t = 0; t < TOK; ++t) {
+          const float xv = to_float(x[static_cast<size_t>(token0 + min(t, here - 1)) * width + c]);
+#pragma unroll
+          for (int g = 0; g < ROUTE_GROUP; ++g) dot[t][g] = __fmaf_rn(xv, from[g][c], dot[t][g]);
+        }
       }
     }
 #pragma unroll
-    for (int g = 0; g < ROUTE_GROUP; ++g) {
-      const float sum = warp_sum(dot[g]);
-      if (lane == 0 && e0 + g < rows) partial[e0 + g] = sum;
-    }
+    for (int t = 0; t < TOK; ++t)
+#pragma unroll
+      for (int g = 0; g < ROUTE_GROUP; ++g) {
+        const float sum = warp_sum(dot[t][g]);
+        if (lane == 0 && e0 + g < rows) route_shared[static_cast<size_t>(t * ROUTE_WARPS + warp) * rows + e0 + g] = sum;
+      }
   }
   __syncthreads();
-  if (warp != 0) return;
-  float* score = route_shared;
+  if (warp >= here) return;
+  const int token = token0 + warp;
+  float* out = weights + static_cast<size_t>(token) * columns;
+  float* sums = route_shared + static_cast<size_t>(warp) * ROUTE_WARPS * rows;   // this token's
+  float* score = sums;
   float best = -INFINITY;
   for (int e = lane; e < rows; e += 32) {
     float sum = score[e];
-    for (int w = 1; w < ROUTE_WARPS; ++w) sum = __fadd_rn(sum, route_shared[static_cast<size_t>(w) * rows + e]);
+    for (int w = 1; w < ROUTE_WARPS; ++w) sum = __fadd_rn(sum, sums[static_cast<size_t>(w) * rows + e]);
     score[e] = sum;
     if (e < experts) best = fmaxf(best, sum);
   }
@@ -995,7 +1011,7 @@ route_top_kernel(const T* __restrict__ x, const float* __restrict__ router, cons
   if (correction != nullptr || group_count > 0) {
     // the choice goes by score + correction among the experts of the best groups; the weights are the scores.  Rows one
     // and two of the warps' sums are used up: they hold the choice scores and the groups' best.
-    float* choice = route_shared + rows;
+    float* choice = sums + rows;
     float* group_best = choice + rows;
     for (int e = lane; e < experts; e += 32) {
       if (sigmoid_scores) score[e] = 1.0f / (1.0f + expf(-score[e]));
@@ -1360,17 +1376,18 @@ SHRIKE_API int shrike_route_top_groups(const void* x, int dtype, const float* ro
   if (columns != least && columns != least + 1) return SHRIKE_BAD_ARGUMENT;
   if (group_count > 0 && (experts % group_count || group_keep < 1 || group_keep > group_count || top > group_keep * (experts / group_count)))
     return SHRIKE_BAD_ARGUMENT;
-  const unsigned blocks = static_cast<unsigned>(n);
-  const size_t smem = static_cast<size_t>(ROUTE_WARPS) * (experts + 1) * sizeof(float);
-  if (dtype == SHRIKE_F32)
-    launch_dependent(route_top_kernel<float>, blocks, ROUTE_WARPS * 32, smem, stream, static_cast<const float*>(x), router,
-                     shared_gate, weights, n, width, experts, top, columns, renorm_eps, sigmoid_scores, renormalise, correction,
-                     group_count, group_keep, identity);
-  else if (dtype == SHRIKE_BF16)
-    launch_dependent(route_top_kernel<__nv_bfloat16>, blocks, ROUTE_WARPS * 32, smem, stream, static_cast<const __nv_bfloat16*>(x),
-                     router, shared_gate, weights, n, width, experts, top, columns, renorm_eps, sigmoid_scores, renormalise, correction,
-                     group_count, group_keep, identity);
+  const size_t each = static_cast<size_t>(ROUTE_WARPS) * (experts + 1) * sizeof(float);
+  const bool several = n > 4 * shrike_device().sm_count && ROUTE_TOKENS * each <= 48 * 1024;   // enough tokens that blocks of several fill the device
+  const unsigned blocks = static_cast<unsigned>(several ? (n + ROUTE_TOKENS - 1) / ROUTE_TOKENS : n);
+  const size_t smem = several ? ROUTE_TOKENS * each : each;
+#define SHRIKE_ROUTE(T)                                                                                                       \
+  launch_dependent(several ? route_top_kernel<T, ROUTE_TOKENS> : route_top_kernel<T, 1>, blocks, ROUTE_WARPS * 32, smem, stream, \
+                   static_cast<const T*>(x), router, shared_gate, weights, n, width, experts, top, columns, renorm_eps,       \
+                   sigmoid_scores, renormalise, correction, group_count, group_keep, identity)
+  if (dtype == SHRIKE_F32) SHRIKE_ROUTE(float);
+  else if (dtype == SHRIKE_BF16) SHRIKE_ROUTE(__nv_bfloat16);
   else return SHRIKE_BAD_ARGUMENT;
+#undef SHRIKE_ROUTE
   return shrike_launch_status();
 }
 

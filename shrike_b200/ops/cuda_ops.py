@@ -134,6 +134,8 @@ class CudaOps:
         self._decay_scratch = None    # the same for the decayed linear attention: a state per run of tokens
         self._scan_scratch = None     # the gated recurrence's runs of tokens: each run's state, decay and first index
         self._delta_scratch = None    # the delta rule's blocks of tokens: what the walk over them reads
+        self._delta_runs = None       # and, where few walks are cut into runs, what those hand to one another
+        self.delta_run_blocks = None  # None: the kernel library's rule; n: runs of n blocks (0: none; tests)
         self.portion_splits = 0  # 0: the kernel library's rule; n: that many key splits for portions (tests)
         self.generation = 0      # grows when the scratch moves
         self._held_stream = None
@@ -195,7 +197,11 @@ class CudaOps:
         lib.shrike_short_conv_keep.argtypes = [_P, _I, _LL, _I, _P, _P, _P, _I, _I, _I, _I, _P]
         lib.shrike_delta_prep.argtypes = [_P, _I, _LL, _I, _P, _P, _P, _P, _P, _P, _P, _P] + [_I] * 12 + [_F, _F, _I, _P]
         lib.shrike_delta_scan.argtypes = ([_P, _I, _LL, _I, _P, _P, _I, _LL, _I, _I, _I, _P, _P, _F, _F, _P, _P, _P, _P] + [_I] * 9
-                                          + [_P, _I, _I, _I, _P])
+                                          + [_P, _I, _I, _I, _I, _I, _P, _P])
+        lib.shrike_delta_scan_run_blocks.argtypes = [_I] * 7
+        lib.shrike_delta_scan_run_blocks.restype = _I
+        lib.shrike_delta_scan_run_floats.argtypes = [_I, _I, _I]
+        lib.shrike_delta_scan_run_floats.restype = _LL
         lib.shrike_delta_scan_record.argtypes = [_I, _I]
         lib.shrike_low_rank.argtypes = [_P, _I, _LL, _I, _I, _P, _I, _I, _I, _P, _I, _I, _P]
         lib.shrike_sum_norm.argtypes = [_P, _P, _P, _P, _P, _I, _P, _P, _I, _F, _P, _P, _F, _P, _I, _I, _I, _P]
@@ -1291,6 +1297,7 @@ class CudaOps:
                 or (bias is not None and bias.numel() != num_heads * each)):
             raise KernelError(f"state {tuple(state.shape)} does not fit {num_heads} heads of {dim} x {vdim}")
         blocks, records, head_count, shorter = 0, None, 0, True
+        run_blocks, runs, run_scratch = 0, 0, None
         record = 0 if self.delta_walks(dim, q_lens) else self.core.shrike_delta_scan_record(dim, int(beta is not None))
         if record:
             if mixed_partials > 1:
@@ -1305,12 +1312,25 @@ class CudaOps:
                 self._delta_scratch = torch.empty(max(need, 1 << 20), dtype=torch.float32, device=self.device)
                 self.generation += 1
             records = self._delta_scratch
-        self.launches += int(shorter) + (2 * -(-num_heads // head_count) if blocks else 0)
+            counts = [-(-length // size) for length in q_lens if length >= self.DELTA_BLOCKS_FROM]
+            delta = int(beta is not None)
+            run_blocks = self.delta_run_blocks
+            if run_blocks is None:
+                run_blocks = self.core.shrike_delta_scan_run_blocks(blocks, max(counts), len(counts), head_count, dim, vdim, delta)
+            if run_blocks:
+                runs = sum(-(-count // run_blocks) for count in counts)
+                need = runs * head_count * self.core.shrike_delta_scan_run_floats(dim, vdim, delta)
+                if self._delta_runs is None or self._delta_runs.numel() < need:
+                    self._delta_runs = torch.empty(max(need, 1 << 20), dtype=torch.float32, device=self.device)
+                    self.generation += 1
+                run_scratch = self._delta_runs
+        self.launches += int(shorter) + ((4 if run_blocks else 2) * -(-num_heads // head_count) if blocks else 0)
         _check(self.core.shrike_delta_scan(
             _ptr(mixed), mixed_partials, mixed_stride, mixed.shape[-1], _ptr(beta), _ptr(gates), partials, stride, gates.shape[-1],
             gate_at, each, _ptr(rate), _ptr(bias), float(sign), float(q_scale), _ptr(state), _ptr(q_start), _ptr(state_slot), _ptr(out),
             num_seqs, num_heads, num_kv_heads, dim, vdim, state.shape[2], state.shape[0], self.DELTA_BLOCKS_FROM if blocks else 0,
-            int(shorter), _ptr(records), blocks, head_count, int(bool(early_state)), self._stream()), "delta_scan")
+            int(shorter), _ptr(records), blocks, head_count, int(bool(early_state)), run_blocks, runs, _ptr(run_scratch),
+            self._stream()), "delta_scan")
 
     def delta_walks(self, dim, q_lens) -> bool:
         """Whether `delta_scan` walks every sequence of such a batch token by token, so that its input may be a stack."""

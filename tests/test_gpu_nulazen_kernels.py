@@ -176,7 +176,8 @@ def test_delta_scan_whole_walked_and_in_portions(heads, kv_heads, dim, vdim, str
     mixed = torch.cat([q.reshape(n, -1), k.reshape(n, -1), v.reshape(n, -1)], -1).cuda().contiguous()
     gates = torch.cat([z.reshape(n, -1), torch.randn(n, 20)], -1)
     size = -(-dim * vdim // 4) * 4
-    for way, cuts in (("blocks", [n]), ("walk", [n]), ("portions", [1, 2, 37, 16, 1, 1, 15, 17, 8, 52]), ("stack", [n])):
+    for way, cuts in (("blocks", [n]), ("walk", [n]), ("portions", [1, 2, 37, 16, 1, 1, 15, 17, 8, 52]), ("stack", [n]), ("runs", [110, 40])):
+        ops.delta_run_blocks = 3 if way == "runs" else 0   # runs of 24 tokens that walk side by side
         gen = torch.Generator().manual_seed(1)
         state = torch.full((3, heads, size), 5.0, device="cuda")
         state[1] = 0.0

@@ -106,7 +106,7 @@ def test_gelu_inside_and_behind_the_product(dtype, n, inter, width):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("experts,each,n,extra", [(3, 16, 33, 1), (4, 5, 7, 0), (16, 8, 70, 1), (1, 200, 2, 0), (7, 4, 5, 2)])
+@pytest.mark.parametrize("experts,each,n,extra", [(9, 328, 300, 1), (3, 16, 33, 1), (4, 5, 7, 0), (16, 8, 70, 1), (1, 200, 2, 0), (7, 4, 5, 2)])
 def test_ungated_experts_activation_times_their_weight(dtype, experts, each, n, extra):
     ops = cuda_ops(dtype)
     g = torch.Generator().manual_seed(each)
@@ -129,12 +129,14 @@ def test_ungated_experts_activation_times_their_weight(dtype, experts, each, n, 
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("experts,identity,top,width", [(8, 4, 3, 64), (12, 1, 1, 96), (5, 0, 2, 50), (3, 3, 6, 64), (1, 7, 2, 36), (60, 20, 9, 128)])
+@pytest.mark.parametrize("n", [70, 702])
 @pytest.mark.parametrize("correct,renormalise,shared", [(True, False, False), (False, False, True), (False, True, False), (True, True, True)])
-def test_router_with_identity_experts(dtype, experts, identity, top, width, correct, renormalise, shared):
-    """Identity experts take part in scores, choice and weights; what they are given leaves as one sum."""
+def test_router_with_identity_experts(dtype, experts, identity, top, width, n, correct, renormalise, shared):
+    """Identity experts take part in scores, choice and weights; what they are given leaves as one sum.  Many tokens go several to
+    a block, with the same bits."""
     ops = cuda_ops(dtype)
     g = torch.Generator().manual_seed(experts + top)
-    n, outputs = 70, experts + identity
+    outputs = experts + identity
     x = torch.randn(n, width, generator=g).to(dtype)
     router = torch.randn(outputs, width, generator=g) * 0.2
     correction = 0.2 * torch.randn(outputs, generator=g) if correct else torch.zeros(outputs)
@@ -158,6 +160,10 @@ def test_router_with_identity_experts(dtype, experts, identity, top, width, corr
             assert float(want[:, experts:].sum()) > 0
     if shared:
         close(got[:, experts], torch.sigmoid(x.double() @ gate.double()), 1e-5, "shared gate")
+    few = torch.empty(9, out.shape[1], device="cuda")
+    ops.route_top(x[:9].cuda().contiguous(), router.cuda(), gate.cuda() if shared else None, few, top, 1e-9, renormalise=renormalise,
+                  correction=correction.cuda() if correct else None, identity=identity)
+    assert torch.equal(few, out[:9])
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -237,7 +243,9 @@ def test_scan_whole_walked_and_in_portions(heads, kv_heads, dim, vdim, kind, str
     arguments, step = recurrence(kind, n, heads, kv_heads, dim, vdim, dim + heads, strength)
     want, last = step(0, n)
     size = -(-dim * vdim // 4) * 4
-    for way, cuts in (("blocks", [n]), ("walk", [n]), ("portions", [1, 2, 37, 16, 1, 1, 15, 17, 8, 52]), ("stack", [n]), ("walked stack", [n])):
+    for way, cuts in (("blocks", [n]), ("walk", [n]), ("portions", [1, 2, 37, 16, 1, 1, 15, 17, 8, 52]), ("stack", [n]), ("walked stack", [n]),
+                      ("runs", [n]), ("runs of one block", [40, 110]), ("runs in portions", [70, 1, 79])):
+        ops.delta_run_blocks = 1 if "one block" in way else 4 if "runs" in way else 0   # (150 tokens are cut into runs only when asked)
         state = torch.full((3, heads, size), 5.0, device="cuda")
         state[1] = 0.0
         out = torch.empty(n, heads * vdim, device="cuda")
@@ -253,10 +261,13 @@ def test_scan_whole_walked_and_in_portions(heads, kv_heads, dim, vdim, kind, str
 
 
 @pytest.mark.parametrize("kind", ["head", "channel"])
-@pytest.mark.parametrize("heads,kv_heads,dim,vdim", [(4, 2, 64, 32), (3, 3, 20, 36), (2, 1, 128, 100)])
-def test_scan_of_unequal_sequences_with_padding_rows(kind, heads, kv_heads, dim, vdim):
-    """Portions beside single tokens beside rows without a slot, more sequences than a warp has lanes; each as alone."""
+@pytest.mark.parametrize("runs", [0, 3])
+@pytest.mark.parametrize("heads,kv_heads,dim,vdim", [(4, 2, 64, 32), (3, 3, 20, 36), (2, 1, 128, 100), (1, 1, 200, 3)])
+def test_scan_of_unequal_sequences_with_padding_rows(kind, runs, heads, kv_heads, dim, vdim):
+    """Portions beside single tokens beside rows without a slot, more sequences than a warp has lanes; each as alone, also
+    where portions are cut into runs that walk side by side."""
     ops = cuda_ops(torch.float32)
+    ops.delta_run_blocks = runs
     lengths = [1, 40, 1, 16, 15, 9, 200, 1] + [1, 17] * 16
     n, count = sum(lengths), len(lengths)
     arguments, step = recurrence(kind, n, heads, kv_heads, dim, vdim, 3, 0.4)
@@ -286,12 +297,35 @@ def test_scan_takes_heads_in_turns_when_the_scratch_is_bounded(kind):
     heads, dim, vdim, n = 5, 24, 12, 100
     arguments, _ = recurrence(kind, n, heads, heads, dim, vdim, 8, 0.5)
     results = []
+    ops.delta_run_blocks = 4
     for bound in (ops.DELTA_SCRATCH_FLOATS, 2 * 13 * ops.core.shrike_delta_scan_record(dim, int(kind == "head"))):
         ops.DELTA_SCRATCH_FLOATS = bound
         state, out = torch.zeros(1, heads, dim * vdim, device="cuda"), torch.empty(n, heads * vdim, device="cuda")
         scan(ops, arguments(0, n), state, [0, n], [0], out, heads, heads, dim, vdim, [n])
         results.append((out, state))
     assert torch.equal(results[0][0], results[1][0]) and torch.equal(results[0][1], results[1][1])
+
+
+@pytest.mark.parametrize("kind,heads", [("head", 4), ("channel", 4), ("channel", 12)])
+def test_a_long_prompt_is_cut_into_runs(kind, heads):
+    """By the library's own rule: few heads and 1,500 tokens in runs, many sequences not; the same numbers either way."""
+    ops = cuda_ops(torch.float32)
+    dim = vdim = 128
+    n = 1500
+    blocks = -(-n // 8)
+    assert ops.core.shrike_delta_scan_run_blocks(blocks, blocks, 1, heads, dim, vdim, int(kind == "head")) >= 16
+    assert ops.core.shrike_delta_scan_run_blocks(64 * blocks, blocks, 64, heads, dim, vdim, int(kind == "head")) == 0
+    assert ops.core.shrike_delta_scan_run_blocks(8, 8, 1, heads, dim, vdim, int(kind == "head")) == 0
+    arguments, step = recurrence(kind, n, heads, heads, dim, vdim, 4, 0.1)
+    want, last = step(0, n)
+    for runs in (None, 0):
+        ops.delta_run_blocks = runs
+        state, out = torch.zeros(1, heads, dim * vdim, device="cuda"), torch.empty(n, heads * vdim, device="cuda")
+        before = ops.launches
+        scan(ops, arguments(0, n), state, [0, n], [0], out, heads, heads, dim, vdim, [n])
+        assert ops.launches - before == (4 if runs is None else 2)
+        close(out.view(n, heads, vdim), want, 2e-5, f"runs {runs}")
+        close(state[0].view(heads, dim, vdim), last, 2e-5, f"state, runs {runs}")
 
 
 def test_scan_refuses_what_no_kernel_serves():
